@@ -7,12 +7,12 @@ hand-written sm_100a CUDA kernels behind a C ABI (include/cdeep.h, libcdeep.so).
 from .core import (RMSNorm, RotaryEmbedding, ComplexityAttention, SwiGLU, TokenRoutedMLP,
                    TransformerBlock, MuGuidance)
 from .models import (ComplexityConfig, ComplexityModel, create_complexity_model,
-                     count_parameters)
+                     count_parameters, PimezenConfig, PimezenModel, load_model)
 
 __version__ = "1.0.0"
 
 __all__ = [
     "RMSNorm", "RotaryEmbedding", "ComplexityAttention", "SwiGLU", "TokenRoutedMLP",
     "TransformerBlock", "MuGuidance", "ComplexityConfig", "ComplexityModel",
-    "create_complexity_model", "count_parameters",
+    "create_complexity_model", "count_parameters", "PimezenConfig", "PimezenModel", "load_model",
 ]

@@ -14,6 +14,30 @@ CHECKS_LIB_PATH = os.path.join(os.path.dirname(os.path.abspath(__file__)), "libc
 
 ABI_VERSION = 3
 
+
+
+class WindowAttn(ctypes.Structure):
+    """cd_window_attn of include/cdeep.h."""
+    _fields_ = ([(n, c_void_p) for n in ("q", "k", "v")] + [("ldp", c_longlong)]
+                + [(n, c_void_p) for n in ("q_w", "k_w", "r1", "r2", "talk", "ring_k", "ring_v", "out")]
+                + [("ldo", c_longlong), ("pos_dev", c_void_p)]
+                + [(n, c_float) for n in ("scale", "eps", "out_scale")]
+                + [(n, c_int) for n in ("B", "S", "H", "G", "dim", "dp", "vdim", "vp", "window", "keep",
+                                        "pos0", "normed")])
+
+
+class LinearAttn(ctypes.Structure):
+    """cd_linear_attn of include/cdeep.h."""
+    _fields_ = ([(n, c_void_p) for n in ("q", "k", "v", "gate", "inner")] + [("ldp", c_longlong)]
+                + [(n, c_void_p) for n in ("a2", "a2_b", "norm_w", "state", "out")]
+                + [("ldo", c_longlong), ("log_decay", c_void_p), ("o_raw", c_void_p)]
+                + [(n, c_float) for n in ("inv_tau", "eps", "out_scale", "q_scale")]
+                + [(n, c_int) for n in ("B", "S", "H", "dk", "dkp", "dv", "dvp", "rank")])
+
+
+_WINDOW_FN = (c_int, [ctypes.POINTER(WindowAttn), c_int, c_void_p])
+_GLA_FN = (c_int, [ctypes.POINTER(LinearAttn), c_int, c_void_p])
+
 # name -> (restype, argtypes); mirrors include/cdeep.h one to one
 SIGNATURES = {
     "cd_version": (c_int, []),
@@ -82,6 +106,22 @@ SIGNATURES = {
                            c_void_p, c_int, c_int, c_void_p]),
     "cd_linear": (c_int, [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
                           c_int, c_int, c_void_p]),
+    "cd_embed_rows": (c_int, [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p]),
+    "cd_rmsnorm_f32": (c_int, [c_void_p, c_void_p, c_float, c_float, c_void_p, c_int, c_int, c_int, c_int, c_void_p]),
+    "cd_linear_f32out": (c_int, [c_void_p] * 5 + [c_int, c_int, c_int, c_void_p]),
+    "cd_linear_f32": (c_int, [c_void_p] * 5 + [c_int, c_int, c_int, c_void_p]),
+    "cd_glu_up": (c_int, [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_float, c_float,
+                          c_void_p]),
+    "cd_glu_f32": (c_int, [c_void_p, c_void_p, c_int, c_int, c_float, c_float, c_float, c_void_p]),
+    "cd_window_attention_supported": (c_int, [ctypes.POINTER(WindowAttn)]),
+    "cd_window_attention_norm": _WINDOW_FN,
+    "cd_window_attention_rows": _WINDOW_FN,
+    "cd_window_attention_append": _WINDOW_FN,
+    "cd_gla_supported": (c_int, [ctypes.POINTER(LinearAttn)]),
+    "cd_gla_step": _GLA_FN,
+    "cd_gla_decay": _GLA_FN,
+    "cd_gla_sequence": _GLA_FN,
+    "cd_gla_finish": _GLA_FN,
 }
 
 _lib = None

@@ -109,10 +109,18 @@ class StaticKVCache:
         self.length = length
         self.state.copy_(torch.tensor([length, length + 1], dtype=torch.int32), non_blocking=False)
 
-    def advance(self) -> None:
-        """One token was appended to every layer: move the device-side position (stream
-        ordered, capturable) and its host mirror."""
+    def as_past(self) -> list:
+        """What a forward call takes as ``past_key_values``."""
+        return self.layers
+
+    def advance_device(self) -> None:
+        """Moves the device-side position by one token (stream ordered, capturable)."""
         self.state.add_(1)
+
+    def advance(self) -> None:
+        """One token was appended to every layer: move the device-side position and its host
+        mirror."""
+        self.advance_device()
         self.length += 1
 
 

@@ -6,6 +6,8 @@ import torch
 import torch.nn as nn
 
 from .. import ops
+from ._cache import DerivedCache
+from .padding import pad_vector
 
 
 class RMSNorm(nn.Module):
@@ -22,3 +24,23 @@ class RMSNorm(nn.Module):
 
     def extra_repr(self) -> str:
         return f"{self.weight.numel()}, eps={self.eps}"
+
+
+class StreamNorm(nn.Module):
+    """RMSNorm of the fp32 residual stream into the weights' dtype:
+    y = x / sqrt(mean(x^2) + eps) * (offset + weight); offset 1 for a weight stored around zero."""
+
+    def __init__(self, hidden_size: int, eps: float, offset: float = 0.0):
+        super().__init__()
+        self.eps, self.offset = eps, offset
+        self.weight = nn.Parameter(torch.full((hidden_size,), 1.0 - offset))
+        self._derived = DerivedCache()
+
+    def forward(self, stream: torch.Tensor) -> torch.Tensor:
+        """stream [T, width padded] fp32 -> [T, width padded]; the padding stays zero."""
+        w = self._derived.get("weight", (self.weight,),
+                              lambda: pad_vector(self.weight.detach(), stream.shape[1]))
+        return ops.rmsnorm_f32(stream, w, self.eps, self.offset, width=self.weight.numel())
+
+    def extra_repr(self) -> str:
+        return f"{self.weight.numel()}, eps={self.eps}, offset={self.offset}"

@@ -554,4 +554,162 @@ int cd_linear(const void* x, const void* w, const void* residual, const void* re
                      choose_store_block_n(T, N, 1, current_sm_count()), as_stream(stream));
 }
 
+int cd_embed_rows(const int64_t* ids, const void* table, float* x, int T, int V, int W, int ldw, int ldx,
+                  int fp32, void* stream) {
+  if (T < 0 || V < 1 || W < 1 || ldw < W || ldx < W || (ldx & 7) || !table) return CD_ERR_INVALID;
+  if (T > 0 && (!ids || !x || !aligned16(x))) return CD_ERR_INVALID;
+  cudaError_t e = launch_embed_rows(reinterpret_cast<const long long*>(ids), table, x, T, V, W, ldw, ldx, fp32,
+                                    as_stream(stream));
+  return e == cudaSuccess ? CD_OK : cuda_fail(e, "embed_rows launch");
+}
+
+int cd_rmsnorm_f32(const float* x, const void* w, float eps, float offset, void* out, int T, int W, int ldx,
+                   int fp32, void* stream) {
+  if (T < 0 || W < 1 || ldx < W || (ldx & 7) || !w || !aligned16(w)) return CD_ERR_INVALID;
+  if (T > 0 && (!x || !out || !aligned16(x) || !aligned16(out))) return CD_ERR_INVALID;
+  cudaError_t e = launch_rmsnorm_f32(x, w, eps, offset, out, T, W, ldx, fp32, as_stream(stream));
+  return e == cudaSuccess ? CD_OK : cuda_fail(e, "rmsnorm_f32 launch");
+}
+
+int cd_linear_f32out(const void* x, const void* w, const float* residual, const void* col_scale, float* out,
+                     int T, int K, int N, void* stream) {
+  if (T < 0 || K < 8 || (K & 7) || N < 8 || (N & 7)) return CD_ERR_INVALID;
+  GemmOperand op0{};
+  op0.a = x;
+  op0.lda = K;
+  op0.b = w;
+  op0.ldb = K;
+  op0.b_rows = N;
+  op0.K = K;
+  GemmEpilogueArgs epi{};
+  epi.kind = kEpiStoreF32;
+  epi.out = out;
+  epi.ldo = N;
+  epi.out_cols = N;
+  epi.residual = residual;
+  epi.ldr = N;
+  epi.col_scale = col_scale;
+  return launch_gemm(T, N, 1, nullptr, op0, nullptr, epi, choose_store_block_n(T, N, 1, current_sm_count()),
+                     as_stream(stream));
+}
+
+int cd_linear_f32(const float* x, const float* w, const float* residual, const float* col_scale, float* out, int T,
+                  int K, int N, void* stream) {
+  if (T < 0 || K < 4 || (K & 3) || N < 1) return CD_ERR_INVALID;
+  if (T > 0 && (!x || !w || !out || !aligned16(x) || !aligned16(w))) return CD_ERR_INVALID;
+  cudaError_t e = launch_linear_f32(x, w, residual, col_scale, out, T, K, N, as_stream(stream));
+  return e == cudaSuccess ? CD_OK : cuda_fail(e, "linear_f32 launch");
+}
+
+int cd_glu_up(const void* x, const void* packed_w, void* h, int T, int H, int I, int block_n, float alpha,
+              float limit, float offset, void* stream) {
+  if (T < 0 || H < 8 || I < 8 || (H & 7) || (I & 7)) return CD_ERR_INVALID;
+  const int rows = cd_gate_up_packed_rows(I, block_n);
+  if (rows == 0) return CD_ERR_INVALID;
+  GemmOperand op{};
+  op.a = x;
+  op.lda = H;
+  op.b = packed_w;
+  op.ldb = H;
+  op.b_rows = rows;
+  op.K = H;
+  GemmEpilogueArgs epi{};
+  epi.kind = kEpiGlu;
+  epi.out = h;
+  epi.ldo = I;
+  epi.out_cols = I;
+  epi.glu_alpha = alpha;
+  epi.glu_limit = limit;
+  epi.glu_offset = offset;
+  return launch_gemm(T, rows, 1, nullptr, op, nullptr, epi, block_n, as_stream(stream));
+}
+
+int cd_glu_f32(const float* gu, float* h, int T, int I, float alpha, float limit, float offset, void* stream) {
+  if (T < 0 || I < 1 || (T > 0 && (!gu || !h))) return CD_ERR_INVALID;
+  cudaError_t e = launch_glu_f32(gu, h, T, I, alpha, limit, offset, as_stream(stream));
+  return e == cudaSuccess ? CD_OK : cuda_fail(e, "glu_f32 launch");
+}
+
+static int window_args_ok(const cd_window_attn* a) {
+  if (!a || a->B < 0 || a->S < 0 || a->B > 65535 || a->H < 1 || a->G < 1 || a->H % a->G || a->dim < 1 ||
+      a->vdim < 1 || a->dp < a->dim || a->vp < a->vdim || (a->dp & 15) || (a->vp & 15) || a->window < 1 ||
+      a->keep < 0 || a->pos0 < 0 || (a->ldp & 7) || (a->ldo & 7))
+    return CD_ERR_INVALID;
+  if (!a->q || !a->k || !a->v || !a->q_w || !a->k_w || !aligned16(a->q) || !aligned16(a->k) || !aligned16(a->v) ||
+      !aligned16(a->q_w) || !aligned16(a->k_w) || !aligned16(a->ring_k) || !aligned16(a->ring_v) ||
+      !aligned16(a->out))
+    return CD_ERR_INVALID;
+  return CD_OK;
+}
+
+int cd_window_attention_supported(const cd_window_attn* a) { return a && window_rows_supported(*a) ? 1 : 0; }
+
+int cd_window_attention_norm(const cd_window_attn* a, int fp32, void* stream) {
+  if (window_args_ok(a) != CD_OK) return CD_ERR_INVALID;
+  cudaError_t e = launch_head_norm(*a, fp32, as_stream(stream));
+  return e == cudaSuccess ? CD_OK : cuda_fail(e, "head norm launch");
+}
+
+int cd_window_attention_rows(const cd_window_attn* a, int fp32, void* stream) {
+  if (window_args_ok(a) != CD_OK || !a->r1 || !a->r2 || !a->talk || !a->ring_k || !a->ring_v || !a->out ||
+      (!a->normed && a->S != 1))
+    return CD_ERR_INVALID;
+  if (!window_rows_supported(*a)) return CD_ERR_UNSUPPORTED;
+  cudaError_t e = launch_window_rows(*a, fp32, as_stream(stream));
+  return e == cudaSuccess ? CD_OK : cuda_fail(e, "window attention launch");
+}
+
+int cd_window_attention_append(const cd_window_attn* a, int fp32, void* stream) {
+  if (window_args_ok(a) != CD_OK || !a->ring_k || !a->ring_v) return CD_ERR_INVALID;
+  cudaError_t e = launch_window_append(*a, fp32, as_stream(stream));
+  return e == cudaSuccess ? CD_OK : cuda_fail(e, "window append launch");
+}
+
+static int gla_args_ok(const cd_linear_attn* a) {
+  if (!a || a->B < 0 || a->S < 0 || a->B > 65535 || a->H < 1 || a->H > 65535 || a->dk < 1 || a->dv < 1 ||
+      a->dkp < a->dk || a->dvp < a->dv || (a->dkp & 15) || (a->dvp & 15) || a->rank < 8 || (a->rank & 7) ||
+      (a->ldp & 7) || (a->ldo & 7))
+    return CD_ERR_INVALID;
+  if (!a->q || !a->k || !a->v || !a->gate || !a->inner || !a->a2 || !a->a2_b || !a->norm_w || !a->state ||
+      !a->out || !aligned16(a->q) || !aligned16(a->k) || !aligned16(a->v) || !aligned16(a->gate) ||
+      !aligned16(a->inner) || !aligned16(a->a2) || !aligned16(a->state) || !aligned16(a->out) ||
+      !aligned16(a->norm_w))
+    return CD_ERR_INVALID;
+  return linear_attention_supported(a->dkp, a->dvp) ? CD_OK : CD_ERR_UNSUPPORTED;
+}
+
+int cd_gla_supported(const cd_linear_attn* a) { return a && linear_attention_supported(a->dkp, a->dvp) ? 1 : 0; }
+
+int cd_gla_step(const cd_linear_attn* a, int fp32, void* stream) {
+  const int st = gla_args_ok(a);
+  if (st != CD_OK) return st;
+  if (a->S != 1) return CD_ERR_INVALID;
+  cudaError_t e = launch_gla_step(*a, fp32, as_stream(stream));
+  return e == cudaSuccess ? CD_OK : cuda_fail(e, "gla step launch");
+}
+
+int cd_gla_decay(const cd_linear_attn* a, int fp32, void* stream) {
+  const int st = gla_args_ok(a);
+  if (st != CD_OK) return st;
+  if (!a->log_decay) return CD_ERR_INVALID;
+  cudaError_t e = launch_gla_decay(*a, fp32, as_stream(stream));
+  return e == cudaSuccess ? CD_OK : cuda_fail(e, "gla decay launch");
+}
+
+int cd_gla_sequence(const cd_linear_attn* a, int fp32, void* stream) {
+  const int st = gla_args_ok(a);
+  if (st != CD_OK) return st;
+  if (!a->log_decay || !a->o_raw) return CD_ERR_INVALID;
+  cudaError_t e = launch_gla_sequence(*a, fp32, as_stream(stream));
+  return e == cudaSuccess ? CD_OK : cuda_fail(e, "gla sequence launch");
+}
+
+int cd_gla_finish(const cd_linear_attn* a, int fp32, void* stream) {
+  const int st = gla_args_ok(a);
+  if (st != CD_OK) return st;
+  if (!a->o_raw) return CD_ERR_INVALID;
+  cudaError_t e = launch_gla_finish(*a, fp32, as_stream(stream));
+  return e == cudaSuccess ? CD_OK : cuda_fail(e, "gla finish launch");
+}
+
 }  // extern "C"

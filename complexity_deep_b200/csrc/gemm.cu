@@ -93,7 +93,7 @@ bool make_map(CUtensorMap* m, const void* base, long long rows, long long cols, 
 
 struct DeviceInfo {
   int sm_count = 0;
-  bool attr_set[4][4][2] = {};  // [BN 32/64/128/256][epilogue][CTA group 1/2]
+  bool attr_set[4][kNumEpilogues][2] = {};  // [BN 32/64/128/256][epilogue][CTA group 1/2]
   int* status = nullptr;
   void* sk_ws = nullptr;        // split-K workspace registered by the caller (nullptr = split-K off)
   size_t sk_bytes = 0;
@@ -150,6 +150,19 @@ template <int CG>
 cudaError_t launch_any(int block_n, int kind, int grid, const CUtensorMap& a0,
                        const CUtensorMap& b0, const CUtensorMap& a1, const CUtensorMap& b1,
                        const GemmParams& p, DeviceInfo& di, cudaStream_t stream) {
+  if (kind == kEpiStoreF32 || kind == kEpiGlu) {
+#define CDEEP_GEMM_CASE(BN)                                                                        \
+  return kind == kEpiGlu ? launch_one<BN, kEpiGlu, CG>(grid, a0, b0, a1, b1, p, di, stream)       \
+                         : launch_one<BN, kEpiStoreF32, CG>(grid, a0, b0, a1, b1, p, di, stream);
+    if (block_n == 256) { CDEEP_GEMM_CASE(256) }
+    if (block_n == 128) { CDEEP_GEMM_CASE(128) }
+    if constexpr (CG == 1) {
+      if (block_n == 64) { CDEEP_GEMM_CASE(64) }
+      if (block_n == 32) { CDEEP_GEMM_CASE(32) }
+    }
+#undef CDEEP_GEMM_CASE
+    return cudaErrorInvalidValue;
+  }
   if (block_n == 256) {
     if (kind == kEpiStoreRope) return launch_one<256, kEpiStoreRope, CG>(grid, a0, b0, a1, b1, p, di, stream);
     if (kind == kEpiStoreSplit) return launch_one<256, kEpiStoreSplit, CG>(grid, a0, b0, a1, b1, p, di, stream);
@@ -402,6 +415,11 @@ int launch_gemm(int M, int N, int num_groups, const int* seg_offsets, const Gemm
       (epi.kind != kEpiStore || epi.out_row_ptrs || !epi.out || !aligned16(epi.out_lo) ||
        !aligned16(epi.residual_lo) || (epi.residual_lo && !epi.residual)))
     return CD_ERR_INVALID;
+  if (epi.kind == kEpiStoreF32 &&
+      (epi.row_map || epi.out_row_ptrs || epi.residual2 || epi.bias || epi.do_clamp || epi.rope_cos ||
+       epi.out_lo || epi.residual_lo || !epi.out || !aligned16(epi.col_scale) || num_groups != 1))
+    return CD_ERR_INVALID;
+  if (epi.kind != kEpiStoreF32 && epi.col_scale) return CD_ERR_INVALID;
   if (second && (epi.kind != kEpiSwiGLU || op1 || !second->b || !second->out || second->n_rows <= 0 ||
                  (second->ldb & 7) || (second->ldo & 7) || (second->out_cols & 7) ||
                  !aligned16(second->b) || !aligned16(second->out)))
@@ -414,7 +432,7 @@ int launch_gemm(int M, int N, int num_groups, const int* seg_offsets, const Gemm
 
   // dense store-epilogue calls of few rows may take the cluster form of split-K (128-wide tiles)
   int csk_splits = 1;
-  if (num_groups == 1 && !second && epi.kind == kEpiStore && !epi.rope_cos && !epi.selftest_stall &&
+  if (num_groups == 1 && !second && (epi.kind == kEpiStore || epi.kind == kEpiStoreF32) && !epi.rope_cos && !epi.selftest_stall &&
       !epi.out_row_ptrs && block_n <= 128 && choose_cta_group(M, 128, di->sm_count) == 1) {
     const int kb64 = (op0.K + kBoxK - 1) / kBoxK + (op1 ? (op1->K + kBoxK - 1) / kBoxK : 0);
     csk_splits = plan_cluster_split(M, N, kb64, block_n, di->sm_count).splits;
@@ -484,6 +502,10 @@ int launch_gemm(int M, int N, int num_groups, const int* seg_offsets, const Gemm
   p.do_clamp = epi.do_clamp;
   p.clamp_lo = epi.clamp_lo;
   p.clamp_hi = epi.clamp_hi;
+  p.col_scale = static_cast<const __nv_bfloat16*>(epi.col_scale);
+  p.glu_alpha = epi.glu_alpha;
+  p.glu_limit = epi.glu_limit;
+  p.glu_offset = epi.glu_offset;
   p.rope_cos = epi.rope_cos;
   p.rope_sin = epi.rope_sin;
   p.rope_qw = static_cast<const __nv_bfloat16*>(epi.rope_qw);
@@ -511,7 +533,7 @@ int launch_gemm(int M, int N, int num_groups, const int* seg_offsets, const Gemm
     const int kblock = kBoxK * gemm_k_boxes(block_n, cg);
     const int kb_total = (op0.K + kblock - 1) / kblock + (op1 ? (op1->K + kblock - 1) / kblock : 0);
     const bool eligible = cg == 1 && num_groups == 1 && !second && !epi.rope_cos &&
-                          !epi.selftest_stall && (epi.kind != kEpiSwiGLU || block_n >= 64);
+                          !epi.selftest_stall && ((epi.kind != kEpiSwiGLU && epi.kind != kEpiGlu) || block_n >= 64);
     const int splits = (eligible && csk_splits == 1)
                            ? plan_splits(*di, M, N, block_n, kb_total, gemm_k_boxes(block_n, cg)) : 1;
     if (csk_splits > 1) {

@@ -50,7 +50,11 @@ enum GemmEpilogue : int {
   kEpiStoreRope = 2,  // store with per-head RMSNorm + rotary embedding (256-wide tiles only)
   kEpiStoreSplit = 3, // store of a split-bf16 value: out = bf16(v), out_lo = bf16(v - out); the
                       // residual may be split the same way (residual + residual_lo)
+  kEpiStoreF32 = 4,   // fp32 store: out[r, n] = residual[r, n] + col_scale[n] * acc (residual fp32, may be out)
+  kEpiGlu = 5,        // out[r, j] = g * sigmoid(alpha g) * (u + offset), g = min(gate, limit),
+                      // u = clamp(up, -limit, limit)
 };
+constexpr int kNumEpilogues = 6;
 
 // Warp roles: warp 0 TMA producer, warp 1 MMA issuer + TMEM owner, warps 2 .. 2 + EW - 1
 // epilogue.  A warp may only read the TMEM lane quarter (warp id % 4); with EW = 8 two warps
@@ -103,6 +107,8 @@ struct GemmParams {
   float bias_lo, bias_hi;
   int do_clamp;            // clamp the result to [clamp_lo, clamp_hi]
   float clamp_lo, clamp_hi;
+  const __nv_bfloat16* col_scale;  // kEpiStoreF32: factor per output column (nullptr = 1)
+  float glu_alpha, glu_limit, glu_offset;   // kEpiGlu
   // optional: per-head RMSNorm + rotary embedding on the first rope_cols output columns
   // (heads of 128 columns; store epilogue with 256-wide tiles only, no residual / bias)
   const float* rope_cos;   // [positions, 128] fp32 (nullptr = off)
@@ -210,6 +216,12 @@ __device__ __forceinline__ uint4 ld_nc_v4(const void* p) {
 }
 
 __device__ __forceinline__ float silu_f(float g) { return g / (1.0f + __expf(-g)); }
+// clamped gated unit: both factors limited before the gate's sigmoid (of slope alpha)
+__device__ __forceinline__ float clamped_glu_f(float g, float u, float alpha, float limit, float offset) {
+  g = fminf(g, limit);
+  u = fminf(fmaxf(u, -limit), limit);
+  return g / (1.0f + __expf(-alpha * g)) * (u + offset);
+}
 
 __device__ __forceinline__ uint32_t pack_bf16x2(float lo, float hi) {
   __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
@@ -226,8 +238,10 @@ gemm_bf16_sm100_kernel(const __grid_constant__ CUtensorMap tmA0,
                        const __grid_constant__ CUtensorMap tmB1, const GemmParams p) {
   constexpr int EW = gemm_epi_warps<BN, EPI>();
   constexpr int kEpiHalves = EW / 4;               // epilogue warps per TMEM lane quarter
-  constexpr bool kStore = (EPI == kEpiStore || EPI == kEpiStoreRope || EPI == kEpiStoreSplit);
+  constexpr bool kStore = (EPI == kEpiStore || EPI == kEpiStoreRope || EPI == kEpiStoreSplit ||
+                           EPI == kEpiStoreF32);
   constexpr bool kSplit = (EPI == kEpiStoreSplit);
+  constexpr bool kF32 = (EPI == kEpiStoreF32);
   using L = GemmSmem<BN, CG, EW>;
   constexpr int S = L::kStages;
   constexpr int kKBoxes = L::kKBoxes;
@@ -525,8 +539,9 @@ gemm_bf16_sm100_kernel(const __grid_constant__ CUtensorMap tmA0,
         }
       }
       // output columns of this tile and the number of sub-tiles (64 columns; 32 for the split
-      // store, whose staged rows hold 64 bytes of high parts followed by 64 bytes of low parts)
-      constexpr int kSubCols = kSplit ? 32 : kEpiCols;
+      // store, whose staged rows hold 64 bytes of high parts followed by 64 bytes of low parts,
+      // and for the fp32 store)
+      constexpr int kSubCols = (kSplit || kF32) ? 32 : kEpiCols;
       // cluster split-K: this CTA finishes only its slice of the tile's columns
       const int sk_col_lo = csk ? sp * (BN / splits) : 0;
       const int ocol_base = (kStore ? c.n0 : c.n0 / 2) + sk_col_lo;
@@ -539,6 +554,21 @@ gemm_bf16_sm100_kernel(const __grid_constant__ CUtensorMap tmA0,
       // i-th sub-tile of THIS warp (sub-tile index ehalf + i * kEpiHalves of the tile)
       auto fetch_residual = [&](int i) {
         uint8_t* buf = stage0 + (i & 1) * kEpiStageBytes;
+        if constexpr (kF32) {
+          const int col = ocol_base + (ehalf + i * kEpiHalves) * kSubCols + cchunk * 4;
+          if (col < col_end) {
+#pragma unroll
+            for (int it = 0; it < 8; ++it) {
+              if ((cvalid >> it) & 1u) {
+                const int rr = it * 4 + crow_l;
+                cp_async_16(buf + rr * 128 + ((cchunk ^ (rr & 7)) << 4),
+                            reinterpret_cast<const float*>(p.residual) + static_cast<long long>(crow[it]) * p.ldr + col);
+              }
+            }
+          }
+          cp_async_commit();
+          return;
+        }
         // split store: chunks 0-3 of a staged row come from the high part, 4-7 from the low part
         const __nv_bfloat16* src = (kSplit && cchunk >= 4) ? p.residual_lo : p.residual;
         const int col = ocol_base + (ehalf + i * kEpiHalves) * kSubCols +
@@ -753,6 +783,20 @@ gemm_bf16_sm100_kernel(const __grid_constant__ CUtensorMap tmA0,
 
       // coalesced copy-out of one staged 32 x 64 sub-tile: 4 rows x 128 bytes per warp instruction
       auto copy_out = [&](const uint8_t* buf, int col0) {
+        if constexpr (kF32) {
+          const int col = col0 + cchunk * 4;
+          if (col < col_end) {
+#pragma unroll
+            for (int it = 0; it < 8; ++it) {
+              if ((cvalid >> it) & 1u) {
+                const int rr = it * 4 + crow_l;
+                const uint4 o = *reinterpret_cast<const uint4*>(buf + rr * 128 + ((cchunk ^ (rr & 7)) << 4));
+                *reinterpret_cast<uint4*>(reinterpret_cast<float*>(p.out) + static_cast<long long>(crow[it]) * p.ldo + col) = o;
+              }
+            }
+          }
+          return;
+        }
         // split store: lanes with chunks 0-3 write the high parts to `out`, 4-7 the low parts to
         // `out_lo` (64 bytes per row and destination)
         __nv_bfloat16* base = (kSplit && cchunk >= 4) ? p.out_lo : out_base;
@@ -864,7 +908,59 @@ gemm_bf16_sm100_kernel(const __grid_constant__ CUtensorMap tmA0,
       for (int i = 0, sub = ehalf; sub < nsub; ++i, sub += kEpiHalves) {
         uint8_t* buf = stage0 + (i & 1) * kEpiStageBytes;
         const int col0 = ocol_base + sub * kSubCols;
-        if constexpr (kSplit) {
+        if constexpr (kF32) {
+          // one round of 32 accumulator columns: v = residual + col_scale * acc, kept in fp32
+          uint4 sc[4];
+          if (p.col_scale) {
+#pragma unroll
+            for (int q = 0; q < 4; ++q)
+              if (col0 + q * 8 < col_end) sc[q] = *reinterpret_cast<const uint4*>(p.col_scale + col0 + q * 8);
+          }
+          uint32_t v[32];
+          tmem_ld32(t_row + sub * 32, v);
+          if constexpr (kChains == 2) {
+            uint32_t v2[32];
+            tmem_ld32(t_row + BN + sub * 32, v2);
+            tmem_ld_wait();
+#pragma unroll
+            for (int j = 0; j < 32; ++j)
+              v[j] = __float_as_uint(__uint_as_float(v[j]) + __uint_as_float(v2[j]));
+          }
+          if (has_res) {
+            if (sub + kEpiHalves < nsub) cp_async_wait<1>(); else cp_async_wait<0>();
+            __syncwarp();
+          }
+          tmem_ld_wait();
+          if (sk_row || csk) sk_sum(sub * 32, v);
+#pragma unroll
+          for (int q = 0; q < 4; ++q) {
+            if (col0 + q * 8 < col_end) {
+              float f[8];
+#pragma unroll
+              for (int j = 0; j < 8; ++j) f[j] = __uint_as_float(v[q * 8 + j]);
+              if (p.col_scale) {
+                const uint32_t sw[4] = {sc[q].x, sc[q].y, sc[q].z, sc[q].w};
+#pragma unroll
+                for (int j = 0; j < 4; ++j) {
+                  f[2 * j] *= bf16_lo(sw[j]);
+                  f[2 * j + 1] *= bf16_hi(sw[j]);
+                }
+              }
+#pragma unroll
+              for (int e = 0; e < 2; ++e) {
+                float4* slot = reinterpret_cast<float4*>(buf + own_off + (((2 * q + e) ^ (lane & 7)) << 4));
+                if (has_res && row_ok) {
+                  const float4 rr = *slot;
+                  f[4 * e] += rr.x;
+                  f[4 * e + 1] += rr.y;
+                  f[4 * e + 2] += rr.z;
+                  f[4 * e + 3] += rr.w;
+                }
+                *slot = make_float4(f[4 * e], f[4 * e + 1], f[4 * e + 2], f[4 * e + 3]);
+              }
+            }
+          }
+        } else if constexpr (kSplit) {
           // one round of 32 accumulator columns: v = acc + bias + residual (high + low) + residual2,
           // stored as hi = bf16(v) and lo = bf16(v - hi)
           uint4 r2[4];
@@ -1069,7 +1165,10 @@ gemm_bf16_sm100_kernel(const __grid_constant__ CUtensorMap tmA0,
               float h[8];
 #pragma unroll
               for (int j = 0; j < 8; ++j)
-                h[j] = silu_f(__uint_as_float(g[q * 8 + j])) * __uint_as_float(u[q * 8 + j]);
+                h[j] = (EPI == kEpiGlu)
+                           ? clamped_glu_f(__uint_as_float(g[q * 8 + j]), __uint_as_float(u[q * 8 + j]),
+                                           p.glu_alpha, p.glu_limit, p.glu_offset)
+                           : silu_f(__uint_as_float(g[q * 8 + j])) * __uint_as_float(u[q * 8 + j]);
               uint4 o;
               o.x = pack_bf16x2(h[0], h[1]);
               o.y = pack_bf16x2(h[2], h[3]);

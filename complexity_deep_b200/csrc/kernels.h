@@ -3,6 +3,7 @@
 #include <cstddef>
 #include <cstdlib>
 #include <cuda_runtime.h>
+#include "../../include/cdeep.h"
 
 namespace cdeep {
 
@@ -98,6 +99,27 @@ cudaError_t launch_decode_attention(const void* q, long long q_stride_b, const v
                                     int L, int D, void* out, void* ws, cudaStream_t stream,
                                     const int* kv_len_dev = nullptr);
 
+// fp32 residual stream (stream_f32.cu)
+cudaError_t launch_embed_rows(const long long* ids, const void* table, float* x, int T, int V, int W, int ldw,
+                              int ldx, int fp32, cudaStream_t stream);
+cudaError_t launch_rmsnorm_f32(const float* x, const void* w, float eps, float offset, void* out, int rows, int W,
+                               int ldx, int fp32, cudaStream_t stream);
+cudaError_t launch_linear_f32(const float* a, const float* b, const float* residual, const float* col_scale,
+                              float* out, int M, int K, int N, cudaStream_t stream);
+cudaError_t launch_glu_f32(const float* gu, float* h, int T, int I, float alpha, float limit, float offset,
+                           cudaStream_t stream);
+
+// window attention (window_attention.cu) and gated linear attention (linear_attention.cu)
+bool window_rows_supported(const cd_window_attn& p);
+cudaError_t launch_head_norm(const cd_window_attn& p, int fp32, cudaStream_t stream);
+cudaError_t launch_window_append(const cd_window_attn& p, int fp32, cudaStream_t stream);
+cudaError_t launch_window_rows(const cd_window_attn& p, int fp32, cudaStream_t stream);
+bool linear_attention_supported(int dkp, int dvp);
+cudaError_t launch_gla_step(const cd_linear_attn& p, int fp32, cudaStream_t stream);
+cudaError_t launch_gla_decay(const cd_linear_attn& p, int fp32, cudaStream_t stream);
+cudaError_t launch_gla_sequence(const cd_linear_attn& p, int fp32, cudaStream_t stream);
+cudaError_t launch_gla_finish(const cd_linear_attn& p, int fp32, cudaStream_t stream);
+
 // One operand pair of the GEMM: row-major bf16 matrices with K contiguous.
 struct GemmOperand {
   const void* a;   // [M, K], leading dimension lda
@@ -127,6 +149,8 @@ struct GemmEpilogueArgs {
   float bias_lo, bias_hi;
   int do_clamp;
   float clamp_lo, clamp_hi;
+  const void* col_scale;    // kEpiStoreF32: bf16 factor per output column
+  float glu_alpha, glu_limit, glu_offset;   // kEpiGlu (see GemmEpilogue)
   // failure-path self-test (see GemmParams)
   int selftest_stall;
   unsigned long long wait_limit_ns;

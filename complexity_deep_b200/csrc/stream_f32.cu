@@ -1,0 +1,195 @@
+// Kernels around a residual stream kept in fp32: embedding gather into the stream, RMSNorm of a
+// stream row into the operand type of the next product, and the 32-bit matrix product used when
+// a model runs entirely in fp32 (no reduced-precision mode anywhere on that path).
+#include "elem.cuh"
+#include "kernels.h"
+
+namespace cdeep {
+
+namespace {
+
+// x[t, :] = table[ids[t], :] in fp32; columns [W, ldx) are zero.  Ids outside the table are
+// clamped to it (as in the dispatch kernels), so a bad id can never read out of bounds.
+template <typename T>
+__global__ void __launch_bounds__(128)
+embed_rows_kernel(const long long* __restrict__ ids, const T* __restrict__ table, float* __restrict__ x,
+                  int V, int W, int ldw, int ldx) {
+  pdl_enter();
+  const int t = blockIdx.x;
+  long long id = ids[t];
+  id = id < 0 ? 0 : (id >= V ? V - 1 : id);
+  const T* src = table + id * ldw;
+  float* dst = x + static_cast<size_t>(t) * ldx;
+  for (int c = threadIdx.x; c < ldx; c += blockDim.x) dst[c] = c < W ? to_f32(src[c]) : 0.f;
+}
+
+// out[t, :] = x[t, :] / sqrt(mean(x^2) + eps) * (w + offset); the mean runs over W columns, rows
+// are ldx apart (a multiple of 8, zero beyond W).  One warp per row.  NV > 0: the row (at most
+// NV * 256 columns) stays in registers between the reduction and the scaling; NV = 0: it is read
+// twice.
+template <typename T, int NV>
+__global__ void __launch_bounds__(128)
+rmsnorm_f32_kernel(const float* __restrict__ x, const T* __restrict__ w, float eps, float offset,
+                   T* __restrict__ out, int rows, int W, int ldx) {
+  pdl_enter();
+  const int row = blockIdx.x * 4 + (threadIdx.x >> 5);
+  if (row >= rows) return;
+  const int lane = threadIdx.x & 31;
+  const float* xr = x + static_cast<size_t>(row) * ldx;
+  T* orow = out + static_cast<size_t>(row) * ldx;
+  constexpr int kBuf = NV ? NV : 1;
+  float buf[kBuf][8];
+  float ss = 0.f;
+  if constexpr (NV > 0) {
+#pragma unroll
+    for (int v = 0; v < NV; ++v) {
+      const int c = (v * 32 + lane) * 8;
+      if (c < ldx) load8(xr + c, buf[v]);
+    }
+#pragma unroll
+    for (int v = 0; v < NV; ++v)
+      if ((v * 32 + lane) * 8 < ldx) {
+#pragma unroll
+        for (int e = 0; e < 8; ++e) ss += buf[v][e] * buf[v][e];
+      }
+  } else {
+    for (int c = lane * 8; c < ldx; c += 256) {
+      load8(xr + c, buf[0]);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) ss += buf[0][e] * buf[0][e];
+    }
+  }
+  const float r = 1.0f / sqrtf(warp_add(ss) / static_cast<float>(W) + eps);
+  auto finish = [&](int c, float (&f)[8]) {
+    float wv[8];
+    load8(w + c, wv);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) f[e] = f[e] * r * (wv[e] + offset);
+    store8(orow + c, f);
+  };
+  if constexpr (NV > 0) {
+#pragma unroll
+    for (int v = 0; v < NV; ++v) {
+      const int c = (v * 32 + lane) * 8;
+      if (c < ldx) finish(c, buf[v]);
+    }
+  } else {
+    for (int c = lane * 8; c < ldx; c += 256) {
+      load8(xr + c, buf[0]);
+      finish(c, buf[0]);
+    }
+  }
+}
+
+// out[m, n] = residual[m, n] + col_scale[n] * sum_k a[m, k] b[n, k], all fp32 (FMA pipe).
+// Tile 64 x 64, 256 threads, 4 x 4 outputs per thread.  The order of the additions over k does not
+// depend on the number of rows.
+constexpr int kTM = 64, kTN = 64, kTK = 16;
+__global__ void __launch_bounds__(256)
+linear_f32_kernel(const float* __restrict__ a, const float* __restrict__ b, const float* residual,
+                  const float* __restrict__ col_scale, float* out, int M, int K, int N) {
+  __shared__ float sa[kTK][kTM + 4], sb[kTK][kTN + 4];
+  pdl_enter();
+  const int m0 = blockIdx.y * kTM, n0 = blockIdx.x * kTN;
+  const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
+  const int lr = threadIdx.x >> 2, lk = (threadIdx.x & 3) * 4;   // this thread's row and k of a tile load
+  float acc[4][4] = {};
+  for (int k0 = 0; k0 < K; k0 += kTK) {
+    float4 va = make_float4(0.f, 0.f, 0.f, 0.f), vb = va;
+    if (m0 + lr < M && k0 + lk < K) va = *reinterpret_cast<const float4*>(a + static_cast<size_t>(m0 + lr) * K + k0 + lk);
+    if (n0 + lr < N && k0 + lk < K) vb = *reinterpret_cast<const float4*>(b + static_cast<size_t>(n0 + lr) * K + k0 + lk);
+    sa[lk][lr] = va.x; sa[lk + 1][lr] = va.y; sa[lk + 2][lr] = va.z; sa[lk + 3][lr] = va.w;
+    sb[lk][lr] = vb.x; sb[lk + 1][lr] = vb.y; sb[lk + 2][lr] = vb.z; sb[lk + 3][lr] = vb.w;
+    __syncthreads();
+#pragma unroll
+    for (int k = 0; k < kTK; ++k) {
+      const float4 fa = *reinterpret_cast<const float4*>(&sa[k][ty * 4]);
+      const float4 fb = *reinterpret_cast<const float4*>(&sb[k][tx * 4]);
+      const float av[4] = {fa.x, fa.y, fa.z, fa.w}, bv[4] = {fb.x, fb.y, fb.z, fb.w};
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(av[i], bv[j], acc[i][j]);
+    }
+    __syncthreads();
+  }
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const int m = m0 + ty * 4 + i;
+    if (m >= M) continue;
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const int n = n0 + tx * 4 + j;
+      if (n >= N) continue;
+      float v = acc[i][j];
+      if (col_scale) v *= col_scale[n];
+      if (residual) v += residual[static_cast<size_t>(m) * N + n];
+      out[static_cast<size_t>(m) * N + n] = v;
+    }
+  }
+}
+
+// h[t, j] = g * sigmoid(alpha g) * (u + offset), g = min(gu[t, j], limit), u = clamp(gu[t, I + j], +-limit)
+__global__ void __launch_bounds__(256)
+glu_f32_kernel(const float* __restrict__ gu, float* __restrict__ h, long long n, int I, float alpha,
+               float limit, float offset) {
+  pdl_enter();
+  for (long long i = blockIdx.x * 256ll + threadIdx.x; i < n; i += gridDim.x * 256ll) {
+    const long long t = i / I;
+    const int j = static_cast<int>(i - t * I);
+    const float g = fminf(gu[t * 2 * I + j], limit);
+    const float u = fminf(fmaxf(gu[t * 2 * I + I + j], -limit), limit);
+    h[i] = g / (1.0f + expf(-alpha * g)) * (u + offset);
+  }
+}
+
+template <typename T>
+cudaError_t rmsnorm_any(const float* x, const void* w, float eps, float offset, void* out, int rows, int W,
+                        int ldx, cudaStream_t st) {
+  auto wp = static_cast<const T*>(w);
+  auto op = static_cast<T*>(out);
+  const dim3 grid((rows + 3) / 4), block(128);
+  const int nv = (ldx + 255) / 256;
+#define CDEEP_NORM(NV) return launch_kernel(rmsnorm_f32_kernel<T, NV>, grid, block, 0, st, x, wp, eps, offset, op, rows, W, ldx)
+  if (nv <= 2) CDEEP_NORM(2);
+  if (nv <= 4) CDEEP_NORM(4);
+  if (nv <= 8) CDEEP_NORM(8);
+  CDEEP_NORM(0);
+#undef CDEEP_NORM
+}
+
+}  // namespace
+
+cudaError_t launch_embed_rows(const long long* ids, const void* table, float* x, int T, int V, int W, int ldw,
+                              int ldx, int fp32, cudaStream_t st) {
+  if (T == 0) return cudaSuccess;
+  return fp32 ? launch_kernel(embed_rows_kernel<float>, dim3(T), dim3(128), 0, st, ids,
+                              static_cast<const float*>(table), x, V, W, ldw, ldx)
+              : launch_kernel(embed_rows_kernel<bf16>, dim3(T), dim3(128), 0, st, ids,
+                              static_cast<const bf16*>(table), x, V, W, ldw, ldx);
+}
+
+cudaError_t launch_rmsnorm_f32(const float* x, const void* w, float eps, float offset, void* out, int rows, int W,
+                               int ldx, int fp32, cudaStream_t st) {
+  if (rows == 0) return cudaSuccess;
+  return fp32 ? rmsnorm_any<float>(x, w, eps, offset, out, rows, W, ldx, st)
+              : rmsnorm_any<bf16>(x, w, eps, offset, out, rows, W, ldx, st);
+}
+
+cudaError_t launch_linear_f32(const float* a, const float* b, const float* residual, const float* col_scale,
+                              float* out, int M, int K, int N, cudaStream_t st) {
+  if (M == 0) return cudaSuccess;
+  return launch_kernel(linear_f32_kernel, dim3((N + kTN - 1) / kTN, (M + kTM - 1) / kTM), dim3(256), 0, st, a, b,
+                       residual, col_scale, out, M, K, N);
+}
+
+cudaError_t launch_glu_f32(const float* gu, float* h, int T, int I, float alpha, float limit, float offset,
+                           cudaStream_t st) {
+  const long long n = static_cast<long long>(T) * I;
+  if (n == 0) return cudaSuccess;
+  const long long blocks = (n + 255) / 256;
+  return launch_kernel(glu_f32_kernel, dim3(static_cast<unsigned>(blocks < 4096 ? blocks : 4096)), dim3(256), 0, st, gu,
+                       h, n, I, alpha, limit, offset);
+}
+
+}  // namespace cdeep

@@ -22,9 +22,11 @@ import torch.nn as nn
 import torch.nn.functional as F
 
 from .. import ops
+from ..core.attention import StaticKVCache
 from ..core.layer import MuClampRequest, SplitStream, TransformerBlock
 from ..core.normalization import RMSNorm
 from .config import ComplexityConfig
+from .generation import GenerationMixin
 
 KVCache = List[Tuple[torch.Tensor, torch.Tensor]]
 
@@ -43,7 +45,8 @@ class CausalLMOutput:
     past_key_values: Optional[KVCache] = None
 
 
-class ComplexityModel(nn.Module):
+class ComplexityModel(nn.Module, GenerationMixin):
+    config_class = ComplexityConfig
     # The residual stream travels between the fused kernels of consecutive blocks as a
     # split-bf16 pair (see core.layer.SplitStream); False keeps it as one bf16 tensor, as the
     # reference's bf16 path does (two fewer tensor reads / writes per block, ~2.5x the error
@@ -167,44 +170,12 @@ class ComplexityModel(nn.Module):
                 labels[..., 1:].reshape(-1), ignore_index=-100)
         return CausalLMOutput(loss=loss, logits=logits, past_key_values=new_kvs)
 
-    # ------------------------------------------------------------------ generation
-    @torch.no_grad()
-    def generate(
-        self,
-        input_ids: torch.Tensor,
-        max_new_tokens: int = 100,
-        temperature: float = 1.0,
-        top_k: int = 50,
-        top_p: float = 0.9,
-        do_sample: bool = True,
-        eos_token_id: Optional[int] = None,
-    ) -> torch.Tensor:
-        """Autoregressive sampling with a KV cache; same filtering rules as the reference
-        (temperature, then top-k, then nucleus top-p that always keeps the best token)."""
-        eos = self.config.eos_token_id if eos_token_id is None else eos_token_id
-        cache: Optional[KVCache] = None
-        for _ in range(max_new_tokens):
-            step_ids = input_ids if cache is None else input_ids[:, -1:]
-            out = self.forward(step_ids, past_key_values=cache, use_cache=True)
-            cache = out.past_key_values
-            scores = out.logits[:, -1, :].float() / temperature
-            if top_k > 0:
-                kth = torch.topk(scores, top_k).values[..., -1:]
-                scores = scores.masked_fill(scores < kth, float("-inf"))
-            if top_p < 1.0:
-                ordered, order = torch.sort(scores, descending=True)
-                mass = torch.cumsum(F.softmax(ordered, dim=-1), dim=-1)
-                drop = mass > top_p
-                drop = torch.cat([torch.zeros_like(drop[..., :1]), drop[..., :-1]], dim=-1)
-                scores = scores.masked_fill(drop.scatter(1, order, drop), float("-inf"))
-            if do_sample:
-                nxt = torch.multinomial(F.softmax(scores, dim=-1), num_samples=1)
-            else:
-                nxt = scores.argmax(dim=-1, keepdim=True)
-            input_ids = torch.cat([input_ids, nxt], dim=-1)
-            if bool((nxt == eos).all()):
-                break
-        return input_ids
+    # ------------------------------------------------------------------ decode cache
+    def make_decode_cache(self, batch: int, capacity: int) -> StaticKVCache:
+        """Fixed-capacity cache for captured decode steps (see ``DecodeGraph``)."""
+        c, w = self.config, self.embed_tokens.weight
+        return StaticKVCache(c.num_hidden_layers, batch, c.num_key_value_heads,
+                             c.hidden_size // c.num_attention_heads, capacity, w.device, dtype=w.dtype)
 
     # ------------------------------------------------------------------ utilities
     def num_parameters(self, trainable_only: bool = True) -> int:

@@ -39,7 +39,7 @@ class PrefillGraph:
         logits = graph(input_ids)        # the returned tensor is overwritten by the next call
     """
 
-    def __init__(self, model: ComplexityModel, batch: int, seq_len: int, warmup: int = 2):
+    def __init__(self, model, batch: int, seq_len: int, warmup: int = 2):
         import torch
         from ..core.token_routed_mlp import ROUTING_CACHE
         self.model = model
@@ -70,7 +70,8 @@ class PrefillGraph:
 
 
 class DecodeGraph:
-    """CUDA-graph replay of one decode step (one new token per sequence) on a StaticKVCache.
+    """CUDA-graph replay of one decode step (one new token per sequence) on the cache that the
+    model makes for it (``make_decode_cache``: a StaticKVCache, or a DecoderState).
 
     A decode step of the 1B model is ~270 launches of a few microseconds each, so the step
     time is set by how fast the host can issue them.  The cache position is a device scalar
@@ -83,18 +84,14 @@ class DecodeGraph:
         logits = dec.step(next_ids)          # [batch, 1, vocab], overwritten by the next step
     """
 
-    def __init__(self, model: ComplexityModel, batch: int, capacity: int, warmup: int = 2):
+    def __init__(self, model, batch: int, capacity: int, warmup: int = 2):
         import torch
-        from ..core.attention import StaticKVCache
         from ..core.token_routed_mlp import ROUTING_CACHE
         self.model = model
-        cfg = model.config
         device = next(model.parameters()).device
         if device.type != "cuda":
             raise RuntimeError("DecodeGraph needs the model on a CUDA device")
-        self.cache = StaticKVCache(cfg.num_hidden_layers, batch, cfg.num_key_value_heads,
-                                   cfg.hidden_size // cfg.num_attention_heads, capacity, device,
-                                   dtype=next(model.parameters()).dtype)
+        self.cache = model.make_decode_cache(batch, capacity)
         self.static_ids = torch.zeros(batch, 1, dtype=torch.int64, device=device)
         stream = torch.cuda.Stream(device=device)
         stream.wait_stream(torch.cuda.current_stream(device))
@@ -112,22 +109,23 @@ class DecodeGraph:
         self.cache.set_length(0)          # the warm-up and capture steps wrote scratch rows
 
     def _eager_step(self):
-        logits = self.model(self.static_ids, past_key_values=self.cache.layers,
+        logits = self.model(self.static_ids, past_key_values=self.cache.as_past(),
                             use_cache=True).logits
-        self.cache.state.add_(1)
+        self.cache.advance_device()
         return logits
 
     def prefill(self, input_ids, attention_mask=None):
-        """Runs the prompt through the model and moves its KV cache into the static buffers."""
+        """Runs the prompt through the model and moves its cache into the static buffers."""
         import torch
+        mask = {} if attention_mask is None else {"attention_mask": attention_mask}
         with torch.no_grad():
-            out = self.model(input_ids, attention_mask=attention_mask, use_cache=True)
+            out = self.model(input_ids, use_cache=True, **mask)
         self.cache.load(out.past_key_values)
         return out.logits
 
     def step(self, input_ids):
         if self.cache.length >= self.cache.capacity:
-            raise RuntimeError(f"KV cache full ({self.cache.capacity} tokens)")
+            raise RuntimeError(f"cache full ({self.cache.capacity} tokens)")
         self.static_ids.copy_(input_ids.view(self.static_ids.shape), non_blocking=True)
         self.graph.replay()
         self.cache.length += 1

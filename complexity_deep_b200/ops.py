@@ -745,3 +745,216 @@ def linear(x: torch.Tensor, w: torch.Tensor, residual: Optional[torch.Tensor] = 
         _lib.check(lib.cd_linear(x.data_ptr(), w.data_ptr(), _ptr(residual), _ptr(lo2),
                                  out.data_ptr(), _ptr(out_lo), T, K, N, _stream()), "cd_linear")
     return (out, out_lo) if want_lo else out
+
+
+# --------------------------------------------------------------------------- fp32 residual stream
+# Decoders that keep the residual stream in fp32.  Operands are bf16, or fp32 when a model runs
+# entirely in 32 bits; which one follows from the operand's dtype.
+def _storage(t: torch.Tensor, name: str) -> int:
+    """Checks an operand of either storage type; returns the C ABI's `fp32` flag."""
+    if t.dtype not in (BF16, torch.float32):
+        raise RuntimeError(f"{name}: expected dtype {BF16} or {torch.float32}, got {t.dtype}")
+    _need(t, name, t.dtype)
+    return 1 if t.dtype == torch.float32 else 0
+
+
+def embed_rows(ids: torch.Tensor, table: torch.Tensor, width: int, ldx: int) -> torch.Tensor:
+    """fp32 stream rows [T, ldx] = table[ids] (columns past `width` are zero)."""
+    lib = _lib.load()
+    ids = ids.reshape(-1)
+    _need(ids, "token_ids", torch.int64)
+    fp32 = _storage(table, "embedding table")
+    T = ids.numel()
+    x = torch.empty(T, ldx, dtype=torch.float32, device=ids.device)
+    with _Span("embed_rows"):
+        _lib.check(lib.cd_embed_rows(ids.data_ptr(), table.data_ptr(), x.data_ptr(), T, table.shape[0],
+                                     width, table.shape[1], ldx, fp32, _stream()), "cd_embed_rows")
+    return x
+
+
+def rmsnorm_f32(x: torch.Tensor, weight: torch.Tensor, eps: float, offset: float = 0.0,
+                width: Optional[int] = None) -> torch.Tensor:
+    """x / sqrt(mean(x^2) + eps) * (weight + offset) of an fp32 stream [T, ldx] into weight's dtype;
+    the mean runs over the first `width` columns (the rest of x and weight must be zero there)."""
+    lib = _lib.load()
+    _need(x, "x", torch.float32)
+    fp32 = _storage(weight, "weight")
+    T, ldx = x.shape
+    if weight.numel() != ldx:
+        raise RuntimeError("norm weight does not match the stream")
+    out = torch.empty(T, ldx, dtype=weight.dtype, device=x.device)
+    with _Span("rmsnorm_f32"):
+        _lib.check(lib.cd_rmsnorm_f32(x.data_ptr(), weight.data_ptr(), float(eps), float(offset),
+                                      out.data_ptr(), T, width or ldx, ldx, fp32, _stream()),
+                   "cd_rmsnorm_f32")
+    return out
+
+
+def linear_to_f32(x: torch.Tensor, w: torch.Tensor, residual: Optional[torch.Tensor] = None,
+                  col_scale: Optional[torch.Tensor] = None, inplace: bool = False,
+                  tag: str = "linear_f32") -> torch.Tensor:
+    """fp32 ``residual + col_scale * (x @ w^T)``; operands bf16 (tcgen05) or fp32 (FMA pipe).
+    inplace: the residual buffer itself receives the result."""
+    lib = _lib.load()
+    fp32 = _storage(x, "x")
+    _need(w, "weight", x.dtype)
+    T, K = x.shape
+    N = w.shape[0]
+    if w.shape[1] != K:
+        raise RuntimeError("weight does not match x")
+    if residual is not None:
+        _need(residual, "residual", torch.float32)
+        if tuple(residual.shape) != (T, N):
+            raise RuntimeError("residual does not match the output")
+    if col_scale is not None:
+        _need(col_scale, "col_scale", x.dtype)
+        if col_scale.numel() != N:
+            raise RuntimeError("col_scale does not match the output")
+    if not fp32:
+        _split_k_auto(x)
+    out = residual if inplace and residual is not None else torch.empty(T, N, dtype=torch.float32,
+                                                                        device=x.device)
+    fn = lib.cd_linear_f32 if fp32 else lib.cd_linear_f32out
+    with _Span(tag):
+        _lib.check(fn(x.data_ptr(), w.data_ptr(), _ptr(residual), _ptr(col_scale), out.data_ptr(), T,
+                      K, N, _stream()), "cd_linear_f32" if fp32 else "cd_linear_f32out")
+    return out
+
+
+def project(x: torch.Tensor, w: torch.Tensor, tag: str = "linear") -> torch.Tensor:
+    """``x @ w^T`` in x's dtype."""
+    return linear_to_f32(x, w, tag=tag) if x.dtype == torch.float32 else linear(x, w, tag=tag)
+
+
+def glu_up(x: torch.Tensor, packed_w: torch.Tensor, width: int, block_n: int, alpha: float,
+           limit: float, offset: float) -> torch.Tensor:
+    """Clamped gated unit on packed gate / up weights (pack_gate_up with one group)."""
+    lib = _lib.load()
+    _need(x, "x")
+    _need(packed_w, "packed gate/up weights")
+    T, H = x.shape
+    if tuple(packed_w.shape) != (1, lib.cd_gate_up_packed_rows(width, block_n), H):
+        raise RuntimeError("packed weights do not match the width / tile width")
+    h = torch.empty(T, width, dtype=BF16, device=x.device)
+    with _Span("glu_up"):
+        _lib.check(lib.cd_glu_up(x.data_ptr(), packed_w.data_ptr(), h.data_ptr(), T, H, width, block_n,
+                                 float(alpha), float(limit), float(offset), _stream()), "cd_glu_up")
+    return h
+
+
+def glu_f32(gate_up: torch.Tensor, alpha: float, limit: float, offset: float) -> torch.Tensor:
+    """The clamped gated unit of fp32 pre-activations [T, 2 I] (gate columns, then up)."""
+    lib = _lib.load()
+    _need(gate_up, "gate_up", torch.float32)
+    T, I = gate_up.shape[0], gate_up.shape[1] // 2
+    h = torch.empty(T, I, dtype=torch.float32, device=gate_up.device)
+    with _Span("glu_f32"):
+        _lib.check(lib.cd_glu_f32(gate_up.data_ptr(), h.data_ptr(), T, I, float(alpha), float(limit),
+                                  float(offset), _stream()), "cd_glu_f32")
+    return h
+
+
+# --------------------------------------------------------------------------- mixers
+def _columns(t: torch.Tensor, name: str, dtype) -> int:
+    """Address of a column slice of a row-major buffer."""
+    if not t.is_cuda or t.dtype != dtype or t.dim() != 2 or t.stride(1) != 1:
+        raise RuntimeError(f"{name}: expected columns of a CUDA {dtype} buffer")
+    return t.data_ptr()
+
+
+def window_attention_(proj: dict, out: torch.Tensor, weights: dict, ring_k: torch.Tensor,
+                      ring_v: torch.Tensor, *, batch: int, seq_len: int, heads: int, kv_heads: int,
+                      dim: int, vdim: int, window: int, keep: int, scale: float, eps: float,
+                      out_scale: float, pos0: int, pos_dev: Optional[torch.Tensor] = None) -> None:
+    """Attention of `seq_len` new tokens per sequence over a sliding window with kept first tokens
+    (cd_window_attn).  proj: 'q', 'k', 'v' column slices of the projection buffer (normed in place
+    when seq_len > 1); weights: 'q_norm', 'k_norm', 'r1', 'r2', 'talk'; the rings receive the new
+    keys and values; `out` = columns of the mixers' output buffer."""
+    lib = _lib.load()
+    dt = out.dtype
+    fp32 = 1 if dt == torch.float32 else 0
+    q, k, v = proj["q"], proj["k"], proj["v"]
+    dp, vp = ring_k.shape[3], ring_v.shape[3]
+    if (q.shape != (batch * seq_len, heads * dp) or k.shape != (batch * seq_len, kv_heads * dp)
+            or v.shape != (batch * seq_len, kv_heads * vp) or out.shape != (batch * seq_len, heads * vp)):
+        raise RuntimeError("window attention: projection columns do not match the head layout")
+    if q.stride(0) != k.stride(0) or q.stride(0) != v.stride(0):
+        raise RuntimeError("window attention: q, k and v must share their row stride")
+    _need(ring_k, "key ring", dt)
+    _need(ring_v, "value ring", dt)
+    for ring in (ring_k, ring_v):
+        if tuple(ring.shape[:3]) != (batch, keep + window, kv_heads):
+            raise RuntimeError("window attention: ring does not match batch / window / heads")
+    for name, n in (("q_norm", dp), ("k_norm", dp), ("r1", heads), ("r2", heads), ("talk", heads * heads)):
+        _need(weights[name], name, dt)
+        if weights[name].numel() != n:
+            raise RuntimeError(f"window attention: {name} has the wrong size")
+    if pos_dev is not None and (pos_dev.dtype != torch.int32 or not pos_dev.is_cuda or pos_dev.numel() != 1):
+        raise RuntimeError("pos_dev: expected one int32 on the device")
+    a = _lib.WindowAttn(
+        q=_columns(q, "q", dt), k=_columns(k, "k", dt), v=_columns(v, "v", dt), ldp=q.stride(0),
+        q_w=weights["q_norm"].data_ptr(), k_w=weights["k_norm"].data_ptr(), r1=weights["r1"].data_ptr(),
+        r2=weights["r2"].data_ptr(), talk=weights["talk"].data_ptr(), ring_k=ring_k.data_ptr(),
+        ring_v=ring_v.data_ptr(), out=_columns(out, "out", dt), ldo=out.stride(0), pos_dev=_ptr(pos_dev),
+        scale=float(scale), eps=float(eps), out_scale=float(out_scale), B=batch, S=seq_len, H=heads,
+        G=kv_heads, dim=dim, dp=dp, vdim=vdim, vp=vp, window=window, keep=keep, pos0=pos0, normed=0)
+    ref = ctypes.byref(a)
+    if seq_len == 1:
+        with _Span("window_attention_decode"):
+            _lib.check(lib.cd_window_attention_rows(ref, fp32, _stream()), "cd_window_attention_rows")
+        return
+    with _Span("head_norm"):
+        _lib.check(lib.cd_window_attention_norm(ref, fp32, _stream()), "cd_window_attention_norm")
+    a.normed = 1
+    with _Span("window_attention_rows"):
+        _lib.check(lib.cd_window_attention_rows(ref, fp32, _stream()), "cd_window_attention_rows")
+    with _Span("window_append"):
+        _lib.check(lib.cd_window_attention_append(ref, fp32, _stream()), "cd_window_attention_append")
+
+
+def linear_attention_(proj: dict, out: torch.Tensor, weights: dict, state: torch.Tensor, *, batch: int,
+                      seq_len: int, heads: int, dim: int, vdim: int, tau: float, eps: float,
+                      out_scale: float) -> None:
+    """Gated linear attention of `seq_len` new tokens per sequence (cd_linear_attn).  proj: 'q', 'k',
+    'v', 'gate', 'inner' column slices; weights: 'a2', 'a2_b', 'norm'; `state` [B, heads, dkp, dvp]
+    fp32 is carried on in place."""
+    lib = _lib.load()
+    dt = out.dtype
+    fp32 = 1 if dt == torch.float32 else 0
+    _need(state, "state", torch.float32)
+    dkp, dvp = state.shape[2], state.shape[3]
+    T = batch * seq_len
+    want = {"q": heads * dkp, "k": heads * dkp, "v": heads * dvp, "gate": heads * dvp,
+            "inner": proj["inner"].shape[1]}
+    ldp = proj["q"].stride(0)
+    for name, n in want.items():
+        if tuple(proj[name].shape) != (T, n) or proj[name].stride(0) != ldp:
+            raise RuntimeError(f"linear attention: {name} columns do not match the head layout")
+    if tuple(out.shape) != (T, heads * dvp) or tuple(state.shape[:2]) != (batch, heads):
+        raise RuntimeError("linear attention: output or state does not match the head layout")
+    for name, n in (("a2", heads * dkp * want["inner"]), ("a2_b", heads * dkp), ("norm", dvp)):
+        _need(weights[name], name, dt)
+        if weights[name].numel() != n:
+            raise RuntimeError(f"linear attention: {name} has the wrong size")
+    a = _lib.LinearAttn(
+        q=_columns(proj["q"], "q", dt), k=_columns(proj["k"], "k", dt), v=_columns(proj["v"], "v", dt),
+        gate=_columns(proj["gate"], "gate", dt), inner=_columns(proj["inner"], "inner", dt), ldp=ldp,
+        a2=weights["a2"].data_ptr(), a2_b=weights["a2_b"].data_ptr(), norm_w=weights["norm"].data_ptr(),
+        state=state.data_ptr(), out=_columns(out, "out", dt), ldo=out.stride(0), inv_tau=1.0 / tau,
+        eps=float(eps), out_scale=float(out_scale), q_scale=float(dim) ** -0.5, B=batch, S=seq_len,
+        H=heads, dk=dim, dkp=dkp, dv=vdim, dvp=dvp, rank=want["inner"])
+    ref = ctypes.byref(a)
+    if seq_len == 1:
+        with _Span("gla_step"):
+            _lib.check(lib.cd_gla_step(ref, fp32, _stream()), "cd_gla_step")
+        return
+    log_decay = torch.empty(T, heads * dkp, dtype=torch.float32, device=out.device)
+    a.log_decay = log_decay.data_ptr()
+    with _Span("gla_decay"):
+        _lib.check(lib.cd_gla_decay(ref, fp32, _stream()), "cd_gla_decay")
+    o_raw = torch.empty(T, heads * dvp, dtype=torch.float32, device=out.device)
+    a.o_raw = o_raw.data_ptr()
+    with _Span("gla_sequence"):
+        _lib.check(lib.cd_gla_sequence(ref, fp32, _stream()), "cd_gla_sequence")
+    with _Span("gla_finish"):
+        _lib.check(lib.cd_gla_finish(ref, fp32, _stream()), "cd_gla_finish")

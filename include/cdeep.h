@@ -374,6 +374,102 @@ int cd_mu_proj(const void* h, const void* w, const void* mu_param, float mu_min,
 int cd_linear(const void* x, const void* w, const void* residual, const void* residual_lo,
               void* out, void* out_lo, int T, int K, int N, void* stream);
 
+/* ------------------------------------------------------------------ fp32 residual stream ----
+ * Pieces of decoders that keep the residual stream in fp32.  `fp32` = 0: operands (weights and
+ * activations outside the stream) are bf16; 1: they are fp32 and nothing on the path uses fewer
+ * bits.  Rows of the stream are ldx elements apart (a multiple of 8, zero beyond the width). */
+
+/* x[t, :W] = table[ids[t], :W] (rows ldw apart), columns [W, ldx) = 0; ids are clamped to [0, V). */
+int cd_embed_rows(const int64_t* ids, const void* table, float* x, int T, int V, int W, int ldw,
+                  int ldx, int fp32, void* stream);
+/* out = x / sqrt(mean_W(x^2) + eps) * (w + offset); x, out [T, ldx], w [ldx]. */
+int cd_rmsnorm_f32(const float* x, const void* w, float eps, float offset, void* out, int T, int W,
+                   int ldx, int fp32, void* stream);
+/* bf16 operands, fp32 result: out = residual + col_scale * (x @ w^T); x [T, K], w [N, K],
+ * col_scale bf16 [N] or NULL, residual fp32 [T, N] or NULL (may be `out`). */
+int cd_linear_f32out(const void* x, const void* w, const float* residual, const void* col_scale,
+                     float* out, int T, int K, int N, void* stream);
+/* The same with fp32 operands (K a multiple of 4). */
+int cd_linear_f32(const float* x, const float* w, const float* residual, const float* col_scale,
+                  float* out, int T, int K, int N, void* stream);
+/* Clamped gated unit on packed gate/up weights (cd_pack_gate_up, one group):
+ * h = g sigmoid(alpha g) (u + offset), g = min(x Wg^T, limit), u = clamp(x Wu^T, -limit, limit). */
+int cd_glu_up(const void* x, const void* packed_w, void* h, int T, int H, int I, int block_n,
+              float alpha, float limit, float offset, void* stream);
+/* The same function of fp32 pre-activations gu [T, 2 I] (gate columns, then up). */
+int cd_glu_f32(const float* gu, float* h, int T, int I, float alpha, float limit, float offset,
+               void* stream);
+
+/* ------------------------------------------------------------------ window attention ---------
+ * Sliding window with kept first tokens, per-head distance bias, mixing of the heads' weights:
+ *   s_h(i, j) = scale q_h(i) . k_c(j) - r1_h ln(1 + r2_h (i - j)),   c = h / (H / G)
+ *   w_h(i, .) = softmax over { j <= i : i - j < window or j < keep }
+ *   out_h(i)  = out_scale sum_j (sum_g talk[h, g] w_g(i, j)) v_c(j)
+ * Keys and values of earlier calls live in a ring of keep + window slots per sequence: position
+ * j < keep in slot j, any other in slot keep + (j - keep) % window. */
+typedef struct cd_window_attn {
+  void* q;              /* projection rows of the call: row b * S + t, ldp elements apart; heads dp */
+  void* k;              /* (q, k) and vp (v) elements wide, multiples of 16, of which dim / vdim are */
+  const void* v;        /* in use and the rest zero; q, k, v 16-byte aligned, ldp a multiple of 8 */
+  long long ldp;
+  const void* q_w;      /* [dp] weights of the query / key head norm */
+  const void* k_w;
+  const void* r1;       /* [H] */
+  const void* r2;
+  const void* talk;     /* [H, H] */
+  void* ring_k;         /* [B, keep + window, G, dp] */
+  void* ring_v;         /* [B, keep + window, G, vp] */
+  void* out;            /* rows of H * vp elements, ldo apart */
+  long long ldo;
+  const int32_t* pos_dev;   /* position of the call's first token, read on the device ... */
+  float scale, eps, out_scale;
+  int B, S, H, G, dim, dp, vdim, vp, window, keep;
+  int pos0;             /* ... or given here when pos_dev is NULL */
+  int normed;           /* q and k rows are normed already */
+} cd_window_attn;
+
+/* 1 when the sizes are within what the kernels take. */
+int cd_window_attention_supported(const cd_window_attn* h_args);
+/* Norms the q and k heads of every row in place. */
+int cd_window_attention_norm(const cd_window_attn* h_args, int fp32, void* stream);
+/* One query per thread-block cluster.  normed = 1: any S, keys of the call from k / v, earlier ones
+ * from the ring.  normed = 0 (S must be 1): q and the new key are normed by the kernel, which also
+ * writes the new key and value into the ring. */
+int cd_window_attention_rows(const cd_window_attn* h_args, int fp32, void* stream);
+/* Writes the call's normed keys and values into the ring (after the attention of the call). */
+int cd_window_attention_append(const cd_window_attn* h_args, int fp32, void* stream);
+
+/* ------------------------------------------------------------------ gated linear attention ---
+ *   log a_t = -softplus(-(a2 u_t + a2_b)) inv_tau,  S_t = diag(a_t) S_{t-1} + k_t v_t^T,
+ *   o_t = q_scale S_t^T q_t,   out_t = out_scale (o_t / rms(o_t) * norm_w) silu(gate_t)   per head */
+typedef struct cd_linear_attn {
+  const void* q;        /* projection rows: row b * S + t, ldp elements apart; heads dkp (q, k) and */
+  const void* k;        /* dvp (v, gate) wide, multiples of 16, dk / dv of which are in use and the */
+  const void* v;        /* rest zero */
+  const void* gate;
+  const void* inner;    /* u, rank wide (rank a multiple of 8) */
+  long long ldp;
+  const void* a2;       /* [H * dkp, rank] */
+  const void* a2_b;     /* [H * dkp] */
+  const void* norm_w;   /* [dvp] */
+  float* state;         /* [B, H, dkp, dvp] fp32, read and replaced */
+  void* out;            /* rows of H * dvp elements, ldo apart */
+  long long ldo;
+  float* log_decay;     /* scratch [B * S, H * dkp] (not for cd_gla_step) */
+  float* o_raw;         /* scratch [B * S, H * dvp] (cd_gla_sequence, cd_gla_finish) */
+  float inv_tau, eps, out_scale, q_scale;
+  int B, S, H, dk, dkp, dv, dvp, rank;
+} cd_linear_attn;
+
+int cd_gla_supported(const cd_linear_attn* h_args);
+/* One token per sequence (S = 1): decay, state update, head norm and gate in one kernel. */
+int cd_gla_step(const cd_linear_attn* h_args, int fp32, void* stream);
+/* Several tokens: cd_gla_decay fills log_decay, cd_gla_sequence walks the tokens (o_raw, state),
+ * cd_gla_finish applies head norm and gate. */
+int cd_gla_decay(const cd_linear_attn* h_args, int fp32, void* stream);
+int cd_gla_sequence(const cd_linear_attn* h_args, int fp32, void* stream);
+int cd_gla_finish(const cd_linear_attn* h_args, int fp32, void* stream);
+
 #ifdef __cplusplus
 }
 #endif
