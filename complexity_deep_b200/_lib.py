@@ -116,6 +116,8 @@ SIGNATURES = {
     "cd_window_attention_supported": (c_int, [ctypes.POINTER(WindowAttn)]),
     "cd_window_attention_norm": _WINDOW_FN,
     "cd_window_attention_rows": _WINDOW_FN,
+    "cd_window_attention_prefill_supported": (c_int, [ctypes.POINTER(WindowAttn)]),
+    "cd_window_attention_prefill": (c_int, [ctypes.POINTER(WindowAttn), c_void_p]),
     "cd_window_attention_append": _WINDOW_FN,
     "cd_gla_supported": (c_int, [ctypes.POINTER(LinearAttn)]),
     "cd_gla_step": _GLA_FN,

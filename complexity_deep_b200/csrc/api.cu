@@ -659,6 +659,18 @@ int cd_window_attention_rows(const cd_window_attn* a, int fp32, void* stream) {
   return e == cudaSuccess ? CD_OK : cuda_fail(e, "window attention launch");
 }
 
+int cd_window_attention_prefill_supported(const cd_window_attn* a) {
+  return window_args_ok(a) == CD_OK && window_prefill_supported(*a) ? 1 : 0;
+}
+
+int cd_window_attention_prefill(const cd_window_attn* a, void* stream) {
+  if (window_args_ok(a) != CD_OK || !a->r1 || !a->r2 || !a->talk || !a->ring_k || !a->ring_v || !a->out || !a->normed)
+    return CD_ERR_INVALID;
+  if (!window_prefill_supported(*a)) return CD_ERR_UNSUPPORTED;
+  cudaError_t e = launch_window_prefill(*a, as_stream(stream));
+  return e == cudaSuccess ? CD_OK : cuda_fail(e, "window attention prefill launch");
+}
+
 int cd_window_attention_append(const cd_window_attn* a, int fp32, void* stream) {
   if (window_args_ok(a) != CD_OK || !a->ring_k || !a->ring_v) return CD_ERR_INVALID;
   cudaError_t e = launch_window_append(*a, fp32, as_stream(stream));

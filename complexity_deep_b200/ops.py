@@ -906,8 +906,12 @@ def window_attention_(proj: dict, out: torch.Tensor, weights: dict, ring_k: torc
     with _Span("head_norm"):
         _lib.check(lib.cd_window_attention_norm(ref, fp32, _stream()), "cd_window_attention_norm")
     a.normed = 1
-    with _Span("window_attention_rows"):
-        _lib.check(lib.cd_window_attention_rows(ref, fp32, _stream()), "cd_window_attention_rows")
+    if not fp32 and lib.cd_window_attention_prefill_supported(ref):
+        with _Span("window_attention_prefill"):
+            _lib.check(lib.cd_window_attention_prefill(ref, _stream()), "cd_window_attention_prefill")
+    else:
+        with _Span("window_attention_rows"):
+            _lib.check(lib.cd_window_attention_rows(ref, fp32, _stream()), "cd_window_attention_rows")
     with _Span("window_append"):
         _lib.check(lib.cd_window_attention_append(ref, fp32, _stream()), "cd_window_attention_append")
 

@@ -436,6 +436,10 @@ int cd_window_attention_norm(const cd_window_attn* h_args, int fp32, void* strea
  * from the ring.  normed = 0 (S must be 1): q and the new key are normed by the kernel, which also
  * writes the new key and value into the ring. */
 int cd_window_attention_rows(const cd_window_attn* h_args, int fp32, void* stream);
+/* Tensor-core form for prompts in bf16 (normed = 1): a tile of queries with all heads per block.
+ * Not every head layout fits (cd_window_attention_prefill_supported); the form above takes any. */
+int cd_window_attention_prefill_supported(const cd_window_attn* h_args);
+int cd_window_attention_prefill(const cd_window_attn* h_args, void* stream);
 /* Writes the call's normed keys and values into the ring (after the attention of the call). */
 int cd_window_attention_append(const cd_window_attn* h_args, int fp32, void* stream);
 
