@@ -124,6 +124,8 @@ SIGNATURES = {
     "cd_gla_decay": _GLA_FN,
     "cd_gla_sequence": _GLA_FN,
     "cd_gla_finish": _GLA_FN,
+    "cd_gla_chunk_workspace_bytes": (c_size_t, [ctypes.POINTER(LinearAttn)]),
+    "cd_gla_chunk": (c_int, [ctypes.POINTER(LinearAttn), c_void_p, c_size_t, c_void_p]),
 }
 
 _lib = None

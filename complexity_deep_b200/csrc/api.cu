@@ -724,4 +724,17 @@ int cd_gla_finish(const cd_linear_attn* a, int fp32, void* stream) {
   return e == cudaSuccess ? CD_OK : cuda_fail(e, "gla finish launch");
 }
 
+size_t cd_gla_chunk_workspace_bytes(const cd_linear_attn* a) {
+  return gla_args_ok(a) == CD_OK && gla_chunk_supported(*a) ? gla_chunk_workspace_bytes(*a) : 0;
+}
+
+int cd_gla_chunk(const cd_linear_attn* a, void* ws, size_t ws_bytes, void* stream) {
+  const int st = gla_args_ok(a);
+  if (st != CD_OK) return st;
+  if (!gla_chunk_supported(*a)) return CD_ERR_UNSUPPORTED;
+  if (!a->log_decay || !ws || !aligned16(ws) || ws_bytes < gla_chunk_workspace_bytes(*a)) return CD_ERR_INVALID;
+  cudaError_t e = launch_gla_chunk(*a, ws, as_stream(stream));
+  return e == cudaSuccess ? CD_OK : cuda_fail(e, "gla chunk launch");
+}
+
 }  // extern "C"

@@ -122,6 +122,10 @@ cudaError_t launch_gla_decay(const cd_linear_attn& p, int fp32, cudaStream_t str
 cudaError_t launch_gla_sequence(const cd_linear_attn& p, int fp32, cudaStream_t stream);
 cudaError_t launch_gla_finish(const cd_linear_attn& p, int fp32, cudaStream_t stream);
 
+bool gla_chunk_supported(const cd_linear_attn& a);
+size_t gla_chunk_workspace_bytes(const cd_linear_attn& a);
+cudaError_t launch_gla_chunk(const cd_linear_attn& a, void* ws, cudaStream_t stream);
+
 // One operand pair of the GEMM: row-major bf16 matrices with K contiguous.
 struct GemmOperand {
   const void* a;   // [M, K], leading dimension lda

@@ -916,6 +916,9 @@ def window_attention_(proj: dict, out: torch.Tensor, weights: dict, ring_k: torc
         _lib.check(lib.cd_window_attention_append(ref, fp32, _stream()), "cd_window_attention_append")
 
 
+_GLA_CHUNK_MIN = 16     # shorter portions walk token by token
+
+
 def linear_attention_(proj: dict, out: torch.Tensor, weights: dict, state: torch.Tensor, *, batch: int,
                       seq_len: int, heads: int, dim: int, vdim: int, tau: float, eps: float,
                       out_scale: float) -> None:
@@ -956,6 +959,12 @@ def linear_attention_(proj: dict, out: torch.Tensor, weights: dict, state: torch
     a.log_decay = log_decay.data_ptr()
     with _Span("gla_decay"):
         _lib.check(lib.cd_gla_decay(ref, fp32, _stream()), "cd_gla_decay")
+    ws_bytes = 0 if fp32 or seq_len < _GLA_CHUNK_MIN else lib.cd_gla_chunk_workspace_bytes(ref)
+    if ws_bytes:
+        ws = torch.empty(ws_bytes, dtype=torch.uint8, device=out.device)
+        with _Span("gla_chunk", 3):
+            _lib.check(lib.cd_gla_chunk(ref, ws.data_ptr(), ws_bytes, _stream()), "cd_gla_chunk")
+        return
     o_raw = torch.empty(T, heads * dvp, dtype=torch.float32, device=out.device)
     a.o_raw = o_raw.data_ptr()
     with _Span("gla_sequence"):

@@ -473,6 +473,10 @@ int cd_gla_step(const cd_linear_attn* h_args, int fp32, void* stream);
 int cd_gla_decay(const cd_linear_attn* h_args, int fp32, void* stream);
 int cd_gla_sequence(const cd_linear_attn* h_args, int fp32, void* stream);
 int cd_gla_finish(const cd_linear_attn* h_args, int fp32, void* stream);
+/* Several tokens in bf16, chunks of 64 on the tensor cores (after cd_gla_decay; writes `out` and the
+ * state).  The workspace size is 0 where the form does not apply (heads wider than 256). */
+size_t cd_gla_chunk_workspace_bytes(const cd_linear_attn* h_args);
+int cd_gla_chunk(const cd_linear_attn* h_args, void* workspace, size_t bytes, void* stream);
 
 #ifdef __cplusplus
 }
