@@ -961,6 +961,166 @@ def run_decode(args):
         dist.destroy_process_group()
 
 
+# ---------------------------------------------------------------- Pimezen beside a dense Complexity model
+PIMEZEN_SIZES = {
+    # width, layers, left heads / kv heads (128 wide), window, kept tokens, right heads (128 x 128), ff
+    "w1024": dict(width=1024, layers=8, heads=8, kv=4, window=512, keep=4, r_heads=4, ff=2816),
+    "w2048": dict(width=2048, layers=8, heads=16, kv=8, window=1024, keep=4, r_heads=8, ff=5632),
+}
+PIMEZEN_VOCAB, PIMEZEN_PREFILL, PIMEZEN_DECODE = 32000, (8, 2048), (32, 256)
+
+
+def pimezen_model(z: dict, device):
+    """Random weights of a Pimezen model of the size `z`."""
+    from complexity_deep_b200.models import PimezenConfig, PimezenModel
+    layer = {"type": "parallel",
+             "mixer": {"left": {"heads": z["heads"], "kv_heads": z["kv"], "dim": 128, "vdim": 128,
+                                "scale": 128 ** -0.5, "mask": {"size": z["window"], "keep_first": z["keep"]}},
+                       "right": {"heads": z["r_heads"], "dim": 128, "vdim": 128, "tau": 16.0},
+                       "left_scale": 0.7, "right_scale": 0.7},
+             "mlp": {"kind": "dense", "ff": z["ff"], "limit": 7.0}}
+    cfg = {"architecture": "Pimezen", "vocab": PIMEZEN_VOCAB, "width": z["width"], "norm": {"eps": 1e-6},
+           "layers": [layer] * z["layers"]}
+    torch.manual_seed(0)
+    with torch.device(device):
+        model = PimezenModel(PimezenConfig.from_dict(cfg))
+    for name, p in model.named_parameters():
+        if name.endswith((".r1", ".r2")):
+            torch.nn.init.uniform_(p, 0.1, 1.0)
+    return model.to(torch.bfloat16).requires_grad_(False).eval()
+
+
+def dense_complexity_model(z: dict, device):
+    """The closest model of the reference at the same width, heads and feed-forward: dense SwiGLU, no
+    mu guidance, attention over the whole sequence."""
+    import complexity_deep_b200 as cd
+    cfg = cd.ComplexityConfig(vocab_size=PIMEZEN_VOCAB, hidden_size=z["width"], intermediate_size=z["ff"],
+                              num_hidden_layers=z["layers"], num_attention_heads=z["heads"],
+                              num_key_value_heads=z["kv"], max_position_embeddings=8192,
+                              use_token_routed_mlp=False, use_mu_guidance=False)
+    torch.manual_seed(0)
+    with torch.device(device):
+        model = cd.ComplexityModel(cfg)
+    return model.to(torch.bfloat16).requires_grad_(False).eval()
+
+
+def pimezen_work(z: dict, T: int, S: int) -> dict:
+    """name -> (FLOP, bytes) of one launch at T tokens (S per sequence; S = 1: a decode step past the window)."""
+    W, H, G, R, ff, V = z["width"], z["heads"], z["kv"], z["r_heads"], z["ff"], PIMEZEN_VOCAB
+    n_in = (H + 2 * G + 4 * R) * 128 + 16
+    n_out = (H + R) * 128
+    win = z["window"] + z["keep"]
+    keys = win if S == 1 else sum(min(i + 1, win) for i in range(S)) / S    # visible keys per query
+    gemm = lambda k, n, out: (2 * T * k * n, 2 * (T * k + k * n) + out * T * n)
+    qkv = (H + 2 * G) * 128
+    return {
+        "mixer_in": gemm(W, n_in, 2), "mixer_out": gemm(n_out, W, 8),
+        "glu_up": (4 * T * W * ff, 2 * (T * W + 2 * W * ff + T * ff)), "glu_down": gemm(ff, W, 8),
+        "mu_qkv": gemm(W, qkv, 2), "linear_o_proj": gemm(H * 128, W, 6),
+        "moe_up_shared": (4 * T * W * ff, 2 * (T * W + 2 * W * ff + T * ff)), "moe_down": gemm(ff, W, 6),
+        "linear_lm_head": gemm(W, V, 4),
+        "rmsnorm_f32": (0, T * W * 6), "rmsnorm": (0, T * W * 6), "head_norm": (0, T * (H + G) * 128 * 4),
+        # scores, mixing of the heads, values
+        "window_attention_prefill": (2 * T * keys * H * (128 + H + 128), T * (2 * H + 2 * G) * 256),
+        "attention_prefill": (2 * T * (S + 1) / 2 * H * 256, T * (2 * H + 2 * G) * 256),
+        "window_attention_decode": (0, T * win * G * 512),
+        # q, k, v, gate, log decays in, result out (the state stays on chip in an ideal kernel)
+        "gla_chunk": (2 * T * R * 128 * 128 * 2, T * R * 128 * (5 * 2 + 4)),
+        "gla_decay": (0, T * R * 128 * 4), "gla_step": (0, T * R * 128 * 128 * 8),
+    }
+
+
+def pimezen_bench(z: dict, make, args, dev) -> dict:
+    """Prefill and decode throughput and the time of every kernel of one model."""
+    from complexity_deep_b200 import ops
+    from complexity_deep_b200.models import DecodeGraph, PrefillGraph
+    model, pk, out = make(z, dev), peaks(), {}
+    gen = torch.Generator(device=dev).manual_seed(1)
+
+    def timed(fn):
+        for _ in range(args.warmup):
+            fn()
+        torch.cuda.synchronize()
+        a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        a.record()
+        for _ in range(args.steps):
+            fn()
+        b.record()
+        torch.cuda.synchronize()
+        return a.elapsed_time(b) / args.steps
+
+    def kernels(fn, T, S, per_step_layers):
+        for _ in range(2):
+            fn()
+        ops.PROFILE.reset(enabled=True)
+        for _ in range(3):
+            fn()
+        prof = ops.PROFILE.collect()
+        ops.PROFILE.reset(enabled=False)
+        work, res = pimezen_work(z, T, S), {}
+        for name, (calls, ms, _) in prof.items():
+            us = ms / calls * 1e3
+            res[name] = {"us": round(us, 1), "calls_per_step": calls // 3}
+            if name in work:
+                flop, byts = work[name]
+                ideal = max(flop / pk["bf16_tflops"] / 1e6, byts / pk["hbm_gbs"] / 1e3)
+                res[name]["of_measured_roofline"] = round(ideal / us, 3)
+        return res
+
+    B, S = PIMEZEN_PREFILL
+    ids = torch.randint(0, PIMEZEN_VOCAB, (B, S), device=dev, generator=gen)
+    with torch.no_grad():
+        graph = PrefillGraph(model, B, S)
+        ms = timed(lambda: graph(ids))
+        out["prefill"] = {"batch": B, "seq_len": S, "ms": round(ms, 3), "tokens_per_s": round(B * S / ms * 1e3),
+                          "kernels": kernels(lambda: model(ids), B * S, S, z["layers"])}
+        del graph
+        torch.cuda.empty_cache()
+        for n in PIMEZEN_DECODE:
+            P = S
+            dec = DecodeGraph(model, batch=n, capacity=P + 2 * (args.steps + args.warmup) + 16)
+            dec.cache.length = P
+            if hasattr(dec.cache, "position"):
+                dec.cache.position.fill_(P)
+                tensors = [t for layer in dec.cache.layers for t in (layer["left"].k, layer["left"].v)]
+            else:
+                dec.cache.set_length(P)
+                tensors = dec.cache.k + dec.cache.v
+            for t in tensors:
+                t.normal_(0.0, 1.0, generator=gen)
+            nxt = torch.randint(0, PIMEZEN_VOCAB, (n, 1), device=dev, generator=gen)
+            ms = timed(lambda: dec.step(nxt))
+            out[f"decode_{n}"] = {"sequences": n, "cached": P, "ms": round(ms, 3), "tokens_per_s": round(n / ms * 1e3),
+                                  "kernels": kernels(dec._eager_step, n, 1, z["layers"])}
+            del dec
+            torch.cuda.empty_cache()
+    ops.status_fetch()
+    return out
+
+
+def run_pimezen(args):
+    """Prefill and decode of Pimezen models (random weights) beside the dense Complexity model of the
+    same width, heads and feed-forward; decode starts at 2 048 tokens."""
+    dev = torch.device("cuda", 0)
+    torch.cuda.set_device(dev)
+    sampler = ClockSampler(0)
+    sampler.start()
+    sizes = {}
+    for name, z in PIMEZEN_SIZES.items():
+        if args.pimezen_size not in ("all", name):
+            continue
+        sizes[name] = {"config": z, "pimezen": pimezen_bench(z, pimezen_model, args, dev),
+                       "dense_complexity": pimezen_bench(z, dense_complexity_model, args, dev)}
+        torch.cuda.empty_cache()
+    last = sizes[list(sizes)[-1]]["pimezen"]["prefill"]
+    print(json.dumps({"metric": "prefill tokens/s (Pimezen, bf16)", "value": last["tokens_per_s"], "unit": "tokens/s",
+                      "n_gpus": 1, "steps": args.steps, "warmup": args.warmup, "ms_per_step": last["ms"],
+                      "higher_is_better": True, "dtype": "bf16", "data": "synthetic", "impl": "b200",
+                      "config": {"workload": "pimezen", "vocab": PIMEZEN_VOCAB,
+                                 "inputs": "weights and activations of a step exceed L2"},
+                      "clocks": sampler.stop(), "sizes": sizes}), flush=True)
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -986,8 +1146,10 @@ def main():
     ap.add_argument("--cache-len", type=int, default=4096, help="decode_1b: prefilled KV tokens")
     ap.add_argument("--seq-len", type=int, default=SEQ_LEN, help="attn_prefill: sequence length")
     ap.add_argument("--workload", default="prefill_1b",
-                    choices=["prefill_1b", "decode_1b", "attn_prefill"] + list(LAYER_CONFIGS),
+                    choices=["prefill_1b", "decode_1b", "attn_prefill", "pimezen"] + list(LAYER_CONFIGS),
                     help="prefill_1b is the headline; the layer modes report MoE-layer TFLOP/s")
+    ap.add_argument("--pimezen-size", default="all", choices=["all"] + list(PIMEZEN_SIZES),
+                    help="pimezen: which size to run")
     args = ap.parse_args()
     if args.warmup < 3 and args.impl == "b200":
         args.warmup = 3
@@ -999,6 +1161,8 @@ def main():
         run_decode(args)
     elif args.workload == "attn_prefill":
         run_attention(args)
+    elif args.workload == "pimezen":
+        run_pimezen(args)
     elif args.workload != "prefill_1b":
         run_layer(args)
     else:

@@ -761,7 +761,7 @@ def _storage(t: torch.Tensor, name: str) -> int:
 def embed_rows(ids: torch.Tensor, table: torch.Tensor, width: int, ldx: int) -> torch.Tensor:
     """fp32 stream rows [T, ldx] = table[ids] (columns past `width` are zero)."""
     lib = _lib.load()
-    ids = ids.reshape(-1)
+    ids = ids.reshape(-1).contiguous()
     _need(ids, "token_ids", torch.int64)
     fp32 = _storage(table, "embedding table")
     T = ids.numel()
