@@ -116,6 +116,8 @@ SIGNATURES = {
     "cd_window_attention_supported": (c_int, [ctypes.POINTER(WindowAttn)]),
     "cd_window_attention_norm": _WINDOW_FN,
     "cd_window_attention_rows": _WINDOW_FN,
+    "cd_window_attention_decode_workspace_bytes": (c_size_t, [ctypes.POINTER(WindowAttn)]),
+    "cd_window_attention_decode": (c_int, [ctypes.POINTER(WindowAttn), c_void_p, c_size_t, c_int, c_void_p]),
     "cd_window_attention_prefill_supported": (c_int, [ctypes.POINTER(WindowAttn)]),
     "cd_window_attention_prefill": (c_int, [ctypes.POINTER(WindowAttn), c_void_p]),
     "cd_window_attention_append": _WINDOW_FN,

@@ -652,11 +652,25 @@ int cd_window_attention_norm(const cd_window_attn* a, int fp32, void* stream) {
 
 int cd_window_attention_rows(const cd_window_attn* a, int fp32, void* stream) {
   if (window_args_ok(a) != CD_OK || !a->r1 || !a->r2 || !a->talk || !a->ring_k || !a->ring_v || !a->out ||
-      (!a->normed && a->S != 1))
+      !a->normed)
     return CD_ERR_INVALID;
   if (!window_rows_supported(*a)) return CD_ERR_UNSUPPORTED;
   cudaError_t e = launch_window_rows(*a, fp32, as_stream(stream));
   return e == cudaSuccess ? CD_OK : cuda_fail(e, "window attention launch");
+}
+
+size_t cd_window_attention_decode_workspace_bytes(const cd_window_attn* a) {
+  return window_args_ok(a) == CD_OK && window_decode_supported(*a) ? window_decode_workspace_bytes(*a) : 0;
+}
+
+int cd_window_attention_decode(const cd_window_attn* a, void* ws, size_t ws_bytes, int fp32, void* stream) {
+  if (window_args_ok(a) != CD_OK || !a->r1 || !a->r2 || !a->talk || !a->ring_k || !a->ring_v || !a->out ||
+      a->normed || a->S != 1)
+    return CD_ERR_INVALID;
+  if (!window_decode_supported(*a)) return CD_ERR_UNSUPPORTED;
+  if (!ws || !aligned16(ws) || ws_bytes < window_decode_workspace_bytes(*a)) return CD_ERR_INVALID;
+  cudaError_t e = launch_window_decode(*a, ws, fp32, as_stream(stream));
+  return e == cudaSuccess ? CD_OK : cuda_fail(e, "window attention decode launch");
 }
 
 int cd_window_attention_prefill_supported(const cd_window_attn* a) {

@@ -114,6 +114,9 @@ bool window_rows_supported(const cd_window_attn& p);
 cudaError_t launch_head_norm(const cd_window_attn& p, int fp32, cudaStream_t stream);
 cudaError_t launch_window_append(const cd_window_attn& p, int fp32, cudaStream_t stream);
 cudaError_t launch_window_rows(const cd_window_attn& p, int fp32, cudaStream_t stream);
+bool window_decode_supported(const cd_window_attn& p);
+size_t window_decode_workspace_bytes(const cd_window_attn& p);
+cudaError_t launch_window_decode(const cd_window_attn& p, void* ws, int fp32, cudaStream_t stream);
 bool window_prefill_supported(const cd_window_attn& p);
 cudaError_t launch_window_prefill(const cd_window_attn& p, cudaStream_t stream);
 bool linear_attention_supported(int dkp, int dvp);

@@ -86,15 +86,68 @@ gla_step_kernel(const LinearAttnParams p) {
 }
 
 // ---------------------------------------------------------------- several tokens
-template <typename T>
+constexpr int kDecayRows = 32;
+
+// A thread keeps its channel's row of a2 in registers (rank <= 8 R8) and takes kDecayRows tokens.
+template <typename T, int R8>
 __global__ void __launch_bounds__(kThreads)
 gla_decay_kernel(const LinearAttnParams p) {
+  extern __shared__ float su[];        // [kDecayRows][8 R8]
+  pdl_enter();
+  const long long rows = static_cast<long long>(p.B) * p.S, row0 = static_cast<long long>(blockIdx.x) * kDecayRows;
+  const int n = static_cast<int>(rows - row0 < kDecayRows ? rows - row0 : kDecayRows);
+  const int ch = p.H * p.dkp, c = blockIdx.y * kThreads + threadIdx.x;
+  for (int x = threadIdx.x; x < n * 8 * R8; x += kThreads) {
+    const int t = x / (8 * R8), r = x - t * 8 * R8;
+    su[x] = r < p.rank ? to_f32(static_cast<const T*>(p.inner)[(row0 + t) * p.ldp + r]) : 0.f;
+  }
+  float w[R8 * 8], bias = 0.f;
+#pragma unroll
+  for (int x = 0; x < R8; ++x) {
+    float f[8] = {};
+    if (c < ch && x * 8 < p.rank) load8(static_cast<const T*>(p.a2) + static_cast<long long>(c) * p.rank + x * 8, f);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) w[x * 8 + e] = f[e];
+  }
+  if (c < ch) bias = to_f32(static_cast<const T*>(p.a2_b)[c]);
+  __syncthreads();
+  if (c >= ch) return;
+  float* out = p.log_decay + row0 * ch + c;
+  for (int t = 0; t < n; ++t) {
+    float z = bias;
+#pragma unroll
+    for (int x = 0; x < R8 * 2; ++x) {
+      const float4 u = *reinterpret_cast<const float4*>(su + t * 8 * R8 + x * 4);
+      z = fmaf(u.x, w[x * 4], z);
+      z = fmaf(u.y, w[x * 4 + 1], z);
+      z = fmaf(u.z, w[x * 4 + 2], z);
+      z = fmaf(u.w, w[x * 4 + 3], z);
+    }
+    out[static_cast<long long>(t) * ch] = log_decay_of(z, p.inv_tau);
+  }
+}
+
+// any rank
+template <typename T>
+__global__ void __launch_bounds__(kThreads)
+gla_decay_wide_kernel(const LinearAttnParams p) {
   pdl_enter();
   const int ch = p.H * p.dkp;
   const long long row = blockIdx.x;
   const T* u = static_cast<const T*>(p.inner) + row * p.ldp;
   for (int c = threadIdx.x; c < ch; c += kThreads)
     p.log_decay[row * ch + c] = log_decay_of(decay_input<T>(p, u, c), p.inv_tau);
+}
+
+template <typename T>
+cudaError_t launch_decay(const LinearAttnParams& p, cudaStream_t st) {
+  const long long rows = static_cast<long long>(p.B) * p.S;
+  const dim3 grid(static_cast<unsigned>((rows + kDecayRows - 1) / kDecayRows), (p.H * p.dkp + kThreads - 1) / kThreads);
+  auto bytes = [](int r8) { return static_cast<size_t>(kDecayRows) * 8 * r8 * sizeof(float); };
+  if (p.rank <= 16) return launch_kernel(gla_decay_kernel<T, 2>, grid, dim3(kThreads), bytes(2), st, p);
+  if (p.rank <= 32) return launch_kernel(gla_decay_kernel<T, 4>, grid, dim3(kThreads), bytes(4), st, p);
+  if (p.rank <= 64) return launch_kernel(gla_decay_kernel<T, 8>, grid, dim3(kThreads), bytes(8), st, p);
+  return launch_kernel(gla_decay_wide_kernel<T>, dim3(static_cast<unsigned>(rows)), dim3(kThreads), 0, st, p);
 }
 
 constexpr int kSteps = 16;      // tokens staged in shared memory at a time
@@ -245,10 +298,8 @@ cudaError_t launch_gla_step(const LinearAttnParams& p, int fp32, cudaStream_t st
 }
 
 cudaError_t launch_gla_decay(const LinearAttnParams& p, int fp32, cudaStream_t st) {
-  const dim3 grid(static_cast<unsigned>(p.B * p.S));
-  if (grid.x == 0) return cudaSuccess;
-  return fp32 ? launch_kernel(gla_decay_kernel<float>, grid, dim3(kThreads), 0, st, p)
-              : launch_kernel(gla_decay_kernel<bf16>, grid, dim3(kThreads), 0, st, p);
+  if (p.B == 0 || p.S == 0) return cudaSuccess;
+  return fp32 ? launch_decay<float>(p, st) : launch_decay<bf16>(p, st);
 }
 
 cudaError_t launch_gla_sequence(const LinearAttnParams& p, int fp32, cudaStream_t st) {

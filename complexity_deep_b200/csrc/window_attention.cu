@@ -1,7 +1,7 @@
 // Sliding-window attention with kept first tokens, distance bias and head mixing: the per-head
 // norm, the ring append, and the kernel that handles one query per thread-block cluster.  The
-// latter serves decoding (norm and append fused) and every call in 32-bit storage; prompts in
-// bf16 take the tensor-core kernel of window_attention_prefill.cu.
+// latter serves prompts in 32-bit storage and head layouts that the kernels of
+// window_attention_prefill.cu (prompts in bf16) and window_attention_decode.cu do not take.
 #include <cfloat>
 #include <cooperative_groups.h>
 #include "kernels.h"
@@ -78,9 +78,9 @@ window_append_kernel(const WindowAttnParams p) {
 }
 
 struct RowsSmem {   // offsets in floats
-  int q, s, m, stat, o, red, k_new, total;
+  int q, s, m, stat, o, red, total;
 };
-__host__ __device__ inline RowsSmem rows_smem(int H, int G, int dp, int vp, int cap) {
+__host__ __device__ inline RowsSmem rows_smem(int H, int dp, int vp, int cap) {
   RowsSmem L;
   L.q = 0;                                  // [H][dp]
   L.s = L.q + H * dp;                       // [H][cap] scores, then weights
@@ -88,15 +88,12 @@ __host__ __device__ inline RowsSmem rows_smem(int H, int G, int dp, int vp, int 
   L.stat = L.m + H * cap;                   // [2][H] this block's maximum and sum
   L.o = L.stat + ((2 * H + 3) & ~3);        // [H][vp] this block's part of the output
   L.red = L.o + H * vp;                     // [kThreads][kRep * 8]
-  L.k_new = L.red + kThreads * kRep * 8;    // [G][dp] normed key of the new token (decode)
-  L.total = L.k_new + G * dp;
+  L.total = L.red + kThreads * kRep * 8;
   return L;
 }
 
 // One query per cluster of `gridDim.x / S` blocks; the blocks share the query's keys and exchange
 // their softmax statistics and parts of the output through distributed shared memory.
-// Decode form (S == 1, !normed): q and the new key are normed here and the new key and value are
-// written to the ring by the block that holds them.
 template <typename T>
 __global__ void __launch_bounds__(kThreads)
 window_rows_kernel(const WindowAttnParams p, int cap) {
@@ -108,7 +105,7 @@ window_rows_kernel(const WindowAttnParams p, int cap) {
   const int rank = static_cast<int>(cluster.block_rank());
   const int t = blockIdx.x / CL, b = blockIdx.y;
   const int H = p.H, G = p.G, rep = H / G, dp = p.dp, vp = p.vp;
-  const RowsSmem L = rows_smem(H, G, dp, vp, cap);
+  const RowsSmem L = rows_smem(H, dp, vp, cap);
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int pos0 = window_pos0(p);
   const int i = pos0 + t;
@@ -119,29 +116,9 @@ window_rows_kernel(const WindowAttnParams p, int cap) {
   const int n0 = min(rank * chunk, count);
   const int nk = min(chunk, count - n0);        // keys of this block (0 possible)
 
-  // queries, pre-scaled; the decode form norms them here
+  // queries, pre-scaled
   const T* qrow = static_cast<const T*>(p.q) + row * p.ldp;
-  const T* krow = static_cast<const T*>(p.k) + row * p.ldp;
-  for (int h = warp; h < H + (p.normed ? 0 : G); h += kThreads / 32) {
-    const bool is_q = h < H;
-    const T* x = is_q ? qrow + static_cast<long long>(h) * dp : krow + static_cast<long long>(h - H) * dp;
-    const T* w = static_cast<const T*>(is_q ? p.q_w : p.k_w);
-    float* dst = is_q ? sm + L.q + h * dp : sm + L.k_new + (h - H) * dp;
-    float r = 1.f;
-    if (!p.normed) {
-      float ss = 0.f;
-      for (int c = lane; c < dp; c += 32) {
-        const float f = to_f32(x[c]);
-        ss += f * f;
-      }
-      r = 1.0f / sqrtf(warp_add(ss) / static_cast<float>(p.dim) + p.eps);
-    }
-    for (int c = lane; c < dp; c += 32) {
-      float f = to_f32(x[c]);
-      if (!p.normed) f = to_f32(from_f32<T>(f * r * to_f32(w[c])));   // as the stored form rounds it
-      dst[c] = is_q ? f * p.scale : f;
-    }
-  }
+  for (int c = tid; c < H * dp; c += kThreads) sm[L.q + c] = to_f32(qrow[c]) * p.scale;
   __syncthreads();
 
   const long long slots = p.keep + p.window;
@@ -154,21 +131,14 @@ window_rows_kernel(const WindowAttnParams p, int cap) {
   for (int item = tid; item < nk * G; item += kThreads) {
     const int c = item / nk, n = item - c * nk;
     const int j = keys.position(n0 + n);
-    const bool own_new = !p.normed && j == i;     // the new token's key, in shared memory
     const T* kp = j >= pos0 ? new_k + (j - pos0) * p.ldp + static_cast<long long>(c) * dp
                             : ring_k + (static_cast<long long>(window_slot(j, p.window, p.keep)) * G + c) * dp;
-    const float* ks = sm + L.k_new + c * dp;
     const float dist = static_cast<float>(i - j);
     for (int r0 = 0; r0 < rep; r0 += kRep) {
       float acc[kRep] = {};
       for (int d = 0; d < dp; d += 8) {
         float f[8];
-        if (own_new) {
-#pragma unroll
-          for (int e = 0; e < 8; ++e) f[e] = ks[d + e];
-        } else {
-          load8(kp + d, f);
-        }
+        load8(kp + d, f);
 #pragma unroll
         for (int r = 0; r < kRep; ++r) {
           if (r0 + r < rep) {
@@ -188,14 +158,6 @@ window_rows_kernel(const WindowAttnParams p, int cap) {
         }
       }
     }
-  }
-  if (!p.normed && nk > 0 && n0 + nk == count) {
-    // this block holds the new token: append it (its slot is not read by this query)
-    const long long slot = window_slot(i, p.window, p.keep);
-    T* rk = static_cast<T*>(p.ring_k) + (b * slots + slot) * G * dp;
-    T* rv = static_cast<T*>(p.ring_v) + (b * slots + slot) * G * vp;
-    for (int c = tid; c < G * dp; c += kThreads) rk[c] = from_f32<T>(sm[L.k_new + c]);
-    for (int c = tid; c < G * vp; c += kThreads) rv[c] = new_v[c];
   }
   __syncthreads();
 
@@ -302,7 +264,7 @@ template <typename T>
 cudaError_t launch_rows(const WindowAttnParams& p, cudaStream_t st) {
   const int n_max = p.keep + p.window;
   auto bytes = [&](int cl) {
-    return static_cast<size_t>(rows_smem(p.H, p.G, p.dp, p.vp, (n_max + cl - 1) / cl).total) * sizeof(float);
+    return static_cast<size_t>(rows_smem(p.H, p.dp, p.vp, (n_max + cl - 1) / cl).total) * sizeof(float);
   };
   // blocks per query: enough to fill the device when there are few queries, and enough for the
   // scores to fit in shared memory
@@ -333,7 +295,7 @@ cudaError_t launch_rows(const WindowAttnParams& p, cudaStream_t st) {
 }  // namespace
 
 bool window_rows_supported(const WindowAttnParams& p) {
-  return static_cast<size_t>(rows_smem(p.H, p.G, p.dp, p.vp, (p.keep + p.window + 7) / 8).total) * sizeof(float) <=
+  return static_cast<size_t>(rows_smem(p.H, p.dp, p.vp, (p.keep + p.window + 7) / 8).total) * sizeof(float) <=
          kMaxDynSmem;
 }
 

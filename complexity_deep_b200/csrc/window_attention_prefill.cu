@@ -26,8 +26,6 @@ namespace cdeep {
 
 namespace {
 
-constexpr int kWarps = 8;
-constexpr int kThreads = kWarps * 32;
 constexpr float kLog2e = 1.4426950408889634f;
 constexpr float kMasked = -1e30f;
 
@@ -50,14 +48,14 @@ struct Tile {
 struct PrefillSmem {   // byte offsets
   int q, k, v, p, bias, stat, talk, total;
 };
-template <int HU, int MB, int KT>
+template <int HU, int MB, int KT, int DQ>
 __host__ __device__ inline PrefillSmem prefill_smem(int H, int G, int dp, int vp) {
   using L = Tile<HU, MB, KT>;
   constexpr int HP = L::kHP;
   PrefillSmem s;
   const int kv = G * (dp > vp ? dp : vp) + 8;            // both buffers can hold a K tile (first pass)
-  s.q = 0;                                               // [MQ][H * dp + 8]
-  s.k = s.q + L::kMQ * (H * dp + 8) * 2;                 // [KT][G * dp + 8]
+  s.q = 0;                                               // [MQ][H * dp + 8] (DQ = 0)
+  s.k = s.q + (DQ ? 0 : L::kMQ * (H * dp + 8) * 2);      // [KT][G * dp + 8]
   s.v = s.k + KT * kv * 2;                               // [KT][G * vp + 8]
   s.p = s.v + KT * kv * 2;                               // high parts, low parts: [HP][MQ][KT]
   s.bias = s.p + 2 * HP * L::kHead * 2;                  // [2][H][MQ + KT]
@@ -67,18 +65,20 @@ __host__ __device__ inline PrefillSmem prefill_smem(int H, int G, int dp, int vp
   return s;
 }
 
-template <int HU, int MB, int NV8, int KT>
-__global__ void __launch_bounds__(kThreads, 1)
+// NV8: value columns / 8 at most; DQ: the queries stay in registers as DQ fragments (head width up to
+// 16 DQ), 0: in shared memory
+template <int kWarps, int HU, int MB, int NV8, int KT, int DQ>
+__global__ void __launch_bounds__(kWarps * 32, 1)
 window_prefill_kernel(const WindowAttnParams p) {
+  constexpr int kThreads = kWarps * 32;
   using L = Tile<HU, MB, KT>;
   constexpr int HP = L::kHP;
   constexpr int kMQ = L::kMQ;
   constexpr int kUnits = HU * MB / kWarps;               // (head, query block) units per warp
-  constexpr int kNT = KT / 8;                            // 8-key column tiles
   extern __shared__ __align__(16) unsigned char smem[];
   pdl_enter();
   const int H = p.H, G = p.G, rep = H / G, dp = p.dp, vp = p.vp;
-  const PrefillSmem off = prefill_smem<HU, MB, KT>(H, G, dp, vp);
+  const PrefillSmem off = prefill_smem<HU, MB, KT, DQ>(H, G, dp, vp);
   bf16* sQ = reinterpret_cast<bf16*>(smem + off.q);
   bf16* sK = reinterpret_cast<bf16*>(smem + off.k);
   bf16* sV = reinterpret_cast<bf16*>(smem + off.v);
@@ -146,11 +146,28 @@ window_prefill_kernel(const WindowAttnParams p) {
   };
 
   // ---------------------------------------------------------------- set-up
-  for (int r = warp; r < kMQ; r += kWarps)
-    for (int c = lane * 8; c < H * dp; c += 256) {
-      if (r < nq) copy16_async(sQ + r * ldq + c, new_q + (t0 + r) * p.ldp + c);
-      else *reinterpret_cast<uint4*>(sQ + r * ldq + c) = make_uint4(0, 0, 0, 0);
+  uint32_t qf[kUnits][DQ ? DQ : 1][4];                  // A fragments of this warp's queries
+  if constexpr (DQ > 0) {
+#pragma unroll
+    for (int u = 0; u < kUnits; ++u) {
+      const int unit = warp * kUnits + u, h = unit / MB, mb = unit - h * MB;
+#pragma unroll
+      for (int x = 0; x < DQ; ++x)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const int r = mb * 16 + (lane >> 2) + (e & 1) * 8, c = x * 16 + (lane & 3) * 2 + (e >> 1) * 8;
+          qf[u][x][e] = (h < H && r < nq && c < dp)
+                            ? *reinterpret_cast<const uint32_t*>(new_q + (t0 + r) * p.ldp + static_cast<long long>(h) * dp + c)
+                            : 0u;
+        }
     }
+  } else {
+    for (int r = warp; r < kMQ; r += kWarps)
+      for (int c = lane * 8; c < H * dp; c += 256) {
+        if (r < nq) copy16_async(sQ + r * ldq + c, new_q + (t0 + r) * p.ldp + c);
+        else *reinterpret_cast<uint4*>(sQ + r * ldq + c) = make_uint4(0, 0, 0, 0);
+      }
+  }
   load_tile(0, sK, ldk, new_k, ring_k, G * dp);          // one group with the queries
   for (int idx = tid; idx < HP * HP; idx += kThreads) {
     const int h = idx / HP, g = idx - h * HP;
@@ -165,22 +182,21 @@ window_prefill_kernel(const WindowAttnParams p) {
   const float scale2 = p.scale * kLog2e;
   const int r_lo = lane >> 2, c_lo = (lane & 3) * 2;     // row and column of a fragment's first element
 
-  // scores of all units of this warp on the K tile in `kbuf` (scaled, biased, masked, log2 domain)
-  auto scores = [&](int t, const bf16* kbuf, float (&s)[kUnits][kNT][4]) {
+  // scores of all units of this warp on 16 keys (from `k0` on) of the K tile in `kbuf` (scaled, biased,
+  // masked, log2 domain)
+  auto scores = [&](int t, int k0, const bf16* kbuf, float (&s)[kUnits][2][4]) {
     int j0, n;
     tile_keys(t, j0, n);
 #pragma unroll
     for (int u = 0; u < kUnits; ++u)
 #pragma unroll
-      for (int nt = 0; nt < kNT; ++nt)
+      for (int nt = 0; nt < 2; ++nt)
 #pragma unroll
         for (int e = 0; e < 4; ++e) s[u][nt][e] = 0.f;
-    const int a_row = lane & 15, a_col = (lane >> 4) * 8;          // ldmatrix addresses: A 16 x 16
     const int b_row = (lane & 7) + ((lane >> 4) << 3), b_col = ((lane >> 3) & 1) * 8;   // B: 16 keys x 16
-    const uint32_t q_base = smem_addr(sQ + a_row * ldq + a_col);
-    const uint32_t k_base = smem_addr(kbuf + b_row * ldk + b_col);
-    for (int d = 0; d < dp; d += 16) {
-      uint32_t kb[kNT / 2][4];
+    const uint32_t k_base = smem_addr(kbuf + (k0 + b_row) * ldk + b_col);
+    auto step = [&](int d, auto query) {                 // 16 elements of the head from d on
+      uint32_t kb[4];
       int loaded = -1;
 #pragma unroll
       for (int u = 0; u < kUnits; ++u) {
@@ -188,18 +204,29 @@ window_prefill_kernel(const WindowAttnParams p) {
         if (h >= H) break;
         const int c = h / rep;
         if (c != loaded) {
-#pragma unroll
-          for (int x = 0; x < kNT / 2; ++x) ldsm4(kb[x], k_base + static_cast<uint32_t>((x * 16 * ldk + c * dp + d) * 2));
+          ldsm4(kb, k_base + static_cast<uint32_t>((c * dp + d) * 2));
           loaded = c;
         }
         uint32_t qa[4];
-        ldsm4(qa, q_base + static_cast<uint32_t>((mb * 16 * ldq + h * dp + d) * 2));
-#pragma unroll
-        for (int x = 0; x < kNT / 2; ++x) {
-          mma16816(s[u][2 * x], qa, kb[x][0], kb[x][1]);
-          mma16816(s[u][2 * x + 1], qa, kb[x][2], kb[x][3]);
-        }
+        query(u, h, mb, qa);
+        mma16816(s[u][0], qa, kb[0], kb[1]);
+        mma16816(s[u][1], qa, kb[2], kb[3]);
       }
+    };
+    if constexpr (DQ > 0) {
+#pragma unroll
+      for (int x = 0; x < DQ; ++x)
+        if (x * 16 < dp)
+          step(x * 16, [&](int u, int, int, uint32_t (&qa)[4]) {
+#pragma unroll
+            for (int e = 0; e < 4; ++e) qa[e] = qf[u][x][e];
+          });
+    } else {
+      const uint32_t q_base = smem_addr(sQ + (lane & 15) * ldq + (lane >> 4) * 8);
+      for (int d = 0; d < dp; d += 16)
+        step(d, [&](int, int h, int mb, uint32_t (&qa)[4]) {
+          ldsm4(qa, q_base + static_cast<uint32_t>((mb * 16 * ldq + h * dp + d) * 2));
+        });
     }
     // every (query, key) of the tile visible?
     const bool full = n == KT && j0 + KT - 1 <= i0 && (i0 + kMQ - 1 - j0 < p.window || j0 + KT - 1 < p.keep);
@@ -212,8 +239,8 @@ window_prefill_kernel(const WindowAttnParams p) {
       for (int e = 0; e < 4; ++e) {
         const int qr = mb * 16 + r_lo + (e >> 1) * 8;
 #pragma unroll
-        for (int nt = 0; nt < kNT; ++nt) {
-          const int kc = nt * 8 + c_lo + (e & 1);
+        for (int nt = 0; nt < 2; ++nt) {
+          const int kc = k0 + nt * 8 + c_lo + (e & 1);
           float v = fmaf(s[u][nt][e], scale2, -bias[qr - kc]);
           if (!full) {
             const int i = i0 + qr, j = j0 + kc;
@@ -238,21 +265,22 @@ window_prefill_kernel(const WindowAttnParams p) {
     __syncthreads();                        // tile t is there; everybody is done with tile t - 1
     const bf16* kbuf = (t & 1) ? sV : sK;
     load_tile(t + 1, (t & 1) ? sK : sV, ldk, new_k, ring_k, G * dp);
-    float s[kUnits][kNT][4];
-    scores(t, kbuf, s);
+    for (int k0 = 0; k0 < KT; k0 += 16) {
+      float s[kUnits][2][4];
+      scores(t, k0, kbuf, s);
 #pragma unroll
-    for (int u = 0; u < kUnits; ++u) {
-      if ((warp * kUnits + u) / MB >= H) break;
+      for (int u = 0; u < kUnits; ++u) {
+        if ((warp * kUnits + u) / MB >= H) break;
 #pragma unroll
-      for (int r = 0; r < 2; ++r) {
-        float m = m_run[u][r];
+        for (int r = 0; r < 2; ++r) {
+          const float m = fmaxf(fmaxf(m_run[u][r], fmaxf(s[u][0][2 * r], s[u][0][2 * r + 1])),
+                                fmaxf(s[u][1][2 * r], s[u][1][2 * r + 1]));
+          float l = l_run[u][r] * exp2_fast(m_run[u][r] - m);
 #pragma unroll
-        for (int nt = 0; nt < kNT; ++nt) m = fmaxf(m, fmaxf(s[u][nt][2 * r], s[u][nt][2 * r + 1]));
-        float l = l_run[u][r] * exp2_fast(m_run[u][r] - m);
-#pragma unroll
-        for (int nt = 0; nt < kNT; ++nt) l += exp2_fast(s[u][nt][2 * r] - m) + exp2_fast(s[u][nt][2 * r + 1] - m);
-        m_run[u][r] = m;
-        l_run[u][r] = l;
+          for (int nt = 0; nt < 2; ++nt) l += exp2_fast(s[u][nt][2 * r] - m) + exp2_fast(s[u][nt][2 * r + 1] - m);
+          m_run[u][r] = m;
+          l_run[u][r] = l;
+        }
       }
     }
   }
@@ -299,9 +327,10 @@ window_prefill_kernel(const WindowAttnParams p) {
     fill_bias(t);
     copy_wait<1>();                         // K of this tile (V may still be on its way)
     __syncthreads();
-    {
-      float s[kUnits][kNT][4];
-      scores(t, sK, s);
+#pragma unroll 1
+    for (int k0 = 0; k0 < KT; k0 += 16) {
+      float s[kUnits][2][4];
+      scores(t, k0, sK, s);
 #pragma unroll
       for (int u = 0; u < kUnits; ++u) {
         const int unit = warp * kUnits + u, h = unit / MB, mb = unit - h * MB;
@@ -310,9 +339,9 @@ window_prefill_kernel(const WindowAttnParams p) {
         for (int r = 0; r < 2; ++r) {
           const int qr = mb * 16 + r_lo + r * 8;
           const float lse = sStat[h * kMQ + qr];
-          const int at = h * L::kHead + qr * L::kRow + c_lo;
+          const int at = h * L::kHead + qr * L::kRow + k0 + c_lo;
 #pragma unroll
-          for (int nt = 0; nt < kNT; ++nt) {
+          for (int nt = 0; nt < 2; ++nt) {
             const float a = s[u][nt][2 * r], c = s[u][nt][2 * r + 1];
             const float pa = a > 0.5f * kMasked ? exp2_fast(a - lse) : 0.f;
             const float pc = c > 0.5f * kMasked ? exp2_fast(c - lse) : 0.f;
@@ -421,29 +450,27 @@ window_prefill_kernel(const WindowAttnParams p) {
 
 constexpr int kMaxDynSmem = 227 * 1024;
 
-template <int HU, int MB, int NV8, int KT>
+template <int W, int HU, int MB, int NV8, int KT, int DQ>
 bool try_launch(const WindowAttnParams& p, cudaStream_t st, cudaError_t& e, bool only_ask) {
-  const int bytes = prefill_smem<HU, MB, KT>(p.H, p.G, p.dp, p.vp).total;
-  if (bytes > kMaxDynSmem) return false;
+  const int bytes = prefill_smem<HU, MB, KT, DQ>(p.H, p.G, p.dp, p.vp).total;
+  if (bytes > kMaxDynSmem || p.H > HU || p.vp > NV8 * 8 || (DQ && p.dp > DQ * 16)) return false;
   if (only_ask) return true;
-  auto kern = window_prefill_kernel<HU, MB, NV8, KT>;
+  auto kern = window_prefill_kernel<W, HU, MB, NV8, KT, DQ>;
   e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, kMaxDynSmem);
   if (e != cudaSuccess) return true;
   const int mq = MB * 16;
-  e = launch_kernel(kern, dim3((p.S + mq - 1) / mq, p.B), dim3(kThreads), bytes, st, p);
+  e = launch_kernel(kern, dim3((p.S + mq - 1) / mq, p.B), dim3(W * 32), bytes, st, p);
   return true;
 }
 
-// Registers per thread bound units x value columns, shared memory the rest: the largest tile first.
+// Registers per thread bound units x (value columns + query fragments), shared memory the rest: the
+// largest tile that fits.
 bool dispatch(const WindowAttnParams& p, cudaStream_t st, cudaError_t& e, bool only_ask) {
-  if (p.H <= 8 && p.vp <= 80 && p.S > 16 && try_launch<8, 2, 10, 32>(p, st, e, only_ask)) return true;
-  if (p.H <= 8 && p.vp <= 128 && p.S > 16 && try_launch<8, 2, 16, 32>(p, st, e, only_ask)) return true;
-  if (p.H <= 8 && p.vp <= 256 && try_launch<8, 1, 32, 16>(p, st, e, only_ask)) return true;
-  if (p.H <= 16 && p.vp <= 64 && try_launch<16, 1, 8, 32>(p, st, e, only_ask)) return true;
-  if (p.H <= 16 && p.vp <= 128 && try_launch<16, 1, 16, 32>(p, st, e, only_ask)) return true;
-  if (p.H <= 16 && p.vp <= 128 && try_launch<16, 1, 16, 16>(p, st, e, only_ask)) return true;
-  if (p.H <= 32 && p.vp <= 64 && try_launch<32, 1, 8, 16>(p, st, e, only_ask)) return true;
-  return false;
+  return (p.S > 16 && try_launch<16, 8, 2, 16, 32, 8>(p, st, e, only_ask)) ||
+         try_launch<16, 16, 1, 16, 32, 8>(p, st, e, only_ask) ||
+         try_launch<16, 16, 1, 16, 16, 0>(p, st, e, only_ask) ||
+         try_launch<8, 8, 1, 32, 16, 0>(p, st, e, only_ask) ||
+         try_launch<16, 32, 1, 8, 16, 0>(p, st, e, only_ask);
 }
 
 }  // namespace

@@ -867,8 +867,8 @@ def window_attention_(proj: dict, out: torch.Tensor, weights: dict, ring_k: torc
                       dim: int, vdim: int, window: int, keep: int, scale: float, eps: float,
                       out_scale: float, pos0: int, pos_dev: Optional[torch.Tensor] = None) -> None:
     """Attention of `seq_len` new tokens per sequence over a sliding window with kept first tokens
-    (cd_window_attn).  proj: 'q', 'k', 'v' column slices of the projection buffer (normed in place
-    when seq_len > 1); weights: 'q_norm', 'k_norm', 'r1', 'r2', 'talk'; the rings receive the new
+    (cd_window_attn).  proj: 'q', 'k', 'v' column slices of the projection buffer (may be normed in
+    place); weights: 'q_norm', 'k_norm', 'r1', 'r2', 'talk'; the rings receive the new
     keys and values; `out` = columns of the mixers' output buffer."""
     lib = _lib.load()
     dt = out.dtype
@@ -899,9 +899,12 @@ def window_attention_(proj: dict, out: torch.Tensor, weights: dict, ring_k: torc
         scale=float(scale), eps=float(eps), out_scale=float(out_scale), B=batch, S=seq_len, H=heads,
         G=kv_heads, dim=dim, dp=dp, vdim=vdim, vp=vp, window=window, keep=keep, pos0=pos0, normed=0)
     ref = ctypes.byref(a)
-    if seq_len == 1:
-        with _Span("window_attention_decode"):
-            _lib.check(lib.cd_window_attention_rows(ref, fp32, _stream()), "cd_window_attention_rows")
+    ws_bytes = lib.cd_window_attention_decode_workspace_bytes(ref) if seq_len == 1 else 0
+    if ws_bytes:
+        ws = torch.empty(ws_bytes, dtype=torch.uint8, device=out.device)
+        with _Span("window_attention_decode", 2):
+            _lib.check(lib.cd_window_attention_decode(ref, ws.data_ptr(), ws_bytes, fp32, _stream()),
+                       "cd_window_attention_decode")
         return
     with _Span("head_norm"):
         _lib.check(lib.cd_window_attention_norm(ref, fp32, _stream()), "cd_window_attention_norm")

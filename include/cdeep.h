@@ -428,13 +428,17 @@ typedef struct cd_window_attn {
   int normed;           /* q and k rows are normed already */
 } cd_window_attn;
 
-/* 1 when the sizes are within what the kernels take. */
-int cd_window_attention_supported(const cd_window_attn* h_args);
 /* Norms the q and k heads of every row in place. */
 int cd_window_attention_norm(const cd_window_attn* h_args, int fp32, void* stream);
-/* One query per thread-block cluster.  normed = 1: any S, keys of the call from k / v, earlier ones
- * from the ring.  normed = 0 (S must be 1): q and the new key are normed by the kernel, which also
- * writes the new key and value into the ring. */
+/* One new token per sequence (S = 1, normed = 0): two kernels that norm q and the new key, write the
+ * new key and value into the ring and stream the ring once.  The workspace size is 0 where the form
+ * does not apply (heads wider than 256). */
+size_t cd_window_attention_decode_workspace_bytes(const cd_window_attn* h_args);
+int cd_window_attention_decode(const cd_window_attn* h_args, void* workspace, size_t bytes, int fp32,
+                               void* stream);
+/* One query per thread-block cluster (normed = 1, any S): keys of the call from k / v, earlier ones
+ * from the ring.  cd_window_attention_supported: the scores of a query fit in a cluster. */
+int cd_window_attention_supported(const cd_window_attn* h_args);
 int cd_window_attention_rows(const cd_window_attn* h_args, int fp32, void* stream);
 /* Tensor-core form for prompts in bf16 (normed = 1): a tile of queries with all heads per block.
  * Not every head layout fits (cd_window_attention_prefill_supported); the form above takes any. */
