@@ -42,6 +42,24 @@ __device__ __forceinline__ void store8(float* p, const float (&f)[8]) {
   *reinterpret_cast<float4*>(p + 4) = make_float4(f[4], f[5], f[6], f[7]);
 }
 
+// the same eight elements as loaded, for values in flight
+template <typename T> struct Raw8;
+template <> struct Raw8<bf16> { uint4 w; };
+template <> struct Raw8<float> { float4 a, b; };
+__device__ __forceinline__ void raw_load(const bf16* p, Raw8<bf16>& r) { r.w = *reinterpret_cast<const uint4*>(p); }
+__device__ __forceinline__ void raw_load(const float* p, Raw8<float>& r) {
+  r.a = *reinterpret_cast<const float4*>(p);
+  r.b = *reinterpret_cast<const float4*>(p + 4);
+}
+__device__ __forceinline__ void raw_unpack(const Raw8<bf16>& r, float (&f)[8]) {
+  f[0] = bf_lo(r.w.x); f[1] = bf_hi(r.w.x); f[2] = bf_lo(r.w.y); f[3] = bf_hi(r.w.y);
+  f[4] = bf_lo(r.w.z); f[5] = bf_hi(r.w.z); f[6] = bf_lo(r.w.w); f[7] = bf_hi(r.w.w);
+}
+__device__ __forceinline__ void raw_unpack(const Raw8<float>& r, float (&f)[8]) {
+  f[0] = r.a.x; f[1] = r.a.y; f[2] = r.a.z; f[3] = r.a.w;
+  f[4] = r.b.x; f[5] = r.b.y; f[6] = r.b.z; f[7] = r.b.w;
+}
+
 __device__ __forceinline__ float warp_add(float v) {
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
@@ -58,6 +76,25 @@ __device__ __forceinline__ float warp_max(float v) {
 __device__ __forceinline__ void pdl_enter() {
   asm volatile("griddepcontrol.wait;" ::: "memory");
   asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
+}
+
+__device__ __forceinline__ float exp2_approx(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+__device__ __forceinline__ float log2_approx(float x) {
+  float y;
+  asm("lg2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+// exp and log(1 + x) of attention scores: the hardware approximations for bf16 storage (absolute
+// error of a score ~1e-7 of its size), the full-precision functions for fp32 storage
+template <typename T> __device__ __forceinline__ float score_exp(float x) {
+  return sizeof(T) == 2 ? exp2_approx(x * 1.4426950408889634f) : expf(x);
+}
+template <typename T> __device__ __forceinline__ float score_log1p(float x) {
+  return sizeof(T) == 2 ? 0.6931471805599453f * log2_approx(1.0f + x) : log1pf(x);
 }
 
 __device__ __forceinline__ float silu_precise(float g) { return g / (1.0f + expf(-g)); }

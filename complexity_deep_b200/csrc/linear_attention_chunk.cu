@@ -26,6 +26,7 @@ constexpr int kC = 64;                 // tokens per chunk
 constexpr int kThreads = 256;
 constexpr float kMaxSpan = 120.f;
 constexpr int kLdA = kC + 8;
+constexpr int kBatch = 8;              // tokens loaded at a time by a channel's thread (divides a segment)
 
 __host__ __device__ inline int segments(int dkp) {   // threads per channel, each with kC / segments tokens
   int s = 8;
@@ -55,7 +56,13 @@ __device__ __forceinline__ Sums chunk_sums(const LinearAttnParams& a, const floa
   r.t_hi = r.t_lo + len;
   float sum = 0.f;
   if (r.c >= 0) {
-    for (int t = r.t_lo; t < min(r.t_hi, n); ++t) sum += ld[static_cast<long long>(t) * ch + r.c];
+    for (int t0 = r.t_lo; t0 < r.t_hi; t0 += kBatch) {
+      float v[kBatch];
+#pragma unroll
+      for (int x = 0; x < kBatch; ++x) v[x] = t0 + x < n ? ld[static_cast<long long>(t0 + x) * ch + r.c] : 0.f;
+#pragma unroll
+      for (int x = 0; x < kBatch; ++x) sum += v[x];
+    }
     s_seg[seg * a.dkp + r.c] = sum;
   }
   __syncthreads();
@@ -107,13 +114,20 @@ gla_chunk_update_kernel(const ChunkParams p) {
   const Sums s = chunk_sums(a, ld, n, s_seg);
   if (s.c >= 0) {
     float cum = s.start;
-    for (int t = s.t_lo; t < s.t_hi; ++t) {
-      float v = 0.f;
-      if (t < n) {
-        cum += ld[static_cast<long long>(t) * ch + s.c];
-        v = to_f32(k[t * a.ldp + s.c]) * expf(s.total - cum);
+    for (int t0 = s.t_lo; t0 < s.t_hi; t0 += kBatch) {
+      float d[kBatch];
+      bf16 kv[kBatch];
+#pragma unroll
+      for (int x = 0; x < kBatch; ++x) {
+        const bool ok = t0 + x < n;
+        d[x] = ok ? ld[static_cast<long long>(t0 + x) * ch + s.c] : 0.f;
+        kv[x] = ok ? k[(t0 + x) * a.ldp + s.c] : __float2bfloat16_rn(0.f);
       }
-      store_split(skh, skl, t * ldk + s.c, v);
+#pragma unroll
+      for (int x = 0; x < kBatch; ++x) {
+        cum += d[x];
+        store_split(skh, skl, (t0 + x) * ldk + s.c, to_f32(kv[x]) * expf(s.total - cum));
+      }
     }
     if (s.t_lo == 0) p.total[slot * a.dkp + s.c] = s.total;
   }
@@ -244,16 +258,24 @@ gla_chunk_output_kernel(const ChunkParams p) {
   const float ref = fast ? 0.5f * s.total : 0.f;
   if (s.c >= 0) {
     float cum = s.start;
-    for (int t = s.t_lo; t < s.t_hi; ++t) {
-      float qv = 0.f, kv = 0.f;
-      if (t < n) {
-        cum += ld[static_cast<long long>(t) * ch + s.c];
-        qv = to_f32(q[t * a.ldp + s.c]) * a.q_scale * expf(cum - ref);
-        if (fast) kv = to_f32(k[t * a.ldp + s.c]) * expf(ref - cum);
+    for (int t0 = s.t_lo; t0 < s.t_hi; t0 += kBatch) {
+      float d[kBatch];
+      bf16 qv[kBatch], kv[kBatch];
+#pragma unroll
+      for (int x = 0; x < kBatch; ++x) {
+        const bool ok = t0 + x < n;
+        d[x] = ok ? ld[static_cast<long long>(t0 + x) * ch + s.c] : 0.f;
+        qv[x] = ok ? q[(t0 + x) * a.ldp + s.c] : __float2bfloat16_rn(0.f);
+        kv[x] = ok ? k[(t0 + x) * a.ldp + s.c] : __float2bfloat16_rn(0.f);
       }
-      store_split(sqh, sql, t * ldk + s.c, qv);
-      if (fast) store_split(skh, skl, t * ldk + s.c, kv);
-      else sB[t * dkp + s.c] = cum;
+#pragma unroll
+      for (int x = 0; x < kBatch; ++x) {
+        const int t = t0 + x;
+        cum += d[x];
+        store_split(sqh, sql, t * ldk + s.c, to_f32(qv[x]) * a.q_scale * expf(cum - ref));
+        if (fast) store_split(skh, skl, t * ldk + s.c, to_f32(kv[x]) * expf(ref - cum));
+        else sB[t * dkp + s.c] = cum;
+      }
     }
     if (s.t_lo == 0) s_ref[s.c] = expf(ref);
   }
@@ -329,40 +351,44 @@ gla_chunk_output_kernel(const ChunkParams p) {
     const int col = (j * kSlots + slot) * 16;
     if (col >= dvp) continue;
     // the state's fragments come straight from memory: rows (lane % 4) * 2 + {0, 1, 8, 9}, column lane / 4
-    float f[8], nxt[8];
-    auto fetch = [&](int d, float (&v)[8]) {
+    constexpr int kFetch = NJ == 1 ? 4 : 2;              // steps of 16 rows in flight
+    for (int d0 = 0; d0 < dkp; d0 += 16 * kFetch) {
+      float f[kFetch][8];
 #pragma unroll
-      for (int y = 0; y < 2; ++y)
+      for (int z = 0; z < kFetch; ++z)
+        if (d0 + z * 16 < dkp) {
 #pragma unroll
-        for (int e = 0; e < 4; ++e) {
-          const int r = d + c_lo + (e & 1) + (e >> 1) * 8;
-          v[y * 4 + e] = S[static_cast<long long>(r) * dvp + col + y * 8 + r_lo];
+          for (int y = 0; y < 2; ++y)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+              const int r = d0 + z * 16 + c_lo + (e & 1) + (e >> 1) * 8;
+              f[z][y * 4 + e] = S[static_cast<long long>(r) * dvp + col + y * 8 + r_lo];
+            }
         }
-    };
-    fetch(0, nxt);
-    for (int d = 0; d < dkp; d += 16) {
 #pragma unroll
-      for (int e = 0; e < 8; ++e) f[e] = nxt[e];
-      if (d + 16 < dkp) fetch(d + 16, nxt);
-      const float2 fa = *reinterpret_cast<const float2*>(s_ref + d + c_lo);
-      const float2 fb = *reinterpret_cast<const float2*>(s_ref + d + c_lo + 8);
-      uint32_t bh[4], bl[4];
-#pragma unroll
-      for (int y = 0; y < 2; ++y) {
-        split_pair(f[y * 4] * fa.x, f[y * 4 + 1] * fa.y, bh[2 * y], bl[2 * y]);
-        split_pair(f[y * 4 + 2] * fb.x, f[y * 4 + 3] * fb.y, bh[2 * y + 1], bl[2 * y + 1]);
-      }
-#pragma unroll
-      for (int m = 0; m < MT; ++m) {
-        const int qa = ((m0 + m) * 16 + (lane & 15)) * ldk + d + (lane >> 4) * 8;
-        uint32_t ah[4], al[4];
-        ldsm4(ah, smem_addr(sqh + qa));
-        ldsm4(al, smem_addr(sql + qa));
+      for (int z = 0; z < kFetch; ++z) {
+        const int d = d0 + z * 16;
+        if (d >= dkp) break;
+        const float2 fa = *reinterpret_cast<const float2*>(s_ref + d + c_lo);
+        const float2 fb = *reinterpret_cast<const float2*>(s_ref + d + c_lo + 8);
+        uint32_t bh[4], bl[4];
 #pragma unroll
         for (int y = 0; y < 2; ++y) {
-          mma16816(acc[j][m][y], ah, bl[2 * y], bl[2 * y + 1]);
-          mma16816(acc[j][m][y], al, bh[2 * y], bh[2 * y + 1]);
-          mma16816(acc[j][m][y], ah, bh[2 * y], bh[2 * y + 1]);
+          split_pair(f[z][y * 4] * fa.x, f[z][y * 4 + 1] * fa.y, bh[2 * y], bl[2 * y]);
+          split_pair(f[z][y * 4 + 2] * fb.x, f[z][y * 4 + 3] * fb.y, bh[2 * y + 1], bl[2 * y + 1]);
+        }
+#pragma unroll
+        for (int m = 0; m < MT; ++m) {
+          const int qa = ((m0 + m) * 16 + (lane & 15)) * ldk + d + (lane >> 4) * 8;
+          uint32_t ah[4], al[4];
+          ldsm4(ah, smem_addr(sqh + qa));
+          ldsm4(al, smem_addr(sql + qa));
+#pragma unroll
+          for (int y = 0; y < 2; ++y) {
+            mma16816(acc[j][m][y], ah, bl[2 * y], bl[2 * y + 1]);
+            mma16816(acc[j][m][y], al, bh[2 * y], bh[2 * y + 1]);
+            mma16816(acc[j][m][y], ah, bh[2 * y], bh[2 * y + 1]);
+          }
         }
       }
     }

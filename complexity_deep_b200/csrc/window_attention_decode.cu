@@ -72,7 +72,7 @@ __device__ __forceinline__ float group8_add(float v) {
 
 // REP query heads per block; DC chunks of 8 elements per lane (head width up to 64 DC)
 template <typename T, int REP, int DC>
-__global__ void __launch_bounds__(kThreads)
+__global__ void __launch_bounds__(kThreads, REP * DC <= 4 && sizeof(T) == 2 ? 3 : 1)
 window_decode_scores_kernel(const DecodeParams p) {
   extern __shared__ float sm[];        // [REP][dp] queries
   __shared__ float s_m[kWarps][REP], s_l[kWarps][REP];
@@ -125,61 +125,71 @@ window_decode_scores_kernel(const DecodeParams p) {
 #pragma unroll
       for (int y = 0; y < 8; ++y) qf[x][e][y] = (x < nh && d < dp) ? sm[x * dp + d + y] : 0.f;
     }
-  // lane `sub` of a row keeps the statistics of head `sub`
-  float r1 = 0.f, r2 = 0.f, m = -FLT_MAX, l = 0.f;
-  if (sub < nh) {
-    r1 = to_f32(static_cast<const T*>(a.r1)[h0 + sub]);
-    r2 = to_f32(static_cast<const T*>(a.r2)[h0 + sub]);
-  }
-  float* out = p.scores + (static_cast<long long>(b) * a.H + h0 + (sub < nh ? sub : 0)) * p.n_max;
-  constexpr int kAhead = DC <= 2 ? 4 : 2;       // rows in flight per lane
+  // Rows in flight per lane.  The kAhead x REP scores of a lane group are finished by its lanes: lane
+  // `sub` takes the head sub % REP and, in `kRounds` rounds, row sub / REP + round * (8 / REP).
+  constexpr int kAhead = DC * sizeof(T) <= 4 ? 4 : 2;
+  constexpr int kRowsRound = 8 / REP < kAhead ? 8 / REP : kAhead;
+  constexpr int kRounds = kAhead / kRowsRound;
   constexpr int kStep = kWarps * 4;             // rows of the block per step
+  const int my_head = sub % REP, my_row = sub / REP;
+  float r1 = 0.f, r2 = 0.f, m = -FLT_MAX, l = 0.f;
+  if (my_head < nh) {
+    r1 = to_f32(static_cast<const T*>(a.r1)[h0 + my_head]);
+    r2 = to_f32(static_cast<const T*>(a.r2)[h0 + my_head]);
+  }
+  float* out = p.scores + (static_cast<long long>(b) * a.H + h0 + (my_head < nh ? my_head : 0)) * p.n_max;
   for (int base = 0; base < r.nk; base += kStep * kAhead) {
-    float kf[kAhead][DC][8];
+    Raw8<T> kf[kAhead][DC];
 #pragma unroll
     for (int u = 0; u < kAhead; ++u) {
-      const int n = base + u * kStep + warp * 4 + rg;
-      const T* k = ring_k + static_cast<long long>(r.slot(r.n0 + (n < r.nk ? n : 0))) * stride;
+      const int n = min(base + u * kStep + warp * 4 + rg, r.nk - 1);      // rows past the end are not used
+      const T* k = ring_k + static_cast<long long>(r.slot(r.n0 + n)) * stride;
 #pragma unroll
       for (int e = 0; e < DC; ++e) {
         const int d = (e * 8 + sub) * 8;
-        if (n < r.nk && d < dp) load8(k + d, kf[u][e]);
-        else
-#pragma unroll
-          for (int y = 0; y < 8; ++y) kf[u][e][y] = 0.f;
+        raw_load(k + (d < dp ? d : 0), kf[u][e]);                         // past the head: the query is zero
       }
     }
+    float s[kAhead][REP];
 #pragma unroll
     for (int u = 0; u < kAhead; ++u) {
-      const int n = base + u * kStep + warp * 4 + rg;
-      float s[REP];
 #pragma unroll
-      for (int x = 0; x < REP; ++x) {
-        float acc = 0.f;
+      for (int x = 0; x < REP; ++x) s[u][x] = 0.f;
 #pragma unroll
-        for (int e = 0; e < DC; ++e)
+      for (int e = 0; e < DC; ++e) {
+        float f[8];
+        raw_unpack(kf[u][e], f);
 #pragma unroll
-          for (int y = 0; y < 8; ++y) acc = fmaf(qf[x][e][y], kf[u][e][y], acc);
-        s[x] = group8_add(acc);
+        for (int x = 0; x < REP; ++x)
+#pragma unroll
+          for (int y = 0; y < 8; ++y) s[u][x] = fmaf(qf[x][e][y], f[y], s[u][x]);
       }
-      if (n < r.nk && sub < nh) {
-        float v = s[0];
 #pragma unroll
-        for (int x = 1; x < REP; ++x) v = sub == x ? s[x] : v;
-        v -= r1 * log1pf(r2 * static_cast<float>(r.distance(r.n0 + n)));
+      for (int x = 0; x < REP; ++x) s[u][x] = group8_add(s[u][x]);
+    }
+#pragma unroll
+    for (int y = 0; y < kRounds; ++y) {
+      float v = 0.f;
+#pragma unroll
+      for (int u = 0; u < kRowsRound; ++u)
+#pragma unroll
+        for (int x = 0; x < REP; ++x) v = (my_row == u && my_head == x) ? s[y * kRowsRound + u][x] : v;
+      const int n = base + (y * kRowsRound + my_row) * kStep + warp * 4 + rg;
+      if (n < r.nk && my_head < nh && my_row < kRowsRound) {
+        v -= r1 * score_log1p<T>(r2 * static_cast<float>(r.distance(r.n0 + n)));
         out[r.n0 + n] = v;
         const float mn = fmaxf(m, v);
-        l = l * expf(m - mn) + expf(v - mn);
+        l = l * score_exp<T>(m - mn) + score_exp<T>(v - mn);
         m = mn;
       }
     }
   }
-  // the block's statistics: the warp's four rows, then the warps
+  // the block's statistics: the lanes of a head, then the warps
 #pragma unroll
-  for (int d = 8; d < 32; d <<= 1) {
+  for (int d = REP; d < 32; d <<= 1) {
     const float mo = __shfl_xor_sync(0xffffffffu, m, d), lo = __shfl_xor_sync(0xffffffffu, l, d);
     const float mn = fmaxf(m, mo);
-    l = l * expf(m - mn) + lo * expf(mo - mn);
+    l = l * score_exp<T>(m - mn) + lo * score_exp<T>(mo - mn);
     m = mn;
   }
   if (lane < nh) {
@@ -201,7 +211,7 @@ window_decode_scores_kernel(const DecodeParams p) {
   }
 }
 
-constexpr int kKeys = 64;       // keys whose weights are formed at a time
+constexpr int kKeys = 128;      // keys whose weights are formed at a time
 
 struct ValuesSmem {   // offsets in floats
   int lse, talk, w, mix, red, o, total;
@@ -220,7 +230,7 @@ __host__ __device__ inline ValuesSmem values_smem(int H, int vp) {
 }
 
 template <typename T, int REP>
-__global__ void __launch_bounds__(kThreads)
+__global__ void __launch_bounds__(kThreads, REP <= 2 && sizeof(T) == 2 ? 3 : 2)
 window_decode_values_kernel(const DecodeParams p) {
   extern __shared__ float sm[];
   pdl_enter();
@@ -260,16 +270,16 @@ window_decode_values_kernel(const DecodeParams p) {
   for (int x = 0; x < REP; ++x)
 #pragma unroll
     for (int e = 0; e < 8; ++e) acc[x][e] = 0.f;
-  constexpr int kAhead = 4;
+  constexpr int kAhead = sizeof(T) == 2 ? 8 : 4;
   for (int base = 0; base < r.nk; base += kKeys) {
     const int n = min(kKeys, r.nk - base);
-    float vf[kAhead][8];
+    Raw8<T> vf[kAhead];
     // the first values are on their way while the weights are formed
     auto fetch = [&](int at) {
 #pragma unroll
       for (int u = 0; u < kAhead; ++u) {
         const int k = at + u * rows;
-        if (active && k < n) load8(ring_v + static_cast<long long>(r.slot(r.n0 + base + k)) * stride + col, vf[u]);
+        if (active && k < n) raw_load(ring_v + static_cast<long long>(r.slot(r.n0 + base + k)) * stride + col, vf[u]);
       }
     };
     fetch(row);
@@ -278,7 +288,7 @@ window_decode_values_kernel(const DecodeParams p) {
       const int h = x / kKeys, k = x - h * kKeys;
       if (k < n)
         sm[L.w + h * (kKeys + 1) + k] =
-            expf(scores[static_cast<long long>(h) * p.n_max + r.n0 + base + k] - sm[L.lse + h]) * sm[L.lse + H + h];
+            score_exp<T>(scores[static_cast<long long>(h) * p.n_max + r.n0 + base + k] - sm[L.lse + h]) * sm[L.lse + H + h];
     }
     __syncthreads();
     for (int x = tid; x < REP * kKeys; x += kThreads) {
@@ -295,11 +305,13 @@ window_decode_values_kernel(const DecodeParams p) {
       for (int u = 0; u < kAhead; ++u) {
         const int k = at + u * rows;
         if (k < n) {
+          float f[8];
+          raw_unpack(vf[u], f);
 #pragma unroll
           for (int x = 0; x < REP; ++x) {
             const float w = sm[L.mix + x * kKeys + k];
 #pragma unroll
-            for (int e = 0; e < 8; ++e) acc[x][e] = fmaf(w, vf[u][e], acc[x][e]);
+            for (int e = 0; e < 8; ++e) acc[x][e] = fmaf(w, f[e], acc[x][e]);
           }
         }
       }

@@ -13,13 +13,15 @@
 //   3. out_h += mixed_h V
 //
 // The distance bias is a table of one tile's distances per head, computed once per tile.  Keys come
-// from the projection buffer (this call's tokens) or from the ring (earlier ones), by cp.async.
+// from the projection buffer (this call's tokens) or from the ring (earlier ones), one bulk copy per
+// key and tile.
 //
 // Why warp-level products: with all heads of a query tile in flight, scores, mixed weights and
 // outputs of H heads x vdim columns exceed the 512 columns of tensor memory for any useful tile,
 // and the mixed weights must pass through registers of warps that see every head anyway.
 #include "kernels.h"
 #include "mma.cuh"
+#include "ptx.cuh"
 #include "window_attention.cuh"
 
 namespace cdeep {
@@ -29,10 +31,11 @@ namespace {
 constexpr float kLog2e = 1.4426950408889634f;
 constexpr float kMasked = -1e30f;
 
-__device__ __forceinline__ float exp2_fast(float x) {
-  float y;
-  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-  return y;
+// one row of `bytes` (a multiple of 16; both addresses 16-byte aligned), completing on `bar`
+__device__ __forceinline__ void bulk_copy(void* dst, const void* src, uint32_t bytes, uint64_t* bar) {
+  asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(
+                   smem_addr(dst)), "l"(src), "r"(bytes), "r"(smem_addr(bar))
+               : "memory");
 }
 
 // HU: heads dealt to the warps (8, 16 or 32); MB: blocks of 16 queries; KT: keys per tile
@@ -46,7 +49,7 @@ struct Tile {
 };
 
 struct PrefillSmem {   // byte offsets
-  int q, k, v, p, bias, stat, talk, total;
+  int q, k, v, p, bias, stat, talk, r, total;
 };
 template <int HU, int MB, int KT, int DQ>
 __host__ __device__ inline PrefillSmem prefill_smem(int H, int G, int dp, int vp) {
@@ -61,7 +64,8 @@ __host__ __device__ inline PrefillSmem prefill_smem(int H, int G, int dp, int vp
   s.bias = s.p + 2 * HP * L::kHead * 2;                  // [2][H][MQ + KT]
   s.stat = s.bias + 2 * H * L::kBias * 4;                // [H][MQ] log2 of the normaliser
   s.talk = s.stat + ((H * L::kMQ * 4 + 15) & ~15);       // [HP][HP + 8] bf16
-  s.total = s.talk + HP * (HP + 8) * 2;
+  s.r = s.talk + HP * (HP + 8) * 2;                      // r1, r2 of the heads
+  s.total = s.r + 2 * H * 4;
   return s;
 }
 
@@ -69,14 +73,23 @@ __host__ __device__ inline PrefillSmem prefill_smem(int H, int G, int dp, int vp
 // 16 DQ), 0: in shared memory
 template <int kWarps, int HU, int MB, int NV8, int KT, int DQ>
 __global__ void __launch_bounds__(kWarps * 32, 1)
-window_prefill_kernel(const WindowAttnParams p) {
+window_prefill_kernel(const WindowAttnParams p, int* status) {
   constexpr int kThreads = kWarps * 32;
   using L = Tile<HU, MB, KT>;
   constexpr int HP = L::kHP;
   constexpr int kMQ = L::kMQ;
   constexpr int kUnits = HU * MB / kWarps;               // (head, query block) units per warp
   extern __shared__ __align__(16) unsigned char smem[];
+  __shared__ uint64_t bars[2];                           // K buffer, V buffer
+  __shared__ int abort_word;
+  if (threadIdx.x == 0) {
+    mbar_init(&bars[0], 1);
+    mbar_init(&bars[1], 1);
+    abort_word = 0;
+    fence_barrier_init();
+  }
   pdl_enter();
+  __syncthreads();
   const int H = p.H, G = p.G, rep = H / G, dp = p.dp, vp = p.vp;
   const PrefillSmem off = prefill_smem<HU, MB, KT, DQ>(H, G, dp, vp);
   bf16* sQ = reinterpret_cast<bf16*>(smem + off.q);
@@ -87,6 +100,7 @@ window_prefill_kernel(const WindowAttnParams p) {
   float* sBias = reinterpret_cast<float*>(smem + off.bias);
   float* sStat = reinterpret_cast<float*>(smem + off.stat);
   bf16* sT = reinterpret_cast<bf16*>(smem + off.talk);
+  float* sR = reinterpret_cast<float*>(smem + off.r);
   const int ldq = H * dp + 8, ldk = G * dp + 8, ldv = G * vp + 8;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int b = blockIdx.y;
@@ -117,22 +131,24 @@ window_prefill_kernel(const WindowAttnParams p) {
       n = min(KT, i_last + 1 - j0);
     }
   };
-  auto load_tile = [&](int t, bf16* dst, int ld, const bf16* fresh, const bf16* ring, int width) {
-    if (t < tiles) {
-      int j0, n;
-      tile_keys(t, j0, n);
-      for (int r = warp; r < KT; r += kWarps) {
-        const int j = j0 + r;
-        const bf16* src = j >= pos0 ? fresh + (j - pos0) * p.ldp
-                                    : ring + static_cast<long long>(window_slot(j, p.window, p.keep)) * width;
-        for (int c = lane * 8; c < width; c += 256) {
-          if (r < n) copy16_async(dst + r * ld + c, src + c);
-          else *reinterpret_cast<uint4*>(dst + r * ld + c) = make_uint4(0, 0, 0, 0);
-        }
-      }
+  // Issued by the first warp, a lane per key; rows past the tile's keys repeat the last one (their
+  // scores are masked, their weights zero).  Called with every thread done with the buffer.
+  auto load_tile = [&](int t, bf16* dst, int ld, const bf16* fresh, const bf16* ring, int width, uint64_t* bar) {
+    if (warp != 0 || t >= tiles) return;
+    int j0, n;
+    tile_keys(t, j0, n);
+    if (lane == 0) mbar_arrive_expect_tx(bar, static_cast<uint32_t>(KT * width * 2));
+    __syncwarp();
+    if (lane < KT) {
+      const int j = j0 + min(lane, n - 1);
+      const bf16* src = j >= pos0 ? fresh + (j - pos0) * p.ldp
+                                  : ring + static_cast<long long>(window_slot(j, p.window, p.keep)) * width;
+      bulk_copy(dst + lane * ld, src, static_cast<uint32_t>(width * 2), bar);
     }
-    copy_commit();
   };
+  volatile int* abort_flag = &abort_word;
+  // use `count` (from 0) of a buffer has arrived
+  auto wait_tile = [&](uint64_t* bar, int count) { mbar_wait(bar, static_cast<uint32_t>(count & 1), abort_flag); };
   auto fill_bias = [&](int t) {
     int j0, n;
     tile_keys(t, j0, n);
@@ -140,8 +156,8 @@ window_prefill_kernel(const WindowAttnParams p) {
     for (int idx = tid; idx < H * L::kBias; idx += kThreads) {
       const int h = idx / L::kBias;
       const int d = max(i0 - j0 + (idx - h * L::kBias) - (KT - 1), 0);
-      const float r1 = to_f32(static_cast<const bf16*>(p.r1)[h]), r2 = to_f32(static_cast<const bf16*>(p.r2)[h]);
-      dst[idx] = r1 * log1pf(r2 * static_cast<float>(d)) * kLog2e;
+      // r1 ln(1 + r2 d) in the log2 domain; its absolute error is that of the logarithm's argument
+      dst[idx] = sR[h] * log2_approx(fmaf(sR[H + h], static_cast<float>(d), 1.0f));
     }
   };
 
@@ -168,7 +184,11 @@ window_prefill_kernel(const WindowAttnParams p) {
         else *reinterpret_cast<uint4*>(sQ + r * ldq + c) = make_uint4(0, 0, 0, 0);
       }
   }
-  load_tile(0, sK, ldk, new_k, ring_k, G * dp);          // one group with the queries
+  load_tile(0, sK, ldk, new_k, ring_k, G * dp, &bars[0]);
+  for (int h = tid; h < H; h += kThreads) {
+    sR[h] = to_f32(static_cast<const bf16*>(p.r1)[h]);
+    sR[H + h] = to_f32(static_cast<const bf16*>(p.r2)[h]);
+  }
   for (int idx = tid; idx < HP * HP; idx += kThreads) {
     const int h = idx / HP, g = idx - h * HP;
     sT[h * (HP + 8) + g] = (h < H && g < H) ? static_cast<const bf16*>(p.talk)[h * H + g] : __float2bfloat16_rn(0.f);
@@ -179,6 +199,9 @@ window_prefill_kernel(const WindowAttnParams p) {
     reinterpret_cast<uint4*>(sPl + H * L::kHead)[idx] = make_uint4(0, 0, 0, 0);
   }
 
+  int key_head[kUnits];
+#pragma unroll
+  for (int u = 0; u < kUnits; ++u) key_head[u] = min((warp * kUnits + u) / MB, H - 1) / rep;
   const float scale2 = p.scale * kLog2e;
   const int r_lo = lane >> 2, c_lo = (lane & 3) * 2;     // row and column of a fragment's first element
 
@@ -202,7 +225,7 @@ window_prefill_kernel(const WindowAttnParams p) {
       for (int u = 0; u < kUnits; ++u) {
         const int unit = warp * kUnits + u, h = unit / MB, mb = unit - h * MB;
         if (h >= H) break;
-        const int c = h / rep;
+        const int c = key_head[u];
         if (c != loaded) {
           ldsm4(kb, k_base + static_cast<uint32_t>((c * dp + d) * 2));
           loaded = c;
@@ -235,19 +258,23 @@ window_prefill_kernel(const WindowAttnParams p) {
       const int unit = warp * kUnits + u, h = unit / MB, mb = unit - h * MB;
       if (h >= H) break;
       const float* bias = sBias + (t & 1) * H * L::kBias + h * L::kBias + KT - 1;
+      if (full) {
 #pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const int qr = mb * 16 + r_lo + (e >> 1) * 8;
+        for (int e = 0; e < 4; ++e)
 #pragma unroll
-        for (int nt = 0; nt < 2; ++nt) {
-          const int kc = k0 + nt * 8 + c_lo + (e & 1);
-          float v = fmaf(s[u][nt][e], scale2, -bias[qr - kc]);
-          if (!full) {
+          for (int nt = 0; nt < 2; ++nt)
+            s[u][nt][e] = fmaf(s[u][nt][e], scale2,
+                               -bias[mb * 16 + r_lo + (e >> 1) * 8 - (k0 + nt * 8 + c_lo + (e & 1))]);
+      } else {
+#pragma unroll
+        for (int e = 0; e < 4; ++e)
+#pragma unroll
+          for (int nt = 0; nt < 2; ++nt) {
+            const int qr = mb * 16 + r_lo + (e >> 1) * 8, kc = k0 + nt * 8 + c_lo + (e & 1);
             const int i = i0 + qr, j = j0 + kc;
-            if (!(kc < n && j <= i && (i - j < p.window || j < p.keep))) v = kMasked;
+            const bool seen = kc < n && j <= i && (i - j < p.window || j < p.keep);
+            s[u][nt][e] = seen ? fmaf(s[u][nt][e], scale2, -bias[qr - kc]) : kMasked;
           }
-          s[u][nt][e] = v;
-        }
       }
     }
   };
@@ -259,12 +286,14 @@ window_prefill_kernel(const WindowAttnParams p) {
     m_run[u][0] = m_run[u][1] = kMasked;
     l_run[u][0] = l_run[u][1] = 0.f;
   }
+  copy_wait<0>();
+  __syncthreads();                          // queries (when staged), talk, r1, r2 are written
   for (int t = 0; t < tiles; ++t) {
     fill_bias(t);
-    copy_wait<0>();
+    wait_tile(&bars[t & 1], t >> 1);
     __syncthreads();                        // tile t is there; everybody is done with tile t - 1
     const bf16* kbuf = (t & 1) ? sV : sK;
-    load_tile(t + 1, (t & 1) ? sK : sV, ldk, new_k, ring_k, G * dp);
+    load_tile(t + 1, (t & 1) ? sK : sV, ldk, new_k, ring_k, G * dp, &bars[(t + 1) & 1]);
     for (int k0 = 0; k0 < KT; k0 += 16) {
       float s[kUnits][2][4];
       scores(t, k0, kbuf, s);
@@ -275,9 +304,9 @@ window_prefill_kernel(const WindowAttnParams p) {
         for (int r = 0; r < 2; ++r) {
           const float m = fmaxf(fmaxf(m_run[u][r], fmaxf(s[u][0][2 * r], s[u][0][2 * r + 1])),
                                 fmaxf(s[u][1][2 * r], s[u][1][2 * r + 1]));
-          float l = l_run[u][r] * exp2_fast(m_run[u][r] - m);
+          float l = l_run[u][r] * exp2_approx(m_run[u][r] - m);
 #pragma unroll
-          for (int nt = 0; nt < 2; ++nt) l += exp2_fast(s[u][nt][2 * r] - m) + exp2_fast(s[u][nt][2 * r + 1] - m);
+          for (int nt = 0; nt < 2; ++nt) l += exp2_approx(s[u][nt][2 * r] - m) + exp2_approx(s[u][nt][2 * r + 1] - m);
           m_run[u][r] = m;
           l_run[u][r] = l;
         }
@@ -296,7 +325,7 @@ window_prefill_kernel(const WindowAttnParams p) {
       for (int x = 1; x < 4; x <<= 1) {
         const float mo = __shfl_xor_sync(0xffffffffu, m, x), lo = __shfl_xor_sync(0xffffffffu, l, x);
         const float mn = fmaxf(m, mo);
-        l = l * exp2_fast(m - mn) + lo * exp2_fast(mo - mn);
+        l = l * exp2_approx(m - mn) + lo * exp2_approx(mo - mn);
         m = mn;
       }
       if ((lane & 3) == 0) sStat[h * kMQ + mb * 16 + r_lo + r * 8] = m + log2f(l);
@@ -311,10 +340,10 @@ window_prefill_kernel(const WindowAttnParams p) {
     for (int x = 0; x < NV8; ++x)
 #pragma unroll
       for (int e = 0; e < 4; ++e) acc[u][x][e] = 0.f;
-  copy_wait<0>();
   __syncthreads();                          // the first pass is done with both buffers; sStat is written
-  load_tile(0, sK, ldk, new_k, ring_k, G * dp);
-  load_tile(0, sV, ldv, new_v, ring_v, G * vp);
+  load_tile(0, sK, ldk, new_k, ring_k, G * dp, &bars[0]);
+  load_tile(0, sV, ldv, new_v, ring_v, G * vp, &bars[1]);
+  const int k_uses = (tiles + 1) / 2, v_uses = tiles / 2;   // of the buffers in the first pass
   // talk as the A operand, kept in registers
   uint32_t ta[HP / 16][HP / 16][4];
 #pragma unroll
@@ -325,7 +354,7 @@ window_prefill_kernel(const WindowAttnParams p) {
 
   for (int t = 0; t < tiles; ++t) {
     fill_bias(t);
-    copy_wait<1>();                         // K of this tile (V may still be on its way)
+    wait_tile(&bars[0], k_uses + t);
     __syncthreads();
 #pragma unroll 1
     for (int k0 = 0; k0 < KT; k0 += 16) {
@@ -343,8 +372,7 @@ window_prefill_kernel(const WindowAttnParams p) {
 #pragma unroll
           for (int nt = 0; nt < 2; ++nt) {
             const float a = s[u][nt][2 * r], c = s[u][nt][2 * r + 1];
-            const float pa = a > 0.5f * kMasked ? exp2_fast(a - lse) : 0.f;
-            const float pc = c > 0.5f * kMasked ? exp2_fast(c - lse) : 0.f;
+            const float pa = exp2_approx(a - lse), pc = exp2_approx(c - lse);   // masked: 0
             uint32_t hi, lo;
             split_pair(pa, pc, hi, lo);
             *reinterpret_cast<uint32_t*>(sP + at + nt * 8) = hi;
@@ -354,7 +382,7 @@ window_prefill_kernel(const WindowAttnParams p) {
       }
     }
     __syncthreads();
-    load_tile(t + 1, sK, ldk, new_k, ring_k, G * dp);
+    load_tile(t + 1, sK, ldk, new_k, ring_k, G * dp, &bars[0]);
     // mix the heads: a warp takes 16 keys of one query at a time
     for (int item = warp; item < kMQ * (KT / 16); item += kWarps) {
       const int qr = item / (KT / 16), k0 = (item - qr * (KT / 16)) * 16;
@@ -392,7 +420,7 @@ window_prefill_kernel(const WindowAttnParams p) {
           }
         }
     }
-    copy_wait<1>();                         // V of this tile (K of the next may still be on its way)
+    wait_tile(&bars[1], v_uses + t);
     __syncthreads();
     // out_h += mixed_h V_c
 #pragma unroll
@@ -412,9 +440,8 @@ window_prefill_kernel(const WindowAttnParams p) {
           int loaded = -1;
 #pragma unroll
           for (int u = 0; u < kUnits; ++u) {
-            const int unit = warp * kUnits + u, h = unit / MB;
-            if (h >= H) break;
-            const int c = h / rep;
+            if ((warp * kUnits + u) / MB >= H) break;
+            const int c = key_head[u];
             if (c != loaded) {
               ldsm4_t(vb, v_base + static_cast<uint32_t>((c * vp + x * 16) * 2));
               loaded = c;
@@ -426,9 +453,9 @@ window_prefill_kernel(const WindowAttnParams p) {
       }
     }
     __syncthreads();
-    load_tile(t + 1, sV, ldv, new_v, ring_v, G * vp);
+    load_tile(t + 1, sV, ldv, new_v, ring_v, G * vp, &bars[1]);
   }
-  copy_wait<0>();
+  if (tid == 0 && *abort_flag) atomicExch(status, 1);
 
   bf16* out = static_cast<bf16*>(p.out);
 #pragma unroll
@@ -448,7 +475,7 @@ window_prefill_kernel(const WindowAttnParams p) {
   }
 }
 
-constexpr int kMaxDynSmem = 227 * 1024;
+constexpr int kMaxDynSmem = 226 * 1024;
 
 template <int W, int HU, int MB, int NV8, int KT, int DQ>
 bool try_launch(const WindowAttnParams& p, cudaStream_t st, cudaError_t& e, bool only_ask) {
@@ -459,7 +486,7 @@ bool try_launch(const WindowAttnParams& p, cudaStream_t st, cudaError_t& e, bool
   e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, kMaxDynSmem);
   if (e != cudaSuccess) return true;
   const int mq = MB * 16;
-  e = launch_kernel(kern, dim3((p.S + mq - 1) / mq, p.B), dim3(W * 32), bytes, st, p);
+  e = launch_kernel(kern, dim3((p.S + mq - 1) / mq, p.B), dim3(W * 32), bytes, st, p, device_status_word());
   return true;
 }
 
