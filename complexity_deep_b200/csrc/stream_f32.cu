@@ -20,7 +20,13 @@ embed_rows_kernel(const long long* __restrict__ ids, const T* __restrict__ table
   id = id < 0 ? 0 : (id >= V ? V - 1 : id);
   const T* src = table + id * ldw;
   float* dst = x + static_cast<size_t>(t) * ldx;
-  for (int c = threadIdx.x; c < ldx; c += blockDim.x) dst[c] = c < W ? to_f32(src[c]) : 0.f;
+  const int whole = (ldw & 7) == 0 ? (W & ~7) : 0;       // columns copied eight at a time
+  for (int c = threadIdx.x * 8; c < whole; c += blockDim.x * 8) {
+    float f[8];
+    load8(src + c, f);
+    store8(dst + c, f);
+  }
+  for (int c = whole + threadIdx.x; c < ldx; c += blockDim.x) dst[c] = c < W ? to_f32(src[c]) : 0.f;
 }
 
 // out[t, :] = x[t, :] / sqrt(mean(x^2) + eps) * (w + offset); the mean runs over W columns, rows

@@ -16,29 +16,33 @@ namespace {
 constexpr int kThreads = 256;
 constexpr int kRep = 4;          // query heads of a group handled together
 
-// q and k heads of every row in place: x / rms(x) * w, mean over `dim` columns.  One warp per head.
-template <typename T>
+// q and k heads of every row in place: x / rms(x) * w, mean over `dim` columns.  LPH lanes per head,
+// eight columns per lane and round.
+template <typename T, int LPH>
 __global__ void __launch_bounds__(256)
 head_norm_kernel(const WindowAttnParams p) {
   pdl_enter();
   const int heads = p.H + p.G;
-  const long long item = blockIdx.x * 8ll + (threadIdx.x >> 5);
-  if (item >= static_cast<long long>(p.B) * p.S * heads) return;
-  const int lane = threadIdx.x & 31;
-  const long long row = item / heads;
-  const int h = static_cast<int>(item - row * heads);
+  const long long item = (blockIdx.x * 256ll + threadIdx.x) / LPH;
+  const bool ok = item < static_cast<long long>(p.B) * p.S * heads;
+  const int sub = threadIdx.x % LPH;
+  const long long row = ok ? item / heads : 0;
+  const int h = ok ? static_cast<int>(item - row * heads) : 0;
   const bool is_q = h < p.H;
   T* x = static_cast<T*>(is_q ? p.q : p.k) + row * p.ldp + static_cast<long long>(is_q ? h : h - p.H) * p.dp;
   const T* w = static_cast<const T*>(is_q ? p.q_w : p.k_w);
   float ss = 0.f;
-  for (int c = lane * 8; c < p.dp; c += 256) {
+  for (int c = sub * 8; c < p.dp; c += LPH * 8) {
     float f[8];
     load8(x + c, f);
 #pragma unroll
     for (int e = 0; e < 8; ++e) ss += f[e] * f[e];
   }
-  const float r = 1.0f / sqrtf(warp_add(ss) / static_cast<float>(p.dim) + p.eps);
-  for (int c = lane * 8; c < p.dp; c += 256) {
+#pragma unroll
+  for (int d = 1; d < LPH; d <<= 1) ss += __shfl_xor_sync(0xffffffffu, ss, d);
+  const float r = 1.0f / sqrtf(ss / static_cast<float>(p.dim) + p.eps);
+  if (!ok) return;
+  for (int c = sub * 8; c < p.dp; c += LPH * 8) {
     float f[8], wv[8];
     load8(x + c, f);
     load8(w + c, wv);
@@ -46,6 +50,15 @@ head_norm_kernel(const WindowAttnParams p) {
     for (int e = 0; e < 8; ++e) f[e] *= r * wv[e];
     store8(x + c, f);
   }
+}
+
+template <typename T>
+cudaError_t head_norm_any(const WindowAttnParams& p, cudaStream_t st) {
+  const long long items = static_cast<long long>(p.B) * p.S * (p.H + p.G);
+  auto grid = [&](int lph) { return dim3(static_cast<unsigned>((items * lph + 255) / 256)); };
+  if (p.dp <= 64) return launch_kernel(head_norm_kernel<T, 8>, grid(8), dim3(256), 0, st, p);
+  if (p.dp <= 128) return launch_kernel(head_norm_kernel<T, 16>, grid(16), dim3(256), 0, st, p);
+  return launch_kernel(head_norm_kernel<T, 32>, grid(32), dim3(256), 0, st, p);
 }
 
 // Rows of the call that later queries may see go into the ring: the kept first positions and the
@@ -300,11 +313,8 @@ bool window_rows_supported(const WindowAttnParams& p) {
 }
 
 cudaError_t launch_head_norm(const WindowAttnParams& p, int fp32, cudaStream_t st) {
-  const long long items = static_cast<long long>(p.B) * p.S * (p.H + p.G);
-  if (items == 0) return cudaSuccess;
-  const dim3 grid(static_cast<unsigned>((items + 7) / 8));
-  return fp32 ? launch_kernel(head_norm_kernel<float>, grid, dim3(256), 0, st, p)
-              : launch_kernel(head_norm_kernel<bf16>, grid, dim3(256), 0, st, p);
+  if (p.B == 0 || p.S == 0) return cudaSuccess;
+  return fp32 ? head_norm_any<float>(p, st) : head_norm_any<bf16>(p, st);
 }
 
 cudaError_t launch_window_append(const WindowAttnParams& p, int fp32, cudaStream_t st) {
