@@ -70,8 +70,9 @@ __host__ __device__ inline PrefillSmem prefill_smem(int H, int G, int dp, int vp
 }
 
 // NV8: value columns / 8 at most; DQ: the queries stay in registers as DQ fragments (head width up to
-// 16 DQ), 0: in shared memory
-template <int kWarps, int HU, int MB, int NV8, int KT, int DQ>
+// 16 DQ), 0: in shared memory; kExact: heads, head width and value columns are exactly HU, 16 DQ and
+// 8 NV8, so that the products of a tile form straight-line code
+template <int kWarps, int HU, int MB, int NV8, int KT, int DQ, bool kExact>
 __global__ void __launch_bounds__(kWarps * 32, 1)
 window_prefill_kernel(const WindowAttnParams p, int* status) {
   constexpr int kThreads = kWarps * 32;
@@ -90,7 +91,8 @@ window_prefill_kernel(const WindowAttnParams p, int* status) {
   }
   pdl_enter();
   __syncthreads();
-  const int H = p.H, G = p.G, rep = H / G, dp = p.dp, vp = p.vp;
+  const int H = kExact ? HU : p.H, G = p.G, rep = H / G;
+  const int dp = kExact ? DQ * 16 : p.dp, vp = kExact ? NV8 * 8 : p.vp;
   const PrefillSmem off = prefill_smem<HU, MB, KT, DQ>(H, G, dp, vp);
   bf16* sQ = reinterpret_cast<bf16*>(smem + off.q);
   bf16* sK = reinterpret_cast<bf16*>(smem + off.k);
@@ -131,20 +133,19 @@ window_prefill_kernel(const WindowAttnParams p, int* status) {
       n = min(KT, i_last + 1 - j0);
     }
   };
-  // Issued by the first warp, a lane per key; rows past the tile's keys repeat the last one (their
-  // scores are masked, their weights zero).  Called with every thread done with the buffer.
+  // Every warp issues its share of the keys, a lane per key; rows past the tile's keys repeat the last
+  // one (their scores are masked, their weights zero).  Called with every thread done with the buffer.
+  constexpr int kRowsWarp = KT / kWarps > 0 ? KT / kWarps : 1;
   auto load_tile = [&](int t, bf16* dst, int ld, const bf16* fresh, const bf16* ring, int width, uint64_t* bar) {
-    if (warp != 0 || t >= tiles) return;
+    const int r = warp * kRowsWarp + lane;
+    if (t >= tiles || lane >= kRowsWarp || r >= KT) return;
+    if (r == 0) mbar_arrive_expect_tx(bar, static_cast<uint32_t>(KT * width * 2));
     int j0, n;
     tile_keys(t, j0, n);
-    if (lane == 0) mbar_arrive_expect_tx(bar, static_cast<uint32_t>(KT * width * 2));
-    __syncwarp();
-    if (lane < KT) {
-      const int j = j0 + min(lane, n - 1);
-      const bf16* src = j >= pos0 ? fresh + (j - pos0) * p.ldp
-                                  : ring + static_cast<long long>(window_slot(j, p.window, p.keep)) * width;
-      bulk_copy(dst + lane * ld, src, static_cast<uint32_t>(width * 2), bar);
-    }
+    const int j = j0 + min(r, n - 1);
+    const bf16* src = fresh + (j - pos0) * p.ldp;
+    if (j < pos0) src = ring + static_cast<long long>(window_slot(j, p.window, p.keep)) * width;
+    bulk_copy(dst + r * ld, src, static_cast<uint32_t>(width * 2), bar);
   };
   volatile int* abort_flag = &abort_word;
   // use `count` (from 0) of a buffer has arrived
@@ -224,7 +225,7 @@ window_prefill_kernel(const WindowAttnParams p, int* status) {
 #pragma unroll
       for (int u = 0; u < kUnits; ++u) {
         const int unit = warp * kUnits + u, h = unit / MB, mb = unit - h * MB;
-        if (h >= H) break;
+        if (!kExact && h >= H) break;
         const int c = key_head[u];
         if (c != loaded) {
           ldsm4(kb, k_base + static_cast<uint32_t>((c * dp + d) * 2));
@@ -239,7 +240,7 @@ window_prefill_kernel(const WindowAttnParams p, int* status) {
     if constexpr (DQ > 0) {
 #pragma unroll
       for (int x = 0; x < DQ; ++x)
-        if (x * 16 < dp)
+        if (kExact || x * 16 < dp)
           step(x * 16, [&](int u, int, int, uint32_t (&qa)[4]) {
 #pragma unroll
             for (int e = 0; e < 4; ++e) qa[e] = qf[u][x][e];
@@ -256,7 +257,7 @@ window_prefill_kernel(const WindowAttnParams p, int* status) {
 #pragma unroll
     for (int u = 0; u < kUnits; ++u) {
       const int unit = warp * kUnits + u, h = unit / MB, mb = unit - h * MB;
-      if (h >= H) break;
+      if (!kExact && h >= H) break;
       const float* bias = sBias + (t & 1) * H * L::kBias + h * L::kBias + KT - 1;
       if (full) {
 #pragma unroll
@@ -294,12 +295,13 @@ window_prefill_kernel(const WindowAttnParams p, int* status) {
     __syncthreads();                        // tile t is there; everybody is done with tile t - 1
     const bf16* kbuf = (t & 1) ? sV : sK;
     load_tile(t + 1, (t & 1) ? sK : sV, ldk, new_k, ring_k, G * dp, &bars[(t + 1) & 1]);
+#pragma unroll
     for (int k0 = 0; k0 < KT; k0 += 16) {
       float s[kUnits][2][4];
       scores(t, k0, kbuf, s);
 #pragma unroll
       for (int u = 0; u < kUnits; ++u) {
-        if ((warp * kUnits + u) / MB >= H) break;
+        if (!kExact && (warp * kUnits + u) / MB >= H) break;
 #pragma unroll
         for (int r = 0; r < 2; ++r) {
           const float m = fmaxf(fmaxf(m_run[u][r], fmaxf(s[u][0][2 * r], s[u][0][2 * r + 1])),
@@ -317,7 +319,7 @@ window_prefill_kernel(const WindowAttnParams p, int* status) {
 #pragma unroll
   for (int u = 0; u < kUnits; ++u) {
     const int unit = warp * kUnits + u, h = unit / MB, mb = unit - h * MB;
-    if (h >= H) break;
+    if (!kExact && h >= H) break;
 #pragma unroll
     for (int r = 0; r < 2; ++r) {
       float m = m_run[u][r], l = l_run[u][r];
@@ -363,7 +365,7 @@ window_prefill_kernel(const WindowAttnParams p, int* status) {
 #pragma unroll
       for (int u = 0; u < kUnits; ++u) {
         const int unit = warp * kUnits + u, h = unit / MB, mb = unit - h * MB;
-        if (h >= H) break;
+        if (!kExact && h >= H) break;
 #pragma unroll
         for (int r = 0; r < 2; ++r) {
           const int qr = mb * 16 + r_lo + r * 8;
@@ -429,18 +431,18 @@ window_prefill_kernel(const WindowAttnParams p, int* status) {
 #pragma unroll
       for (int u = 0; u < kUnits; ++u) {
         const int unit = warp * kUnits + u, h = unit / MB, mb = unit - h * MB;
-        if (h < H)
+        if (kExact || h < H)
           ldsm4(pa[u], smem_addr(sP + h * L::kHead + (mb * 16 + (lane & 15)) * L::kRow + kk * 16 + (lane >> 4) * 8));
       }
       const uint32_t v_base = smem_addr(sV + (kk * 16 + (lane & 15)) * ldv + (lane >> 4) * 8);
 #pragma unroll
       for (int x = 0; x < NV8 / 2; ++x) {
-        if (x * 16 < vp) {
+        if (kExact || x * 16 < vp) {
           uint32_t vb[4];
           int loaded = -1;
 #pragma unroll
           for (int u = 0; u < kUnits; ++u) {
-            if ((warp * kUnits + u) / MB >= H) break;
+            if (!kExact && (warp * kUnits + u) / MB >= H) break;
             const int c = key_head[u];
             if (c != loaded) {
               ldsm4_t(vb, v_base + static_cast<uint32_t>((c * vp + x * 16) * 2));
@@ -461,7 +463,7 @@ window_prefill_kernel(const WindowAttnParams p, int* status) {
 #pragma unroll
   for (int u = 0; u < kUnits; ++u) {
     const int unit = warp * kUnits + u, h = unit / MB, mb = unit - h * MB;
-    if (h >= H) break;
+    if (!kExact && h >= H) break;
 #pragma unroll
     for (int r = 0; r < 2; ++r) {
       const int qr = mb * 16 + r_lo + r * 8;
@@ -477,12 +479,13 @@ window_prefill_kernel(const WindowAttnParams p, int* status) {
 
 constexpr int kMaxDynSmem = 226 * 1024;
 
-template <int W, int HU, int MB, int NV8, int KT, int DQ>
+template <int W, int HU, int MB, int NV8, int KT, int DQ, bool kExact = false>
 bool try_launch(const WindowAttnParams& p, cudaStream_t st, cudaError_t& e, bool only_ask) {
   const int bytes = prefill_smem<HU, MB, KT, DQ>(p.H, p.G, p.dp, p.vp).total;
   if (bytes > kMaxDynSmem || p.H > HU || p.vp > NV8 * 8 || (DQ && p.dp > DQ * 16)) return false;
+  if (kExact && (p.H != HU || p.vp != NV8 * 8 || p.dp != DQ * 16)) return false;
   if (only_ask) return true;
-  auto kern = window_prefill_kernel<W, HU, MB, NV8, KT, DQ>;
+  auto kern = window_prefill_kernel<W, HU, MB, NV8, KT, DQ, kExact>;
   e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, kMaxDynSmem);
   if (e != cudaSuccess) return true;
   const int mq = MB * 16;
@@ -493,7 +496,9 @@ bool try_launch(const WindowAttnParams& p, cudaStream_t st, cudaError_t& e, bool
 // Registers per thread bound units x (value columns + query fragments), shared memory the rest: the
 // largest tile that fits.
 bool dispatch(const WindowAttnParams& p, cudaStream_t st, cudaError_t& e, bool only_ask) {
-  return (p.S > 16 && try_launch<16, 8, 2, 16, 32, 8>(p, st, e, only_ask)) ||
+  return (p.S > 16 && try_launch<16, 8, 2, 16, 32, 8, true>(p, st, e, only_ask)) ||
+         try_launch<16, 16, 1, 16, 32, 8, true>(p, st, e, only_ask) ||
+         (p.S > 16 && try_launch<16, 8, 2, 16, 32, 8>(p, st, e, only_ask)) ||
          try_launch<16, 16, 1, 16, 32, 8>(p, st, e, only_ask) ||
          try_launch<16, 16, 1, 16, 16, 0>(p, st, e, only_ask) ||
          try_launch<8, 8, 1, 32, 16, 0>(p, st, e, only_ask) ||
