@@ -227,7 +227,7 @@ window_prefill_kernel(const WindowAttnParams p, int* status) {
         const int unit = warp * kUnits + u, h = unit / MB, mb = unit - h * MB;
         if (!kExact && h >= H) break;
         const int c = key_head[u];
-        if (c != loaded) {
+        if (u == 0 || c != loaded) {
           ldsm4(kb, k_base + static_cast<uint32_t>((c * dp + d) * 2));
           loaded = c;
         }
@@ -386,7 +386,9 @@ window_prefill_kernel(const WindowAttnParams p, int* status) {
     __syncthreads();
     load_tile(t + 1, sK, ldk, new_k, ring_k, G * dp, &bars[0]);
     // mix the heads: a warp takes 16 keys of one query at a time
-    for (int item = warp; item < kMQ * (KT / 16); item += kWarps) {
+#pragma unroll
+    for (int it = 0; it < kMQ * (KT / 16) / kWarps; ++it) {
+      const int item = it * kWarps + warp;
       const int qr = item / (KT / 16), k0 = (item - qr * (KT / 16)) * 16;
       float d[HP / 16][2][4];
 #pragma unroll
@@ -444,7 +446,7 @@ window_prefill_kernel(const WindowAttnParams p, int* status) {
           for (int u = 0; u < kUnits; ++u) {
             if (!kExact && (warp * kUnits + u) / MB >= H) break;
             const int c = key_head[u];
-            if (c != loaded) {
+            if (u == 0 || c != loaded) {
               ldsm4_t(vb, v_base + static_cast<uint32_t>((c * vp + x * 16) * 2));
               loaded = c;
             }
