@@ -1,14 +1,16 @@
 // Window attention of one new token per sequence (decoding), bound by the two passes over the ring.
 // The heads' weights are mixed after the softmax, so the values cannot be weighted before the
-// normalisers of all heads are known; two kernels:
+// normalisers of all heads are known; three kernels:
 //
 //   scores   grid (splits, key heads x query-head groups, sequences): a block streams its share of the
 //            keys of one key head for up to four query heads; 8 lanes share a key.  Scores (scaled,
 //            biased) go to a workspace that stays in L2, with every block's softmax statistics.  The
 //            block that holds the new token norms its key and writes key and value into the ring.
-//   values   same grid, the splits of a (head group, sequence) form a thread-block cluster: combines
-//            the statistics, forms and mixes the weights of all heads for its keys, streams its share
-//            of the values; the parts are added through distributed shared memory.
+//   mix      grid (64 keys, sequences): combines the statistics, replaces the scores of all heads by
+//            their mixed weights.
+//   values   grid as for the scores, the splits of a (head group, sequence) form a thread-block
+//            cluster: streams its share of the values; the parts are added through distributed shared
+//            memory.
 #include <cfloat>
 #include <cooperative_groups.h>
 #include "kernels.h"
@@ -27,7 +29,7 @@ struct DecodeParams {
   WindowAttnParams a;
   int splits;
   int n_max;        // keep + window
-  float* scores;    // [B, H, n_max]
+  float* scores;    // [B, H, n_max], then the mixed weights
   float* stats;     // [B, H, splits, 2]
 };
 
@@ -211,41 +213,19 @@ window_decode_scores_kernel(const DecodeParams p) {
   }
 }
 
-constexpr int kKeys = 128;      // keys whose weights are formed at a time
+constexpr int kMixKeys = 64;       // keys per block of the mixing kernel
 
-struct ValuesSmem {   // offsets in floats
-  int lse, talk, w, mix, red, o, total;
-};
-template <int REP>
-__host__ __device__ inline ValuesSmem values_smem(int H, int vp) {
-  ValuesSmem s;
-  s.lse = 0;                                   // [H] maximum, [H] 1 / sum
-  s.talk = s.lse + 2 * H;                      // [REP][H]
-  s.w = s.talk + REP * H;                      // [H][kKeys + 1]
-  s.mix = s.w + H * (kKeys + 1);               // [REP][kKeys]
-  s.o = s.mix + REP * kKeys;                   // [REP][vp]
-  s.red = s.o + REP * vp;                      // [REP * 8][kThreads]
-  s.total = s.red + REP * 8 * kThreads;
-  return s;
-}
-
-template <typename T, int REP>
-__global__ void __launch_bounds__(kThreads, REP <= 2 && sizeof(T) == 2 ? 3 : 2)
-window_decode_values_kernel(const DecodeParams p) {
-  extern __shared__ float sm[];
+template <typename T>
+__global__ void __launch_bounds__(kThreads)
+window_decode_mix_kernel(const DecodeParams p) {
+  extern __shared__ float sm[];        // [H] maximum, [H] 1 / sum, [H][kMixKeys] weights
   pdl_enter();
-  cg::cluster_group cluster = cg::this_cluster();
   const WindowAttnParams& a = p.a;
-  const int split = blockIdx.x, b = blockIdx.z, rep = a.H / a.G, groups = (rep + REP - 1) / REP;
-  const int c = blockIdx.y / groups, h0 = c * rep + (blockIdx.y % groups) * REP;
-  const int nh = min(REP, (c + 1) * rep - h0);
-  const int tid = threadIdx.x, H = a.H, vp = a.vp;
-  const ValuesSmem L = values_smem<REP>(H, vp);
-  const KeyRange r(a, split, p.splits);
-  const long long slots = a.keep + a.window;
-  const T* ring_v = static_cast<const T*>(a.ring_v) + (b * slots * a.G + c) * vp;
-  const long long stride = static_cast<long long>(a.G) * vp;
-  for (int h = tid; h < H; h += kThreads) {
+  const int H = a.H, b = blockIdx.y, n0 = blockIdx.x * kMixKeys;
+  const KeyRange r(a, 0, 1);
+  const int n = min(kMixKeys, r.count - n0);
+  if (n <= 0) return;
+  for (int h = threadIdx.x; h < H; h += kThreads) {
     const float* st = p.stats + (static_cast<long long>(b) * H + h) * p.splits * 2;
     float m = -FLT_MAX, l = 0.f;
     for (int s = 0; s < p.splits; ++s) {
@@ -254,86 +234,99 @@ window_decode_values_kernel(const DecodeParams p) {
       l = l * expf(m - mn) + st[2 * s + 1] * expf(st[2 * s] - mn);
       m = mn;
     }
-    sm[L.lse + h] = m;
-    sm[L.lse + H + h] = 1.0f / l;
+    sm[h] = m;
+    sm[H + h] = 1.0f / l;
   }
-  for (int x = tid; x < REP * H; x += kThreads)
-    sm[L.talk + x] = x / H < nh ? to_f32(static_cast<const T*>(a.talk)[(h0 + x / H) * H + x % H]) : 0.f;
+  __syncthreads();
+  float* scores = p.scores + static_cast<long long>(b) * H * p.n_max + n0;
+  float* w = sm + 2 * H;
+  for (int x = threadIdx.x; x < H * kMixKeys; x += kThreads) {
+    const int h = x / kMixKeys, k = x - h * kMixKeys;
+    w[x] = k < n ? score_exp<T>(scores[static_cast<long long>(h) * p.n_max + k] - sm[h]) * sm[H + h] : 0.f;
+  }
+  __syncthreads();
+  const T* talk = static_cast<const T*>(a.talk);
+  for (int x = threadIdx.x; x < H * kMixKeys; x += kThreads) {
+    const int h = x / kMixKeys, k = x - h * kMixKeys;
+    float v = 0.f;
+    for (int g = 0; g < H; ++g) v = fmaf(to_f32(talk[h * H + g]), w[g * kMixKeys + k], v);
+    if (k < n) scores[static_cast<long long>(h) * p.n_max + k] = v;
+  }
+}
 
+template <int REP>
+__host__ __device__ inline int values_smem_floats(int vp) {
+  return REP * 8 * kThreads + REP * vp;          // the threads' sums [REP * 8][kThreads], the block's output [REP][vp]
+}
+
+template <typename T, int REP>
+__global__ void __launch_bounds__(kThreads, REP <= 2 && sizeof(T) == 2 ? 4 : 2)
+window_decode_values_kernel(const DecodeParams p) {
+  extern __shared__ float sm[];
+  pdl_enter();
+  cg::cluster_group cluster = cg::this_cluster();
+  const WindowAttnParams& a = p.a;
+  const int split = blockIdx.x, b = blockIdx.z, rep = a.H / a.G, groups = (rep + REP - 1) / REP;
+  const int c = blockIdx.y / groups, h0 = c * rep + (blockIdx.y % groups) * REP;
+  const int nh = min(REP, (c + 1) * rep - h0);
+  const int tid = threadIdx.x, vp = a.vp;
+  float* s_out = sm + REP * 8 * kThreads;
+  const KeyRange r(a, split, p.splits);
+  const long long slots = a.keep + a.window;
+  const T* ring_v = static_cast<const T*>(a.ring_v) + (b * slots * a.G + c) * vp;
+  const long long stride = static_cast<long long>(a.G) * vp;
   // a thread takes eight columns and every `rows`-th key
-  const int cols = vp / 8, rows = kThreads / cols;               // vp <= 2048
+  const int cols = vp / 8, rows = kThreads / cols;               // vp <= 1024
   const int row = tid / cols, col = (tid - row * cols) * 8;
   const bool active = row < rows;
-  const float* scores = p.scores + static_cast<long long>(b) * H * p.n_max;
+  const float* weights = p.scores + (static_cast<long long>(b) * a.H + h0) * p.n_max + r.n0;
   float acc[REP][8];
 #pragma unroll
   for (int x = 0; x < REP; ++x)
 #pragma unroll
     for (int e = 0; e < 8; ++e) acc[x][e] = 0.f;
-  constexpr int kAhead = sizeof(T) == 2 ? 8 : 4;
-  for (int base = 0; base < r.nk; base += kKeys) {
-    const int n = min(kKeys, r.nk - base);
-    Raw8<T> vf[kAhead];
-    // the first values are on their way while the weights are formed
-    auto fetch = [&](int at) {
+  constexpr int kAhead = 4;
+  if (active) {
+    for (int at = row; at < r.nk; at += rows * kAhead) {
+      Raw8<T> vf[kAhead];
+      float w[kAhead][REP];
 #pragma unroll
       for (int u = 0; u < kAhead; ++u) {
         const int k = at + u * rows;
-        if (active && k < n) raw_load(ring_v + static_cast<long long>(r.slot(r.n0 + base + k)) * stride + col, vf[u]);
+        const int kc = min(k, r.nk - 1);                         // past the end: weight zero
+        raw_load(ring_v + static_cast<long long>(r.slot(r.n0 + kc)) * stride + col, vf[u]);
+#pragma unroll
+        for (int x = 0; x < REP; ++x)
+          w[u][x] = k < r.nk && x < nh ? weights[static_cast<long long>(x) * p.n_max + k] : 0.f;
       }
-    };
-    fetch(row);
-    __syncthreads();                                             // statistics written / old weights used up
-    for (int x = tid; x < H * kKeys; x += kThreads) {
-      const int h = x / kKeys, k = x - h * kKeys;
-      if (k < n)
-        sm[L.w + h * (kKeys + 1) + k] =
-            score_exp<T>(scores[static_cast<long long>(h) * p.n_max + r.n0 + base + k] - sm[L.lse + h]) * sm[L.lse + H + h];
-    }
-    __syncthreads();
-    for (int x = tid; x < REP * kKeys; x += kThreads) {
-      const int h = x / kKeys, k = x - h * kKeys;
-      float v = 0.f;
-      if (k < n)
-        for (int g = 0; g < H; ++g) v = fmaf(sm[L.talk + h * H + g], sm[L.w + g * (kKeys + 1) + k], v);
-      sm[L.mix + x] = v;
-    }
-    __syncthreads();
-    for (int at = row; active && at < n; at += rows * kAhead) {
-      if (at != row) fetch(at);
 #pragma unroll
       for (int u = 0; u < kAhead; ++u) {
-        const int k = at + u * rows;
-        if (k < n) {
-          float f[8];
-          raw_unpack(vf[u], f);
+        float f[8];
+        raw_unpack(vf[u], f);
 #pragma unroll
-          for (int x = 0; x < REP; ++x) {
-            const float w = sm[L.mix + x * kKeys + k];
+        for (int x = 0; x < REP; ++x)
 #pragma unroll
-            for (int e = 0; e < 8; ++e) acc[x][e] = fmaf(w, f[e], acc[x][e]);
-          }
-        }
+          for (int e = 0; e < 8; ++e) acc[x][e] = fmaf(w[u][x], f[e], acc[x][e]);
       }
     }
   }
 #pragma unroll
   for (int x = 0; x < REP; ++x)
 #pragma unroll
-    for (int e = 0; e < 8; ++e) sm[L.red + (x * 8 + e) * kThreads + tid] = active ? acc[x][e] : 0.f;
+    for (int e = 0; e < 8; ++e) sm[(x * 8 + e) * kThreads + tid] = acc[x][e];
   __syncthreads();
   for (int idx = tid; idx < REP * vp; idx += kThreads) {
     const int x = idx / vp, d = idx - x * vp;
-    const float* src = sm + L.red + (x * 8 + (d & 7)) * kThreads + (d >> 3);
+    const float* src = sm + (x * 8 + (d & 7)) * kThreads + (d >> 3);
     float v = 0.f;
     for (int y = 0; y < rows; ++y) v += src[y * cols];
-    sm[L.o + idx] = v;
+    s_out[idx] = v;
   }
   if (p.splits > 1) cluster.sync(); else __syncthreads();
   T* out = static_cast<T*>(a.out) + b * a.ldo + static_cast<long long>(h0) * vp;
   for (int idx = split * kThreads + tid; idx < nh * vp; idx += p.splits * kThreads) {
     float v = 0.f;
-    for (int s = 0; s < p.splits; ++s) v += cluster.map_shared_rank(sm + L.o, s)[idx];
+    for (int s = 0; s < p.splits; ++s) v += cluster.map_shared_rank(s_out, s)[idx];
     out[idx] = from_f32<T>(v * a.out_scale);
   }
   if (p.splits > 1) cluster.sync();     // the other blocks read this block's shared memory until here
@@ -365,7 +358,13 @@ cudaError_t launch_both(const DecodeParams& p, cudaStream_t st) {
                   : p.a.dp <= 128 ? launch_scores<T, REP, 2>(p, grid, st)
                                   : launch_scores<T, REP, 4>(p, grid, st);
   if (e != cudaSuccess) return e;
-  const int bytes = values_smem<REP>(p.a.H, p.a.vp).total * static_cast<int>(sizeof(float));
+  const int mix_bytes = p.a.H * (2 + kMixKeys) * static_cast<int>(sizeof(float));
+  e = cudaFuncSetAttribute(window_decode_mix_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, mix_bytes);
+  if (e != cudaSuccess) return e;
+  e = launch_kernel(window_decode_mix_kernel<T>, dim3((p.n_max + kMixKeys - 1) / kMixKeys, p.a.B), dim3(kThreads),
+                    mix_bytes, st, p);
+  if (e != cudaSuccess) return e;
+  const int bytes = values_smem_floats<REP>(p.a.vp) * static_cast<int>(sizeof(float));
   auto kern = window_decode_values_kernel<T, REP>;
   e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, bytes);
   if (e != cudaSuccess) return e;
@@ -398,8 +397,7 @@ cudaError_t launch_typed(const DecodeParams& p, cudaStream_t st) {
 }  // namespace
 
 bool window_decode_supported(const WindowAttnParams& a) {
-  return a.dp <= 256 && a.vp <= 1024 && a.H <= 256 && a.G * ((a.H / a.G + 3) / 4) <= 65535 &&
-         values_smem<4>(a.H, a.vp).total * sizeof(float) <= 227 * 1024;
+  return a.dp <= 256 && a.vp <= 1024 && a.H <= 256 && a.G * ((a.H / a.G + 3) / 4) <= 65535;
 }
 
 size_t window_decode_workspace_bytes(const WindowAttnParams& a) {

@@ -902,7 +902,7 @@ def window_attention_(proj: dict, out: torch.Tensor, weights: dict, ring_k: torc
     ws_bytes = lib.cd_window_attention_decode_workspace_bytes(ref) if seq_len == 1 else 0
     if ws_bytes:
         ws = torch.empty(ws_bytes, dtype=torch.uint8, device=out.device)
-        with _Span("window_attention_decode", 2):
+        with _Span("window_attention_decode", 3):
             _lib.check(lib.cd_window_attention_decode(ref, ws.data_ptr(), ws_bytes, fp32, _stream()),
                        "cd_window_attention_decode")
         return

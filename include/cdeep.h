@@ -430,7 +430,7 @@ typedef struct cd_window_attn {
 
 /* Norms the q and k heads of every row in place. */
 int cd_window_attention_norm(const cd_window_attn* h_args, int fp32, void* stream);
-/* One new token per sequence (S = 1, normed = 0): two kernels that norm q and the new key, write the
+/* One new token per sequence (S = 1, normed = 0): three kernels that norm q and the new key, write the
  * new key and value into the ring and stream the ring once.  The workspace size is 0 where the form
  * does not apply (heads wider than 256). */
 size_t cd_window_attention_decode_workspace_bytes(const cd_window_attn* h_args);
