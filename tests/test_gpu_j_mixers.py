@@ -103,7 +103,9 @@ class Window:
 TOL = {BF: 2.5e-2, F32: 3e-5}
 SHAPES = [  # T, H, G, dim, vdim, size, keep, B
     (70, 4, 2, 32, 48, 20, 3, 2),
-    (130, 8, 4, 64, 80, 50, 6, 1),
+    (130, 8, 2, 64, 112, 50, 7, 1),
+    (96, 8, 8, 128, 128, 40, 3, 1),
+    (83, 16, 8, 128, 128, 37, 2, 2),
     (101, 6, 3, 24, 40, 33, 0, 1),
     (90, 16, 4, 128, 128, 64, 5, 1),
     (75, 5, 1, 40, 112, 19, 40, 1),
@@ -134,14 +136,14 @@ def test_window_attention_whole_portions_and_decode(shape, dtype):
 
 
 @pytest.mark.parametrize("dtype", [BF, F32], ids=["bf16", "fp32"])
-@pytest.mark.parametrize("H,G,dim,vdim,size,keep", [(8, 4, 64, 80, 50, 6), (3, 1, 48, 32, 32, 4)])
+@pytest.mark.parametrize("H,G,dim,vdim,size,keep", [(8, 2, 64, 112, 50, 7), (3, 1, 48, 32, 32, 4), (16, 4, 128, 128, 45, 5)])
 def test_window_edges_show(dtype, H, G, dim, vdim, size, keep):
     """One query looks for one key that stands out by far: just inside and just outside the window,
     the last kept token and the one after it, and the query's own token; as part of a prompt, as a
     decoded token and in a portion of two."""
     T, i = 2 * size + keep + 9, 2 * size + keep + 5
     for j in (i, i - 1, i - size + 1, i - size, keep - 1, keep, 0):
-        w = Window(dtype, T, H, G, dim, vdim, size, keep, seed=j, scale=0.6)
+        w = Window(dtype, T, H, G, dim, vdim, size, keep, seed=j, scale=28.0 / dim)
         w.q *= 0.1
         w.k *= 0.1
         u = np.sign(np.random.default_rng(5).standard_normal(dim))
@@ -228,7 +230,7 @@ class Linear:
 
 LINEAR_TOL = {BF: 1e-2, F32: 1e-4}
 LINEAR_SHAPES = [  # T, H, dk, dv, rank, tau, B
-    (150, 4, 32, 64, 16, 16.0, 1),
+    (150, 6, 48, 64, 16, 12.0, 1),
     (97, 3, 24, 40, 5, 2.0, 2),
     (200, 2, 128, 128, 16, 16.0, 1),
     (130, 5, 16, 96, 24, 1.0, 1),
@@ -282,7 +284,7 @@ def test_linear_attention_remembers_a_far_key():
 
 
 # ------------------------------------------------------------------------------ fp32 stream
-@pytest.mark.parametrize("T,K,N", [(1, 64, 40), (33, 320, 72), (130, 200, 320), (300, 64, 1000), (2300, 512, 768),
+@pytest.mark.parametrize("T,K,N", [(1, 64, 40), (33, 312, 72), (130, 200, 328), (300, 64, 1000), (2300, 512, 768),
                                    (40, 4096, 2048)])
 def test_linear_into_fp32_stream(T, K, N):
     from complexity_deep_b200 import ops
@@ -303,7 +305,7 @@ def test_linear_into_fp32_stream(T, K, N):
     ops.status_fetch()
 
 
-@pytest.mark.parametrize("T,H,I", [(5, 64, 40), (300, 320, 384), (2100, 256, 704)])
+@pytest.mark.parametrize("T,H,I", [(5, 64, 40), (300, 296, 392), (2100, 256, 704)])
 @pytest.mark.parametrize("limit", [0.5, 3.0, 1e30])
 def test_clamped_glu(T, H, I, limit):
     from complexity_deep_b200.core.mlp import ClampedGLU
@@ -322,7 +324,7 @@ def test_clamped_glu(T, H, I, limit):
     ops.status_fetch()
 
 
-@pytest.mark.parametrize("T,W", [(1, 20), (37, 320), (5, 1500), (9, 2304)])
+@pytest.mark.parametrize("T,W", [(1, 20), (37, 328), (5, 1500), (9, 2304)])
 def test_stream_norm_and_embedding(T, W):
     from complexity_deep_b200 import ops
     from complexity_deep_b200.core.normalization import StreamNorm
