@@ -12,7 +12,7 @@ from ctypes import c_char_p, c_float, c_int, c_longlong, c_size_t, c_void_p
 LIB_PATH = os.path.join(os.path.dirname(os.path.abspath(__file__)), "libcdeep.so")
 CHECKS_LIB_PATH = os.path.join(os.path.dirname(os.path.abspath(__file__)), "libcdeep_checks.so")
 
-ABI_VERSION = 3
+ABI_VERSION = 4
 
 
 
@@ -35,7 +35,29 @@ class LinearAttn(ctypes.Structure):
                 + [(n, c_int) for n in ("B", "S", "H", "dk", "dkp", "dv", "dvp", "rank")])
 
 
+class LatentAttn(ctypes.Structure):
+    """cd_latent_attn of include/cdeep.h."""
+    _fields_ = ([(n, c_void_p) for n in ("q", "kv", "gate")] + [("ldp", c_longlong)]
+                + [(n, c_void_p) for n in ("norm_w", "cos_t", "sin_t", "uk", "uk_t", "uv", "cache", "out")]
+                + [("ldo", c_longlong), ("pos_dev", c_void_p)]
+                + [(n, c_float) for n in ("scale", "eps", "out_scale")]
+                + [(n, c_int) for n in ("B", "S", "H", "dim", "dimp", "rot", "rotp", "rank", "rankp", "vdim", "vp",
+                                        "capacity", "positions", "pos0")])
+
+
+class DeltaAttn(ctypes.Structure):
+    """cd_delta_attn of include/cdeep.h."""
+    _fields_ = ([(n, c_void_p) for n in ("q", "k", "v", "b")] + [("ldp", c_longlong), ("zg", c_void_p),
+                                                                 ("ldz", c_longlong)]
+                + [(n, c_void_p) for n in ("taps_w", "rate", "dt_bias", "norm_w", "ring", "state", "out")]
+                + [("ldo", c_longlong)] + [(n, c_void_p) for n in ("act", "inv", "o_raw", "pos_dev")]
+                + [(n, c_float) for n in ("eps", "out_scale")]
+                + [(n, c_int) for n in ("B", "S", "H", "G", "dk", "dkp", "dv", "dvp", "taps", "pos0")])
+
+
 _WINDOW_FN = (c_int, [ctypes.POINTER(WindowAttn), c_int, c_void_p])
+_LATENT_FN = (c_int, [ctypes.POINTER(LatentAttn), c_int, c_void_p])
+_DELTA_FN = (c_int, [ctypes.POINTER(DeltaAttn), c_int, c_void_p])
 _GLA_FN = (c_int, [ctypes.POINTER(LinearAttn), c_int, c_void_p])
 
 # name -> (restype, argtypes); mirrors include/cdeep.h one to one
@@ -108,10 +130,15 @@ SIGNATURES = {
                           c_int, c_int, c_void_p]),
     "cd_embed_rows": (c_int, [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p]),
     "cd_rmsnorm_f32": (c_int, [c_void_p, c_void_p, c_float, c_float, c_void_p, c_int, c_int, c_int, c_int, c_void_p]),
-    "cd_linear_f32out": (c_int, [c_void_p] * 5 + [c_int, c_int, c_int, c_void_p]),
-    "cd_linear_f32": (c_int, [c_void_p] * 5 + [c_int, c_int, c_int, c_void_p]),
-    "cd_glu_up": (c_int, [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_float, c_float,
-                          c_void_p]),
+    "cd_embed_positions": (c_int, [c_void_p] * 4 + [c_int] * 5 + [c_void_p] + [c_int] * 4 + [c_void_p]),
+    "cd_layernorm_f32": (c_int, [c_void_p, c_void_p, c_float, c_void_p, c_int, c_int, c_int, c_int, c_void_p]),
+    "cd_linear_f32out": (c_int, [c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_int, c_int,
+                                 c_int, c_void_p]),
+    "cd_project": (c_int, [c_void_p, c_longlong, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_void_p]),
+    "cd_linear_f32": (c_int, [c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_float, c_int, c_void_p, c_void_p,
+                              c_int, c_int, c_int, c_int, c_void_p]),
+    "cd_glu_up": (c_int, [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_float,
+                          c_float, c_void_p]),
     "cd_glu_f32": (c_int, [c_void_p, c_void_p, c_int, c_int, c_float, c_float, c_float, c_void_p]),
     "cd_window_attention_supported": (c_int, [ctypes.POINTER(WindowAttn)]),
     "cd_window_attention_norm": _WINDOW_FN,
@@ -127,6 +154,15 @@ SIGNATURES = {
     "cd_gla_sequence": _GLA_FN,
     "cd_gla_finish": _GLA_FN,
     "cd_gla_chunk_workspace_bytes": (c_size_t, [ctypes.POINTER(LinearAttn)]),
+    "cd_latent_prepare": _LATENT_FN,
+    "cd_latent_rows": _LATENT_FN,
+    "cd_delta_supported": (c_int, [ctypes.POINTER(DeltaAttn)]),
+    "cd_delta_prepare": _DELTA_FN,
+    "cd_delta_sequence": _DELTA_FN,
+    "cd_delta_finish": _DELTA_FN,
+    "cd_route_top": (c_int, [c_void_p, c_longlong, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p]),
+    "cd_gather_div": (c_int, [c_void_p, c_void_p, c_int, c_void_p, c_longlong, c_int, c_int, c_void_p]),
+    "cd_combine_top": (c_int, [c_void_p, c_void_p, c_void_p, c_int, c_float, c_void_p, c_int, c_int, c_int, c_void_p]),
     "cd_gla_chunk": (c_int, [ctypes.POINTER(LinearAttn), c_void_p, c_size_t, c_void_p]),
 }
 

@@ -1,6 +1,6 @@
 """Dense MLPs on the fused up-projection and down-projection kernels: SwiGLU with the reference's
-parameters (complexity_deep/core/mlp.py:19-40), and the clamped gated unit of designs that keep the
-residual stream in fp32."""
+parameters (complexity_deep/core/mlp.py:19-40), and for designs that keep the residual stream in fp32
+the clamped gated unit and the squared relu."""
 from __future__ import annotations
 
 import torch
@@ -8,7 +8,7 @@ import torch.nn as nn
 
 from .. import ops
 from ._cache import DerivedCache
-from .padding import pad_rows
+from .padding import ROW_ALIGN, pad_rows, round_up
 
 
 class SwiGLU(nn.Module):
@@ -75,10 +75,31 @@ class ClampedGLU(nn.Module):
         return ops.glu_up(x, self._derived.get(f"gate_up_{bn}", src, make), rows, bn, self.alpha,
                           self.limit, self.offset)
 
-    def run(self, x: torch.Tensor, stream: torch.Tensor, layer_scale=None) -> torch.Tensor:
-        """stream += layer_scale * mlp(x), in place; x [T, width padded], stream fp32."""
+    def run(self, x: torch.Tensor, stream: torch.Tensor, layer_scale=None, scale: float = 1.0) -> torch.Tensor:
+        """stream += scale * layer_scale * mlp(x), in place; x [T, width padded], stream fp32."""
         h = self._up(x)
         w = self._derived.get("down", (self.down_proj.weight,), lambda: pad_rows(
             self.down_proj.weight.detach(), stream.shape[1], h.shape[1]).contiguous())
         return ops.linear_to_f32(h, w, residual=stream, col_scale=layer_scale, inplace=True,
-                                 tag="glu_down")
+                                 tag="glu_down", scale=scale)
+
+
+class SquaredReLU(nn.Module):
+    """down_proj(relu(up_proj(x))^2); two bias-free nn.Linear."""
+
+    def __init__(self, hidden_size: int, intermediate_size: int):
+        super().__init__()
+        self.up_proj = nn.Linear(hidden_size, intermediate_size, bias=False)
+        self.down_proj = nn.Linear(intermediate_size, hidden_size, bias=False)
+        self._derived = DerivedCache()
+
+    def run(self, x: torch.Tensor, stream: torch.Tensor, layer_scale=None, scale: float = 1.0) -> torch.Tensor:
+        """stream += scale * layer_scale * mlp(x), in place; x [T, width padded], stream fp32."""
+        rows = round_up(self.up_proj.weight.shape[0], ROW_ALIGN)
+        up = self._derived.get("up", (self.up_proj.weight,), lambda: pad_rows(
+            self.up_proj.weight.detach(), rows, x.shape[1]).contiguous())
+        down = self._derived.get("down", (self.down_proj.weight,), lambda: pad_rows(
+            self.down_proj.weight.detach(), stream.shape[1], rows).contiguous())
+        h = ops.project(x, up, tag="relu2_up", act="relu2")
+        return ops.linear_to_f32(h, down, residual=stream, col_scale=layer_scale, inplace=True,
+                                 tag="relu2_down", scale=scale)

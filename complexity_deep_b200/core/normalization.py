@@ -28,11 +28,14 @@ class RMSNorm(nn.Module):
 
 class StreamNorm(nn.Module):
     """RMSNorm of the fp32 residual stream into the weights' dtype:
-    y = x / sqrt(mean(x^2) + eps) * (offset + weight); offset 1 for a weight stored around zero."""
+    y = x / sqrt(mean(x^2) + eps) * (offset + weight); offset 1 for a weight stored around zero.
+    centred: layer norm without a bias, the same of x - mean(x)."""
 
-    def __init__(self, hidden_size: int, eps: float, offset: float = 0.0):
+    def __init__(self, hidden_size: int, eps: float, offset: float = 0.0, centred: bool = False):
         super().__init__()
-        self.eps, self.offset = eps, offset
+        if centred and offset:
+            raise ValueError("a centred norm has a plain weight")
+        self.eps, self.offset, self.centred = eps, offset, centred
         self.weight = nn.Parameter(torch.full((hidden_size,), 1.0 - offset))
         self._derived = DerivedCache()
 
@@ -40,7 +43,9 @@ class StreamNorm(nn.Module):
         """stream [T, width padded] fp32 -> [T, width padded]; the padding stays zero."""
         w = self._derived.get("weight", (self.weight,),
                               lambda: pad_vector(self.weight.detach(), stream.shape[1]))
+        if self.centred:
+            return ops.layernorm_f32(stream, w, self.eps, width=self.weight.numel())
         return ops.rmsnorm_f32(stream, w, self.eps, self.offset, width=self.weight.numel())
 
     def extra_repr(self) -> str:
-        return f"{self.weight.numel()}, eps={self.eps}, offset={self.offset}"
+        return f"{self.weight.numel()}, eps={self.eps}, offset={self.offset}, centred={self.centred}"

@@ -51,6 +51,16 @@ class RotaryEmbedding(nn.Module):
         return self.cos_cached, self.sin_cached
 
 
+def interleaved_tables(positions: int, dims: int, width: int, base: float, device) -> Tuple[torch.Tensor, torch.Tensor]:
+    """fp32 cos / sin [positions, width / 2] of position * base^(-2i / dims) for the pairs
+    (2i, 2i + 1) of a vector of `width` elements; pairs beyond the first `dims` elements do not turn.
+    Angles are evaluated in 64 bits and the results rounded once."""
+    freq = torch.zeros(width // 2, dtype=torch.float64, device=device)
+    freq[: dims // 2] = base ** (-torch.arange(0, dims, 2, dtype=torch.float64, device=device) / dims)
+    angles = torch.outer(torch.arange(positions, dtype=torch.float64, device=device), freq)
+    return angles.cos().float().contiguous(), angles.sin().float().contiguous()
+
+
 def rotate_half(x: torch.Tensor) -> torch.Tensor:
     half = x.shape[-1] // 2
     return torch.cat([-x[..., half:], x[..., :half]], dim=-1)

@@ -1,5 +1,6 @@
-"""Per-sequence state of decoders whose memory does not grow with the sequence: rings of keys and
-values for window attention, fp32 matrices for recurrences.
+"""Per-sequence state of decoders that mix several kinds of layer: rings of keys and values for window
+attention, fp32 matrices for recurrences, rings of inputs for short convolutions, and latent rows that
+grow with the sequence.
 
 ``StaticKVCache`` (core.attention) keeps every cached token; here each mixer of a layer declares
 what it carries from call to call (``new_state``), ``DecoderState`` holds one such state per mixer
@@ -43,6 +44,51 @@ class RecurrentState:
 
     def copy_(self, other: "RecurrentState") -> None:
         self.s.copy_(other.s)
+
+
+class DeltaState(RecurrentState):
+    """A recurrence's matrices together with the last inputs of the short convolution ahead of it:
+    position p in slot ``p % taps``.  Slots of positions before 0 are never read."""
+
+    def __init__(self, batch: int, heads: int, rows: int, cols: int, taps: int, channels: int, device,
+                 dtype) -> None:
+        super().__init__(batch, heads, rows, cols, device)
+        self.ring = torch.zeros(batch, taps, channels, dtype=dtype, device=device)
+
+    def copy_(self, other: "DeltaState") -> None:
+        super().copy_(other)
+        self.ring.copy_(other.ring)
+
+
+class LatentState:
+    """One row per cached token, shared by all heads: [batch, capacity, width].  The buffer grows by
+    doubling up to `limit` rows; with a given capacity it is fixed (captured steps keep its address).
+    Rows beyond the sequence's length are never read."""
+
+    def __init__(self, batch: int, width: int, limit: int, device, dtype, capacity: Optional[int] = None) -> None:
+        self.limit, self.fixed = limit, capacity is not None
+        self.rows = torch.zeros(batch, min(capacity or 256, limit), width, dtype=dtype, device=device)
+
+    def reserve(self, tokens: int) -> torch.Tensor:
+        """The buffer, with room for `tokens` rows per sequence."""
+        have = self.rows.shape[1]
+        if tokens > have:
+            if self.fixed or tokens > self.limit:
+                raise RuntimeError(f"{tokens} tokens do not fit a cache of {have if self.fixed else self.limit}")
+            grown = self.rows.new_zeros(self.rows.shape[0], min(max(tokens, 2 * have), self.limit), self.rows.shape[2])
+            grown[:, :have] = self.rows
+            self.rows = grown
+        return self.rows
+
+    def reset(self) -> None:
+        pass
+
+    def copy_(self, other: "LatentState") -> None:
+        n = other.rows.shape[1]
+        if not self.fixed:
+            self.reserve(n)
+        n = min(n, self.rows.shape[1])
+        self.rows[:, :n] = other.rows[:, :n]
 
 
 class DecoderState:

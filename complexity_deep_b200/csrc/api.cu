@@ -21,7 +21,7 @@ static inline bool aligned16(const void* p) { return (reinterpret_cast<uintptr_t
 
 extern "C" {
 
-int cd_version(void) { return 3; }
+int cd_version(void) { return 4; }
 
 const char* cd_error_string(int status) {
   switch (status) {
@@ -563,20 +563,40 @@ int cd_embed_rows(const int64_t* ids, const void* table, float* x, int T, int V,
   return e == cudaSuccess ? CD_OK : cuda_fail(e, "embed_rows launch");
 }
 
-int cd_rmsnorm_f32(const float* x, const void* w, float eps, float offset, void* out, int T, int W, int ldx,
-                   int fp32, void* stream) {
+int cd_embed_positions(const int64_t* ids, const void* table, const void* pos, float* x, int T, int V, int P, int S,
+                       int pos0, const int32_t* pos_dev, int W, int ldw, int ldx, int fp32, void* stream) {
+  if (T < 0 || V < 1 || P < 1 || S < 1 || W < 1 || ldw < W || ldx < W || (ldx & 7) || !table || !pos)
+    return CD_ERR_INVALID;
+  if (T > 0 && (!ids || !x || !aligned16(x))) return CD_ERR_INVALID;
+  cudaError_t e = launch_embed_rows(reinterpret_cast<const long long*>(ids), table, x, T, V, W, ldw, ldx, fp32,
+                                    as_stream(stream), pos, P, S, pos0, pos_dev);
+  return e == cudaSuccess ? CD_OK : cuda_fail(e, "embed_positions launch");
+}
+
+static int norm_f32(const float* x, const void* w, float eps, float offset, void* out, int T, int W, int ldx, int fp32,
+                    void* stream, bool centred) {
   if (T < 0 || W < 1 || ldx < W || (ldx & 7) || !w || !aligned16(w)) return CD_ERR_INVALID;
   if (T > 0 && (!x || !out || !aligned16(x) || !aligned16(out))) return CD_ERR_INVALID;
-  cudaError_t e = launch_rmsnorm_f32(x, w, eps, offset, out, T, W, ldx, fp32, as_stream(stream));
+  cudaError_t e = launch_rmsnorm_f32(x, w, eps, offset, out, T, W, ldx, fp32, as_stream(stream), centred);
   return e == cudaSuccess ? CD_OK : cuda_fail(e, "rmsnorm_f32 launch");
 }
 
-int cd_linear_f32out(const void* x, const void* w, const float* residual, const void* col_scale, float* out,
-                     int T, int K, int N, void* stream) {
-  if (T < 0 || K < 8 || (K & 7) || N < 8 || (N & 7)) return CD_ERR_INVALID;
+int cd_rmsnorm_f32(const float* x, const void* w, float eps, float offset, void* out, int T, int W, int ldx,
+                   int fp32, void* stream) {
+  return norm_f32(x, w, eps, offset, out, T, W, ldx, fp32, stream, false);
+}
+
+int cd_layernorm_f32(const float* x, const void* w, float eps, void* out, int T, int W, int ldx, int fp32,
+                     void* stream) {
+  return norm_f32(x, w, eps, 0.f, out, T, W, ldx, fp32, stream, true);
+}
+
+int cd_linear_f32out(const void* x, int64_t ldx, const void* w, const float* residual, const void* col_scale,
+                     float scale, float* out, int T, int K, int N, void* stream) {
+  if (T < 0 || K < 8 || (K & 7) || N < 8 || (N & 7) || ldx < K) return CD_ERR_INVALID;
   GemmOperand op0{};
   op0.a = x;
-  op0.lda = K;
+  op0.lda = ldx;
   op0.b = w;
   op0.ldb = K;
   op0.b_rows = N;
@@ -589,21 +609,45 @@ int cd_linear_f32out(const void* x, const void* w, const float* residual, const 
   epi.residual = residual;
   epi.ldr = N;
   epi.col_scale = col_scale;
+  epi.acc_scale = scale;
   return launch_gemm(T, N, 1, nullptr, op0, nullptr, epi, choose_store_block_n(T, N, 1, current_sm_count()),
                      as_stream(stream));
 }
 
-int cd_linear_f32(const float* x, const float* w, const float* residual, const float* col_scale, float* out, int T,
-                  int K, int N, void* stream) {
-  if (T < 0 || K < 4 || (K & 3) || N < 1) return CD_ERR_INVALID;
+int cd_project(const void* x, int64_t ldx, const void* w, int act, void* out, int T, int K, int N, void* stream) {
+  if (T < 0 || K < 8 || (K & 7) || N < 8 || (N & 7) || ldx < K || act < 0 || act > 1) return CD_ERR_INVALID;
+  GemmOperand op0{};
+  op0.a = x;
+  op0.lda = ldx;
+  op0.b = w;
+  op0.ldb = K;
+  op0.b_rows = N;
+  op0.K = K;
+  GemmEpilogueArgs epi{};
+  epi.kind = kEpiStore;
+  epi.out = out;
+  epi.ldo = N;
+  epi.out_cols = N;
+  epi.act = act;
+  return launch_gemm(T, N, 1, nullptr, op0, nullptr, epi, choose_store_block_n(T, N, 1, current_sm_count()),
+                     as_stream(stream));
+}
+
+int cd_linear_f32(const float* x, int64_t ldx, const float* w, const float* residual, const float* col_scale,
+                  float scale, int act, float* out, const int32_t* seg_offsets, int groups, int T, int K, int N,
+                  void* stream) {
+  if (T < 0 || K < 4 || (K & 3) || N < 1 || ldx < K || (ldx & 3) || act < 0 || act > 1 || groups < 1 || groups > 65535 ||
+      (groups > 1 && !seg_offsets))
+    return CD_ERR_INVALID;
   if (T > 0 && (!x || !w || !out || !aligned16(x) || !aligned16(w))) return CD_ERR_INVALID;
-  cudaError_t e = launch_linear_f32(x, w, residual, col_scale, out, T, K, N, as_stream(stream));
+  cudaError_t e = launch_linear_f32(x, ldx, w, residual, col_scale, scale, act, out, seg_offsets, groups, T, K, N,
+                                    as_stream(stream));
   return e == cudaSuccess ? CD_OK : cuda_fail(e, "linear_f32 launch");
 }
 
-int cd_glu_up(const void* x, const void* packed_w, void* h, int T, int H, int I, int block_n, float alpha,
-              float limit, float offset, void* stream) {
-  if (T < 0 || H < 8 || I < 8 || (H & 7) || (I & 7)) return CD_ERR_INVALID;
+int cd_glu_up(const void* x, const int32_t* seg_offsets, int groups, const void* packed_w, void* h, int T, int H, int I,
+              int block_n, float alpha, float limit, float offset, void* stream) {
+  if (T < 0 || H < 8 || I < 8 || (H & 7) || (I & 7) || groups < 1) return CD_ERR_INVALID;
   const int rows = cd_gate_up_packed_rows(I, block_n);
   if (rows == 0) return CD_ERR_INVALID;
   GemmOperand op{};
@@ -611,7 +655,8 @@ int cd_glu_up(const void* x, const void* packed_w, void* h, int T, int H, int I,
   op.lda = H;
   op.b = packed_w;
   op.ldb = H;
-  op.b_rows = rows;
+  op.b_rows = static_cast<long long>(groups) * rows;
+  op.b_group_rows = rows;
   op.K = H;
   GemmEpilogueArgs epi{};
   epi.kind = kEpiGlu;
@@ -621,7 +666,7 @@ int cd_glu_up(const void* x, const void* packed_w, void* h, int T, int H, int I,
   epi.glu_alpha = alpha;
   epi.glu_limit = limit;
   epi.glu_offset = offset;
-  return launch_gemm(T, rows, 1, nullptr, op, nullptr, epi, block_n, as_stream(stream));
+  return launch_gemm(T, rows, groups, seg_offsets, op, nullptr, epi, block_n, as_stream(stream));
 }
 
 int cd_glu_f32(const float* gu, float* h, int T, int I, float alpha, float limit, float offset, void* stream) {
@@ -749,6 +794,100 @@ int cd_gla_chunk(const cd_linear_attn* a, void* ws, size_t ws_bytes, void* strea
   if (!a->log_decay || !ws || !aligned16(ws) || ws_bytes < gla_chunk_workspace_bytes(*a)) return CD_ERR_INVALID;
   cudaError_t e = launch_gla_chunk(*a, ws, as_stream(stream));
   return e == cudaSuccess ? CD_OK : cuda_fail(e, "gla chunk launch");
+}
+
+static int latent_args_ok(const cd_latent_attn* a) {
+  if (!a || a->B < 0 || a->S < 0 || a->B > 65535 || a->H < 1 || a->dim < 1 || a->rank < 1 || a->vdim < 1 || a->rot < 2 ||
+      a->dimp < a->dim || a->rotp < a->rot || a->rankp < a->rank || a->vp < a->vdim || (a->dimp & 15) || (a->rotp & 15) ||
+      (a->rankp & 15) || (a->vp & 15) || (a->ldp & 7) || (a->ldo & 7) || a->pos0 < 0 || a->capacity < 1 ||
+      a->positions < 1)
+    return CD_ERR_INVALID;
+  if (!a->pos_dev && (a->pos0 + a->S > a->capacity || a->pos0 + a->S > a->positions)) return CD_ERR_INVALID;
+  if (!a->q || !a->kv || !a->gate || !a->norm_w || !a->cos_t || !a->sin_t || !a->uk || !a->uk_t || !a->uv || !a->cache ||
+      !a->out || !aligned16(a->q) || !aligned16(a->kv) || !aligned16(a->gate) || !aligned16(a->norm_w) ||
+      !aligned16(a->cos_t) || !aligned16(a->sin_t) || !aligned16(a->uk) || !aligned16(a->uk_t) || !aligned16(a->uv) ||
+      !aligned16(a->cache) || !aligned16(a->out))
+    return CD_ERR_INVALID;
+  return CD_OK;
+}
+
+int cd_latent_prepare(const cd_latent_attn* a, int fp32, void* stream) {
+  if (latent_args_ok(a) != CD_OK) return CD_ERR_INVALID;
+  cudaError_t e = launch_latent_prepare(*a, fp32, as_stream(stream));
+  return e == cudaSuccess ? CD_OK : cuda_fail(e, "latent prepare launch");
+}
+
+int cd_latent_rows(const cd_latent_attn* a, int fp32, void* stream) {
+  if (latent_args_ok(a) != CD_OK) return CD_ERR_INVALID;
+  if (!latent_rows_supported(*a)) return CD_ERR_UNSUPPORTED;
+  cudaError_t e = launch_latent_rows(*a, fp32, as_stream(stream));
+  return e == cudaSuccess ? CD_OK : cuda_fail(e, "latent rows launch");
+}
+
+static int delta_args_ok(const cd_delta_attn* a) {
+  if (!a || a->B < 0 || a->S < 0 || a->B > 65535 || a->H < 1 || a->H > 65535 || a->G < 1 || a->H % a->G || a->dk < 1 ||
+      a->dv < 1 || a->dkp < a->dk || a->dvp < a->dv || (a->dkp & 15) || (a->dvp & 15) || a->taps < 1 || (a->ldp & 7) ||
+      (a->ldo & 7) || (a->ldz & 3) || a->pos0 < 0)
+    return CD_ERR_INVALID;
+  if (!a->q || !a->k || !a->v || !a->b || !a->zg || !a->taps_w || !a->rate || !a->dt_bias || !a->norm_w || !a->ring ||
+      !a->state || !a->out || !aligned16(a->q) || !aligned16(a->k) || !aligned16(a->v) || !aligned16(a->zg) ||
+      !aligned16(a->taps_w) || !aligned16(a->dt_bias) || !aligned16(a->norm_w) || !aligned16(a->ring) ||
+      !aligned16(a->state) || !aligned16(a->out) || !aligned16(a->act) || !aligned16(a->o_raw))
+    return CD_ERR_INVALID;
+  return delta_supported(*a) ? CD_OK : CD_ERR_UNSUPPORTED;
+}
+
+int cd_delta_supported(const cd_delta_attn* a) { return a && delta_supported(*a) ? 1 : 0; }
+
+int cd_delta_prepare(const cd_delta_attn* a, int fp32, void* stream) {
+  const int st = delta_args_ok(a);
+  if (st != CD_OK) return st;
+  if (!a->act || !a->inv) return CD_ERR_INVALID;
+  cudaError_t e = launch_delta_prepare(*a, fp32, as_stream(stream));
+  return e == cudaSuccess ? CD_OK : cuda_fail(e, "delta prepare launch");
+}
+
+int cd_delta_sequence(const cd_delta_attn* a, int fp32, void* stream) {
+  const int st = delta_args_ok(a);
+  if (st != CD_OK) return st;
+  if (!a->act || !a->inv || !a->o_raw) return CD_ERR_INVALID;
+  cudaError_t e = launch_delta_sequence(*a, fp32, as_stream(stream));
+  return e == cudaSuccess ? CD_OK : cuda_fail(e, "delta sequence launch");
+}
+
+int cd_delta_finish(const cd_delta_attn* a, int fp32, void* stream) {
+  const int st = delta_args_ok(a);
+  if (st != CD_OK) return st;
+  if (!a->o_raw) return CD_ERR_INVALID;
+  cudaError_t e = launch_delta_finish(*a, fp32, as_stream(stream));
+  return e == cudaSuccess ? CD_OK : cuda_fail(e, "delta finish launch");
+}
+
+int cd_route_top(const float* logits, int64_t ld, int T, int E, int count, int keep, int top, int64_t* ids,
+                 float* weights, void* stream) {
+  if (T < 0 || E < 1 || E > kMaxGroups || count < 1 || E % count || keep < 1 || keep > count || top < 1 ||
+      top > keep * (E / count) || ld < E || (T > 0 && (!logits || !ids || !weights)))
+    return CD_ERR_INVALID;
+  cudaError_t e = launch_route_top(logits, ld, T, E, count, keep, top, reinterpret_cast<long long*>(ids), weights,
+                                   as_stream(stream));
+  return e == cudaSuccess ? CD_OK : cuda_fail(e, "route_top launch");
+}
+
+int cd_gather_div(const void* x, const int32_t* perm, int div, void* out, int64_t n, int rows, int row_bytes,
+                  void* stream) {
+  if (n < 0 || div < 1 || rows < 0 || row_bytes < 16 || (row_bytes & 15)) return CD_ERR_INVALID;
+  if (n > 0 && (!x || !perm || !out || rows < 1 || !aligned16(x) || !aligned16(out))) return CD_ERR_INVALID;
+  cudaError_t e = launch_gather_div(x, perm, div, out, n, rows, row_bytes, as_stream(stream));
+  return e == cudaSuccess ? CD_OK : cuda_fail(e, "gather_div launch");
+}
+
+int cd_combine_top(const void* y, const int32_t* inv_perm, const float* weights, int top, float scale,
+                   float* stream_rows, int T, int ldx, int fp32, void* stream) {
+  if (T < 0 || top < 1 || ldx < 8 || (ldx & 7)) return CD_ERR_INVALID;
+  if (T > 0 && (!y || !inv_perm || !weights || !stream_rows || !aligned16(y) || !aligned16(stream_rows)))
+    return CD_ERR_INVALID;
+  cudaError_t e = launch_combine_top(y, inv_perm, weights, top, scale, stream_rows, T, ldx, fp32, as_stream(stream));
+  return e == cudaSuccess ? CD_OK : cuda_fail(e, "combine_top launch");
 }
 
 }  // extern "C"

@@ -1,0 +1,231 @@
+// Delta rule with one decay per key channel: convolution and norms ahead of the recurrence, the
+// token-by-token recurrence (any storage type), and the head norm and gate behind it.
+#include "delta_rule.cuh"
+#include "kernels.h"
+
+namespace cdeep {
+
+namespace {
+
+constexpr int kThreads = 256;
+
+// ---------------------------------------------------------------- convolution, silu, norms
+// A warp takes `run` tokens of one head of q, k or v; a lane owns eight channels at a time.  The warp
+// of the first run also moves the last inputs of the call into the ring, after it has read the earlier
+// ones (run >= taps - 1: nobody else reads the ring).
+template <typename T>
+__global__ void __launch_bounds__(kThreads)
+delta_prepare_kernel(const DeltaParams p, int run) {
+  pdl_enter();
+  const int lane = threadIdx.x & 31;
+  const int slots = 2 * p.G + p.H, C = delta_channels(p);
+  const int item = blockIdx.x * (kThreads / 32) + (threadIdx.x >> 5), b = blockIdx.y;
+  const int slot = item % slots, t0 = item / slots * run;
+  if (t0 >= p.S) return;
+  const bool is_v = slot >= 2 * p.G;
+  const int width = is_v ? p.dvp : p.dkp;
+  const int col = is_v ? 2 * p.G * p.dkp + (slot - 2 * p.G) * p.dvp : slot * p.dkp;
+  const T* src = static_cast<const T*>(is_v ? p.v : slot < p.G ? p.q : p.k) +
+                 (is_v ? (slot - 2 * p.G) * p.dvp : (slot < p.G ? slot : slot - p.G) * p.dkp);
+  const long long row0 = static_cast<long long>(b) * p.S;
+  const T* taps = static_cast<const T*>(p.taps_w) + col;
+  T* ring = static_cast<T*>(p.ring) + static_cast<long long>(b) * p.taps * C + col;
+  T* act = static_cast<T*>(p.act) + col;
+  const int pos0 = first_position(p);
+  const float scale = slot < p.G ? 1.0f / sqrtf(static_cast<float>(p.dk)) : 1.0f;
+  for (int t = t0; t < min(t0 + run, p.S); ++t) {
+    float ss = 0.f;
+    for (int c = lane * 8; c < width; c += 256) {
+      float y[8] = {};
+      for (int j = p.taps - 1; j >= 0; --j) {              // j tokens back
+        const int pos = pos0 + t - j;
+        if (pos < 0) continue;
+        float x[8], w[8];
+        if (t - j >= 0) load8(src + (row0 + t - j) * p.ldp + c, x);
+        else load8(ring + static_cast<long long>(pos % p.taps) * C + c, x);
+        load8(taps + static_cast<long long>(p.taps - 1 - j) * C + c, w);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) y[e] = fmaf(w[e], x[e], y[e]);
+      }
+#pragma unroll
+      for (int e = 0; e < 8; ++e) {
+        y[e] = to_f32(from_f32<T>(silu_precise(y[e])));
+        ss += y[e] * y[e];
+      }
+      store8(act + (row0 + t) * C + c, y);
+    }
+    if (!is_v) {
+      ss = warp_add(ss);
+      if (lane == 0) p.inv[(row0 + t) * 2 * p.G + slot] = scale / sqrtf(ss + 1e-6f);
+    }
+  }
+  if (t0 == 0)
+    for (int t = max(0, p.S - p.taps); t < p.S; ++t)
+      for (int c = lane * 8; c < width; c += 256) {
+        float x[8];
+        load8(src + (row0 + t) * p.ldp + c, x);
+        store8(ring + static_cast<long long>((pos0 + t) % p.taps) * C + c, x);
+      }
+}
+
+// ---------------------------------------------------------------- token by token
+constexpr int kSteps = 16;     // tokens staged in shared memory at a time
+constexpr int kCols = 32;      // state columns per block, four per warp
+
+// A lane owns M rows (lane % 8, + 8, ...) of one column of the state (dkp <= 8 M).
+template <typename T, int M>
+__global__ void __launch_bounds__(kThreads)
+delta_sequence_kernel(const DeltaParams p) {
+  extern __shared__ float sm[];
+  pdl_enter();
+  const int h = blockIdx.y, b = blockIdx.z, g = h / (p.H / p.G);
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int dkp = p.dkp, dvp = p.dvp, C = delta_channels(p);
+  float* sq = sm;                          // [kSteps][dkp]
+  float* sk = sq + kSteps * dkp;
+  float* sa = sk + kSteps * dkp;           // decays
+  float* sv = sa + kSteps * dkp;           // [kSteps][kCols]
+  float* sb = sv + kSteps * kCols;         // [kSteps] beta
+  float* sx = sb + kSteps;                 // [kSteps] k . q
+  const int cl = warp * 4 + (lane >> 3), r0 = lane & 7, col = blockIdx.x * kCols + cl;
+  const bool col_ok = col < dvp;
+  float* S = p.state + (static_cast<long long>(b) * p.H + h) * dkp * dvp + col;
+  float s[M];
+#pragma unroll
+  for (int m = 0; m < M; ++m) {
+    const int r = r0 + 8 * m;
+    s[m] = (r < dkp && col_ok) ? S[static_cast<long long>(r) * dvp] : 0.f;
+  }
+  const long long row0 = static_cast<long long>(b) * p.S;
+  const float rate = p.rate[h];
+  for (int t0 = 0; t0 < p.S; t0 += kSteps) {
+    const int n = min(kSteps, p.S - t0);
+    for (int idx = tid; idx < n * dkp; idx += kThreads) {
+      const int t = idx / dkp, c = idx - t * dkp;
+      const long long row = row0 + t0 + t;
+      const T* act = static_cast<const T*>(p.act) + row * C;
+      const float* inv = p.inv + row * 2 * p.G;
+      sq[idx] = to_f32(act[g * dkp + c]) * inv[g];
+      sk[idx] = to_f32(act[(p.G + g) * dkp + c]) * inv[p.G + g];
+      sa[idx] = expf(-rate * softplus_precise(p.zg[row * p.ldz + h * dkp + c] + p.dt_bias[h * dkp + c]));
+    }
+    for (int idx = tid; idx < n * kCols; idx += kThreads) {
+      const int t = idx / kCols, c = blockIdx.x * kCols + idx - t * kCols;
+      sv[idx] = c < dvp ? to_f32(static_cast<const T*>(p.act)[(row0 + t0 + t) * C + 2 * p.G * dkp + h * dvp + c]) : 0.f;
+    }
+    for (int t = tid; t < n; t += kThreads)
+      sb[t] = sigmoid_precise(to_f32(static_cast<const T*>(p.b)[(row0 + t0 + t) * p.ldp + h]));
+    __syncthreads();
+    for (int t = warp; t < n; t += kThreads / 32) {
+      float x = 0.f;
+      for (int c = lane; c < dkp; c += 32) x += sk[t * dkp + c] * sq[t * dkp + c];
+      x = warp_add(x);
+      if (lane == 0) sx[t] = x;
+    }
+    __syncthreads();
+    for (int t = 0; t < n; ++t) {
+      float a = 0.f, o = 0.f;
+#pragma unroll
+      for (int m = 0; m < M; ++m) {
+        const int r = r0 + 8 * m;
+        if (r < dkp) {
+          s[m] *= sa[t * dkp + r];
+          a = fmaf(s[m], sk[t * dkp + r], a);
+          o = fmaf(s[m], sq[t * dkp + r], o);
+        }
+      }
+#pragma unroll
+      for (int d = 1; d < 8; d <<= 1) {
+        a += __shfl_xor_sync(0xffffffffu, a, d);
+        o += __shfl_xor_sync(0xffffffffu, o, d);
+      }
+      const float u = sb[t] * (sv[t * kCols + cl] - a);
+#pragma unroll
+      for (int m = 0; m < M; ++m) {
+        const int r = r0 + 8 * m;
+        if (r < dkp) s[m] = fmaf(sk[t * dkp + r], u, s[m]);
+      }
+      if (r0 == 0 && col_ok)
+        p.o_raw[(row0 + t0 + t) * (p.H * dvp) + static_cast<long long>(h) * dvp + col] = fmaf(sx[t], u, o);
+    }
+    __syncthreads();
+  }
+#pragma unroll
+  for (int m = 0; m < M; ++m) {
+    const int r = r0 + 8 * m;
+    if (r < dkp && col_ok) S[static_cast<long long>(r) * dvp] = s[m];
+  }
+}
+
+// ---------------------------------------------------------------- head norm and gate
+// one warp per (row, head)
+template <typename T>
+__global__ void __launch_bounds__(kThreads)
+delta_finish_kernel(const DeltaParams p) {
+  pdl_enter();
+  const long long item = blockIdx.x * 8ll + (threadIdx.x >> 5);
+  if (item >= static_cast<long long>(p.B) * p.S * p.H) return;
+  const int lane = threadIdx.x & 31;
+  const long long row = item / p.H;
+  const int h = static_cast<int>(item - row * p.H);
+  const float* o = p.o_raw + item * p.dvp;
+  const float* gate = p.zg + row * p.ldz + p.H * p.dkp + static_cast<long long>(h) * p.dvp;
+  T* out = static_cast<T*>(p.out) + row * p.ldo + static_cast<long long>(h) * p.dvp;
+  float ss = 0.f;
+  for (int c = lane; c < p.dvp; c += 32) ss += o[c] * o[c];
+  const float r = 1.0f / sqrtf(warp_add(ss) / static_cast<float>(p.dv) + p.eps);
+  for (int c = lane; c < p.dvp; c += 32)
+    out[c] = from_f32<T>(o[c] * r * to_f32(static_cast<const T*>(p.norm_w)[c]) * sigmoid_precise(gate[c]) * p.out_scale);
+}
+
+template <typename T>
+cudaError_t launch_prepare(const DeltaParams& p, cudaStream_t st) {
+  const int run = p.taps > 9 ? p.taps - 1 : 8;
+  const long long items = static_cast<long long>((p.S + run - 1) / run) * (2 * p.G + p.H);
+  return launch_kernel(delta_prepare_kernel<T>, dim3(static_cast<unsigned>((items + 7) / 8), p.B), dim3(kThreads), 0, st,
+                       p, run);
+}
+
+template <typename T, int M>
+cudaError_t launch_sequence_m(const DeltaParams& p, cudaStream_t st) {
+  const size_t bytes = (3 * kSteps * p.dkp + kSteps * kCols + 2 * kSteps) * sizeof(float);
+  cudaError_t e = cudaFuncSetAttribute(delta_sequence_kernel<T, M>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                       static_cast<int>(bytes));
+  if (e != cudaSuccess) return e;
+  return launch_kernel(delta_sequence_kernel<T, M>, dim3((p.dvp + kCols - 1) / kCols, p.H, p.B), dim3(kThreads), bytes,
+                       st, p);
+}
+
+template <typename T>
+cudaError_t launch_sequence(const DeltaParams& p, cudaStream_t st) {
+  if (p.dkp <= 32) return launch_sequence_m<T, 4>(p, st);
+  if (p.dkp <= 64) return launch_sequence_m<T, 8>(p, st);
+  if (p.dkp <= 128) return launch_sequence_m<T, 16>(p, st);
+  if (p.dkp <= 256) return launch_sequence_m<T, 32>(p, st);
+  if (p.dkp <= 512) return launch_sequence_m<T, 64>(p, st);
+  return cudaErrorInvalidValue;
+}
+
+}  // namespace
+
+bool delta_supported(const DeltaParams& p) { return p.dkp <= 512 && p.B <= 65535; }
+
+cudaError_t launch_delta_prepare(const DeltaParams& p, int fp32, cudaStream_t st) {
+  if (p.B == 0 || p.S == 0) return cudaSuccess;
+  return fp32 ? launch_prepare<float>(p, st) : launch_prepare<bf16>(p, st);
+}
+
+cudaError_t launch_delta_sequence(const DeltaParams& p, int fp32, cudaStream_t st) {
+  if (p.B == 0 || p.S == 0) return cudaSuccess;
+  return fp32 ? launch_sequence<float>(p, st) : launch_sequence<bf16>(p, st);
+}
+
+cudaError_t launch_delta_finish(const DeltaParams& p, int fp32, cudaStream_t st) {
+  const long long items = static_cast<long long>(p.B) * p.S * p.H;
+  if (items == 0) return cudaSuccess;
+  const dim3 grid(static_cast<unsigned>((items + 7) / 8));
+  return fp32 ? launch_kernel(delta_finish_kernel<float>, grid, dim3(kThreads), 0, st, p)
+              : launch_kernel(delta_finish_kernel<bf16>, grid, dim3(kThreads), 0, st, p);
+}
+
+}  // namespace cdeep

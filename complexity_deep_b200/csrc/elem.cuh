@@ -97,6 +97,7 @@ template <typename T> __device__ __forceinline__ float score_log1p(float x) {
   return sizeof(T) == 2 ? 0.6931471805599453f * log2_approx(1.0f + x) : log1pf(x);
 }
 
+__device__ __forceinline__ float sigmoid_precise(float z) { return 1.0f / (1.0f + expf(-z)); }
 __device__ __forceinline__ float silu_precise(float g) { return g / (1.0f + expf(-g)); }
 
 }  // namespace cdeep

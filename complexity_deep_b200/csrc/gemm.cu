@@ -503,6 +503,8 @@ int launch_gemm(int M, int N, int num_groups, const int* seg_offsets, const Gemm
   p.clamp_lo = epi.clamp_lo;
   p.clamp_hi = epi.clamp_hi;
   p.col_scale = static_cast<const __nv_bfloat16*>(epi.col_scale);
+  p.acc_scale = epi.acc_scale;
+  p.act = epi.act;
   p.glu_alpha = epi.glu_alpha;
   p.glu_limit = epi.glu_limit;
   p.glu_offset = epi.glu_offset;

@@ -50,7 +50,7 @@ enum GemmEpilogue : int {
   kEpiStoreRope = 2,  // store with per-head RMSNorm + rotary embedding (256-wide tiles only)
   kEpiStoreSplit = 3, // store of a split-bf16 value: out = bf16(v), out_lo = bf16(v - out); the
                       // residual may be split the same way (residual + residual_lo)
-  kEpiStoreF32 = 4,   // fp32 store: out[r, n] = residual[r, n] + col_scale[n] * acc (residual fp32, may be out)
+  kEpiStoreF32 = 4,   // fp32 store: out[r, n] = residual[r, n] + acc_scale * col_scale[n] * acc (residual fp32, may be out)
   kEpiGlu = 5,        // out[r, j] = g * sigmoid(alpha g) * (u + offset), g = min(gate, limit),
                       // u = clamp(up, -limit, limit)
 };
@@ -108,6 +108,8 @@ struct GemmParams {
   int do_clamp;            // clamp the result to [clamp_lo, clamp_hi]
   float clamp_lo, clamp_hi;
   const __nv_bfloat16* col_scale;  // kEpiStoreF32: factor per output column (nullptr = 1)
+  float acc_scale;         // kEpiStoreF32: factor of the accumulator
+  int act;                 // kEpiStore: 1 = the square of relu on the accumulator
   float glu_alpha, glu_limit, glu_offset;   // kEpiGlu
   // optional: per-head RMSNorm + rotary embedding on the first rope_cols output columns
   // (heads of 128 columns; store epilogue with 256-wide tiles only, no residual / bias)
@@ -937,7 +939,7 @@ gemm_bf16_sm100_kernel(const __grid_constant__ CUtensorMap tmA0,
             if (col0 + q * 8 < col_end) {
               float f[8];
 #pragma unroll
-              for (int j = 0; j < 8; ++j) f[j] = __uint_as_float(v[q * 8 + j]);
+              for (int j = 0; j < 8; ++j) f[j] = __uint_as_float(v[q * 8 + j]) * p.acc_scale;
               if (p.col_scale) {
                 const uint32_t sw[4] = {sc[q].x, sc[q].y, sc[q].z, sc[q].w};
 #pragma unroll
@@ -1093,6 +1095,12 @@ gemm_bf16_sm100_kernel(const __grid_constant__ CUtensorMap tmA0,
               float f[8];
 #pragma unroll
               for (int j = 0; j < 8; ++j) f[j] = __uint_as_float(v[q * 8 + j]);
+              if constexpr (EPI == kEpiStore) {
+                if (p.act == 1) {
+#pragma unroll
+                  for (int j = 0; j < 8; ++j) f[j] = fmaxf(f[j], 0.f) * fmaxf(f[j], 0.f);
+                }
+              }
               uint8_t* slot = buf + own_off + (((hh * 4 + q) ^ (lane & 7)) << 4);
               if (col < col_end) {
                 if (p.bias) {

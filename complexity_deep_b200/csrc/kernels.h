@@ -101,11 +101,13 @@ cudaError_t launch_decode_attention(const void* q, long long q_stride_b, const v
 
 // fp32 residual stream (stream_f32.cu)
 cudaError_t launch_embed_rows(const long long* ids, const void* table, float* x, int T, int V, int W, int ldw,
-                              int ldx, int fp32, cudaStream_t stream);
+                              int ldx, int fp32, cudaStream_t stream, const void* pos = nullptr, int P = 0, int S = 1,
+                              int pos0 = 0, const int* pos_dev = nullptr);
 cudaError_t launch_rmsnorm_f32(const float* x, const void* w, float eps, float offset, void* out, int rows, int W,
-                               int ldx, int fp32, cudaStream_t stream);
-cudaError_t launch_linear_f32(const float* a, const float* b, const float* residual, const float* col_scale,
-                              float* out, int M, int K, int N, cudaStream_t stream);
+                               int ldx, int fp32, cudaStream_t stream, bool centred = false);
+cudaError_t launch_linear_f32(const float* a, long long lda, const float* b, const float* residual,
+                              const float* col_scale, float scale, int act, float* out, const int* seg, int groups,
+                              int M, int K, int N, cudaStream_t stream);
 cudaError_t launch_glu_f32(const float* gu, float* h, int T, int I, float alpha, float limit, float offset,
                            cudaStream_t stream);
 
@@ -128,6 +130,21 @@ cudaError_t launch_gla_finish(const cd_linear_attn& p, int fp32, cudaStream_t st
 bool gla_chunk_supported(const cd_linear_attn& a);
 size_t gla_chunk_workspace_bytes(const cd_linear_attn& a);
 cudaError_t launch_gla_chunk(const cd_linear_attn& a, void* ws, cudaStream_t stream);
+
+// latent attention (latent_attention.cu), delta rule (delta_rule.cu), learned routing (routed_experts.cu)
+bool latent_rows_supported(const cd_latent_attn& p);
+cudaError_t launch_latent_prepare(const cd_latent_attn& p, int fp32, cudaStream_t stream);
+cudaError_t launch_latent_rows(const cd_latent_attn& p, int fp32, cudaStream_t stream);
+bool delta_supported(const cd_delta_attn& p);
+cudaError_t launch_delta_prepare(const cd_delta_attn& p, int fp32, cudaStream_t stream);
+cudaError_t launch_delta_sequence(const cd_delta_attn& p, int fp32, cudaStream_t stream);
+cudaError_t launch_delta_finish(const cd_delta_attn& p, int fp32, cudaStream_t stream);
+cudaError_t launch_route_top(const float* logits, long long ld, int T, int E, int count, int keep, int top,
+                             long long* ids, float* weights, cudaStream_t stream);
+cudaError_t launch_gather_div(const void* x, const int* perm, int div, void* out, long long n, int rows, int row_bytes,
+                              cudaStream_t stream);
+cudaError_t launch_combine_top(const void* y, const int* inv_perm, const float* weights, int top, float scale,
+                               float* x, int T, int ldx, int fp32, cudaStream_t stream);
 
 // One operand pair of the GEMM: row-major bf16 matrices with K contiguous.
 struct GemmOperand {
@@ -159,6 +176,8 @@ struct GemmEpilogueArgs {
   int do_clamp;
   float clamp_lo, clamp_hi;
   const void* col_scale;    // kEpiStoreF32: bf16 factor per output column
+  float acc_scale = 1.f;    // kEpiStoreF32: factor of the accumulator
+  int act = 0;              // kEpiStore: 1 = the square of relu on the accumulator
   float glu_alpha, glu_limit, glu_offset;   // kEpiGlu (see GemmEpilogue)
   // failure-path self-test (see GemmParams)
   int selftest_stall;

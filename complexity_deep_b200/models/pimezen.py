@@ -8,9 +8,7 @@ checkpoint.  Storage is bf16 (tensor-core kernels) or fp32 (every operation in 3
 """
 from __future__ import annotations
 
-import json
 from dataclasses import dataclass
-from pathlib import Path
 from typing import Any, Dict, List, Optional
 
 import torch
@@ -21,11 +19,9 @@ from ..core._cache import DerivedCache
 from ..core.mixers import GatedLinearAttention, ParallelMixers, WindowAttention
 from ..core.mlp import ClampedGLU
 from ..core.normalization import StreamNorm
-from ..core.padding import ROW_ALIGN, pad_rows, pad_vector, round_up
-from ..core.state import DecoderState, StatePool
-from .generation import GenerationMixin
-from .modeling import CausalLMOutput
-from .weights import read_safetensors, write_safetensors
+from ..core.padding import pad_vector
+from ..core.state import DecoderState
+from .decoder import StreamDecoder
 
 
 @dataclass
@@ -143,68 +139,26 @@ class PimezenLayer(nn.Module):
         return x
 
 
-class PimezenModel(nn.Module, GenerationMixin):
+class PimezenModel(StreamDecoder):
     config_class = PimezenConfig
 
     def __init__(self, config: PimezenConfig) -> None:
-        super().__init__()
-        self.config = config
+        super().__init__(config)
         self.embed_tokens = nn.Embedding(config.vocab, config.width)
         self.layers = nn.ModuleList(PimezenLayer(config.width, s, config.eps) for s in config.layers)
         self.norm = StreamNorm(config.width, config.eps, offset=1.0)
-        self._derived = DerivedCache()
         for m in self.modules():
             if isinstance(m, (nn.Linear, nn.Embedding)):
                 nn.init.normal_(m.weight, std=0.02)
 
-    # ------------------------------------------------------------------ state
-    def new_state(self, batch: int, capacity: Optional[int] = None) -> DecoderState:
-        w = self.embed_tokens.weight
-        return DecoderState([layer.mixers.new_state(batch, w.device, w.dtype) for layer in self.layers],
-                            batch, w.device, capacity)
-
-    def make_decode_cache(self, batch: int, capacity: int) -> DecoderState:
-        """State for captured decode steps: the position is read on the device."""
-        state = self.new_state(batch, capacity)
-        state.device_position = True
-        return state
-
-    def state_pool(self, batch: int = 1) -> StatePool:
-        return StatePool(lambda: self.new_state(batch))
-
     # ------------------------------------------------------------------ forward
-    def _table(self) -> torch.Tensor:
-        w = self.embed_tokens.weight
-        return self._derived.get("table", (w,), lambda: pad_rows(
-            w.detach(), round_up(self.config.vocab, ROW_ALIGN), round_up(self.config.width, ROW_ALIGN)))
+    def embed(self, input_ids: torch.Tensor, state: DecoderState) -> torch.Tensor:
+        table = self.padded_rows("table", self.embed_tokens.weight)
+        return ops.embed_rows(input_ids, table, self.config.width, table.shape[1])
 
-    @torch.no_grad()
-    def forward(self, input_ids: torch.Tensor, past_key_values: Optional[DecoderState] = None,
-                use_cache: bool = False, logit_rows: Optional[torch.Tensor] = None) -> CausalLMOutput:
-        """input_ids [B, S]: the next S tokens of B sequences.  ``past_key_values``: the state
-        returned by an earlier call, which is carried on IN PLACE; None starts new sequences.
-        ``logit_rows`` (indices into the B * S tokens) restricts the logits to those tokens, which
-        then come back as [rows, vocab]."""
-        B, S = input_ids.shape
-        state = past_key_values if past_key_values is not None else self.new_state(B)
-        if state.batch != B:
-            raise ValueError(f"the state holds {state.batch} sequences, the call has {B}")
-        if state.device_position and S != 1:
-            raise RuntimeError("a device-side position takes one new token per sequence")
-        table = self._table()
-        x = ops.embed_rows(input_ids, table, self.config.width, table.shape[1])
-        for layer, parts in zip(self.layers, state.layers):
-            x = layer(x, parts, state, B, S)
-        state.advance(S)
-        if logit_rows is not None:
-            x = x[logit_rows].contiguous()
-        if x.shape[0] == 0:
-            return CausalLMOutput(logits=x.new_empty(0, self.config.vocab),
-                                  past_key_values=state if use_cache else None)
-        logits = ops.linear_to_f32(self.norm(x), table, tag="linear_lm_head")[:, : self.config.vocab]
-        if logit_rows is None:
-            logits = logits.unflatten(0, (B, S))
-        return CausalLMOutput(logits=logits, past_key_values=state if use_cache else None)
+    def logits(self, x: torch.Tensor) -> torch.Tensor:
+        table = self.padded_rows("table", self.embed_tokens.weight)
+        return ops.linear_to_f32(self.norm(x), table, tag="linear_lm_head")[:, : self.config.vocab]
 
     # ------------------------------------------------------------------ checkpoints
     def checkpoint_names(self) -> Dict[str, str]:
@@ -229,40 +183,8 @@ class PimezenModel(nn.Module, GenerationMixin):
         return names
 
     @classmethod
-    def from_pretrained(cls, path: str, device: str = "cpu", dtype: Optional[torch.dtype] = None
-                        ) -> "PimezenModel":
-        """Loads config.json and model.safetensors; dtype None keeps bfloat16."""
-        source = Path(path)
-        config = PimezenConfig.from_dict(json.loads((source / "config.json").read_text()))
-        tensors = read_safetensors(source / "model.safetensors")
+    def sizes_from_tensors(cls, config: PimezenConfig, tensors: Dict[str, torch.Tensor]) -> None:
         for i, layer in enumerate(config.layers):
             a1 = tensors.get(f"l{i}.mix.right.a1")
-            if a1 is not None:                       # a missing tensor is reported below
+            if a1 is not None:                       # a missing tensor is reported by the loader
                 layer.right.rank = a1.shape[0]
-        with torch.device("meta"):
-            model = cls(config)
-        dtype = dtype or torch.bfloat16
-        names = model.checkpoint_names()
-        params = dict(model.named_parameters())
-        missing = [v for v in names.values() if v not in tensors]
-        extra = sorted(set(tensors) - set(names.values()))
-        if missing or extra:
-            raise ValueError(f"checkpoint does not fit the config: missing {missing}, unexpected {extra}")
-        state = {}
-        for k, v in names.items():
-            if tensors[v].shape != params[k].shape:
-                raise ValueError(f"{v}: shape {tuple(tensors[v].shape)}, the config implies {tuple(params[k].shape)}")
-            state[k] = tensors[v].to(device=device, dtype=dtype, copy=True)
-        model.load_state_dict(state, strict=True, assign=True)
-        return model.requires_grad_(False).eval()
-
-    def save_pretrained(self, path: str) -> None:
-        target = Path(path)
-        target.mkdir(parents=True, exist_ok=True)
-        (target / "config.json").write_text(json.dumps(self.config.to_dict(), indent=1))
-        params = dict(self.named_parameters())
-        write_safetensors(target / "model.safetensors",
-                          {v: params[k] for k, v in self.checkpoint_names().items()})
-
-    def num_parameters(self, trainable_only: bool = True) -> int:
-        return sum(p.numel() for p in self.parameters() if p.requires_grad or not trainable_only)

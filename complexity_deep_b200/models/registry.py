@@ -10,11 +10,13 @@ import torch
 
 from .modeling import ComplexityModel
 from .pimezen import PimezenModel
+from .rugedra import RugedraModel
 
 DEFAULT_ARCHITECTURE = "Complexity"
 MODELS: Dict[str, Type[torch.nn.Module]] = {
     DEFAULT_ARCHITECTURE: ComplexityModel,
     "Pimezen": PimezenModel,
+    "Rugedra": RugedraModel,
 }
 
 

@@ -772,6 +772,44 @@ def embed_rows(ids: torch.Tensor, table: torch.Tensor, width: int, ldx: int) -> 
     return x
 
 
+def embed_positions(ids: torch.Tensor, table: torch.Tensor, pos_table: torch.Tensor, width: int, ldx: int,
+                    seq_len: int, pos0: int, pos_dev: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """fp32 stream rows [T, ldx] = table[ids] + pos_table[position]; ids [B, seq_len], positions from
+    pos0 (or the device scalar pos_dev) in every sequence."""
+    lib = _lib.load()
+    ids = ids.reshape(-1).contiguous()
+    _need(ids, "token_ids", torch.int64)
+    fp32 = _storage(table, "embedding table")
+    _need(pos_table, "position table", table.dtype)
+    if pos_table.shape[1] != table.shape[1]:
+        raise RuntimeError("embedding and position tables differ in width")
+    if pos_dev is None and pos0 + seq_len > pos_table.shape[0]:
+        raise RuntimeError(f"position {pos0 + seq_len - 1} is beyond the {pos_table.shape[0]} learned ones")
+    T = ids.numel()
+    x = torch.empty(T, ldx, dtype=torch.float32, device=ids.device)
+    with _Span("embed_rows"):
+        _lib.check(lib.cd_embed_positions(ids.data_ptr(), table.data_ptr(), pos_table.data_ptr(), x.data_ptr(), T,
+                                          table.shape[0], pos_table.shape[0], seq_len, pos0, _ptr(pos_dev), width,
+                                          table.shape[1], ldx, fp32, _stream()), "cd_embed_positions")
+    return x
+
+
+def layernorm_f32(x: torch.Tensor, weight: torch.Tensor, eps: float, width: Optional[int] = None) -> torch.Tensor:
+    """(x - mean) / sqrt(var + eps) * weight of an fp32 stream [T, ldx] into weight's dtype, over the first
+    `width` columns (the rest of x and weight must be zero there)."""
+    lib = _lib.load()
+    _need(x, "x", torch.float32)
+    fp32 = _storage(weight, "weight")
+    T, ldx = x.shape
+    if weight.numel() != ldx:
+        raise RuntimeError("norm weight does not match the stream")
+    out = torch.empty(T, ldx, dtype=weight.dtype, device=x.device)
+    with _Span("layernorm_f32"):
+        _lib.check(lib.cd_layernorm_f32(x.data_ptr(), weight.data_ptr(), float(eps), out.data_ptr(), T, width or ldx,
+                                        ldx, fp32, _stream()), "cd_layernorm_f32")
+    return out
+
+
 def rmsnorm_f32(x: torch.Tensor, weight: torch.Tensor, eps: float, offset: float = 0.0,
                 width: Optional[int] = None) -> torch.Tensor:
     """x / sqrt(mean(x^2) + eps) * (weight + offset) of an fp32 stream [T, ldx] into weight's dtype;
@@ -790,13 +828,20 @@ def rmsnorm_f32(x: torch.Tensor, weight: torch.Tensor, eps: float, offset: float
     return out
 
 
+def _rows(x: torch.Tensor, name: str) -> int:
+    """Checks a matrix whose rows may be columns of a wider buffer; returns the C ABI's `fp32` flag."""
+    if not x.is_cuda or x.dim() != 2 or x.dtype not in (BF16, torch.float32) or x.stride(1) != 1:
+        raise RuntimeError(f"{name}: expected rows of a CUDA {BF16} or {torch.float32} buffer")
+    return 1 if x.dtype == torch.float32 else 0
+
+
 def linear_to_f32(x: torch.Tensor, w: torch.Tensor, residual: Optional[torch.Tensor] = None,
                   col_scale: Optional[torch.Tensor] = None, inplace: bool = False,
-                  tag: str = "linear_f32") -> torch.Tensor:
-    """fp32 ``residual + col_scale * (x @ w^T)``; operands bf16 (tcgen05) or fp32 (FMA pipe).
-    inplace: the residual buffer itself receives the result."""
+                  tag: str = "linear_f32", scale: float = 1.0) -> torch.Tensor:
+    """fp32 ``residual + scale * col_scale * (x @ w^T)``; operands bf16 (tcgen05) or fp32 (FMA pipe); x
+    may be columns of a wider buffer.  inplace: the residual buffer itself receives the result."""
     lib = _lib.load()
-    fp32 = _storage(x, "x")
+    fp32 = _rows(x, "x")
     _need(w, "weight", x.dtype)
     T, K = x.shape
     N = w.shape[0]
@@ -814,31 +859,76 @@ def linear_to_f32(x: torch.Tensor, w: torch.Tensor, residual: Optional[torch.Ten
         _split_k_auto(x)
     out = residual if inplace and residual is not None else torch.empty(T, N, dtype=torch.float32,
                                                                         device=x.device)
-    fn = lib.cd_linear_f32 if fp32 else lib.cd_linear_f32out
     with _Span(tag):
-        _lib.check(fn(x.data_ptr(), w.data_ptr(), _ptr(residual), _ptr(col_scale), out.data_ptr(), T,
-                      K, N, _stream()), "cd_linear_f32" if fp32 else "cd_linear_f32out")
+        if fp32:
+            _lib.check(lib.cd_linear_f32(x.data_ptr(), x.stride(0), w.data_ptr(), _ptr(residual), _ptr(col_scale),
+                                         float(scale), 0, out.data_ptr(), None, 1, T, K, N, _stream()), "cd_linear_f32")
+        else:
+            _lib.check(lib.cd_linear_f32out(x.data_ptr(), x.stride(0), w.data_ptr(), _ptr(residual), _ptr(col_scale),
+                                            float(scale), out.data_ptr(), T, K, N, _stream()), "cd_linear_f32out")
     return out
 
 
-def project(x: torch.Tensor, w: torch.Tensor, tag: str = "linear") -> torch.Tensor:
-    """``x @ w^T`` in x's dtype."""
-    return linear_to_f32(x, w, tag=tag) if x.dtype == torch.float32 else linear(x, w, tag=tag)
+ACTIVATIONS = {None: 0, "relu2": 1}     # codes of the C ABI
+
+
+def project(x: torch.Tensor, w: torch.Tensor, tag: str = "linear", act: Optional[str] = None) -> torch.Tensor:
+    """``act(x @ w^T)`` in x's dtype; x may be columns of a wider buffer."""
+    lib = _lib.load()
+    fp32 = _rows(x, "x")
+    _need(w, "weight", x.dtype)
+    T, K = x.shape
+    N = w.shape[0]
+    if w.shape[1] != K:
+        raise RuntimeError("weight does not match x")
+    out = torch.empty(T, N, dtype=x.dtype, device=x.device)
+    if not fp32:
+        _split_k_auto(x)
+    with _Span(tag):
+        if fp32:
+            _lib.check(lib.cd_linear_f32(x.data_ptr(), x.stride(0), w.data_ptr(), None, None, 1.0, ACTIVATIONS[act],
+                                         out.data_ptr(), None, 1, T, K, N, _stream()), "cd_linear_f32")
+        else:
+            _lib.check(lib.cd_project(x.data_ptr(), x.stride(0), w.data_ptr(), ACTIVATIONS[act], out.data_ptr(), T, K,
+                                      N, _stream()), "cd_project")
+    return out
+
+
+def grouped_linear_f32(x: torch.Tensor, w: torch.Tensor, seg_offsets: torch.Tensor, tag: str) -> torch.Tensor:
+    """fp32 ``x[rows of g] @ w[g]^T`` for the row ranges given by seg_offsets; w [G, N, K]."""
+    lib = _lib.load()
+    _need(x, "x", torch.float32)
+    _need(w, "weights", torch.float32)
+    _need(seg_offsets, "seg_offsets", torch.int32)
+    (T, K), (G, N, K2) = x.shape, w.shape
+    if K != K2 or seg_offsets.numel() != G + 1:
+        raise RuntimeError("grouped weights do not match x / seg_offsets")
+    out = torch.empty(T, N, dtype=torch.float32, device=x.device)
+    with _Span(tag):
+        _lib.check(lib.cd_linear_f32(x.data_ptr(), K, w.data_ptr(), None, None, 1.0, 0, out.data_ptr(),
+                                     seg_offsets.data_ptr(), G, T, K, N, _stream()), "cd_linear_f32")
+    return out
 
 
 def glu_up(x: torch.Tensor, packed_w: torch.Tensor, width: int, block_n: int, alpha: float,
-           limit: float, offset: float) -> torch.Tensor:
-    """Clamped gated unit on packed gate / up weights (pack_gate_up with one group)."""
+           limit: float, offset: float, seg_offsets: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """Clamped gated unit on packed gate / up weights (pack_gate_up); with several groups the row
+    ranges of x come from seg_offsets."""
     lib = _lib.load()
     _need(x, "x")
     _need(packed_w, "packed gate/up weights")
     T, H = x.shape
-    if tuple(packed_w.shape) != (1, lib.cd_gate_up_packed_rows(width, block_n), H):
+    G = packed_w.shape[0]
+    if tuple(packed_w.shape[1:]) != (lib.cd_gate_up_packed_rows(width, block_n), H):
         raise RuntimeError("packed weights do not match the width / tile width")
+    if seg_offsets is not None:
+        _need(seg_offsets, "seg_offsets", torch.int32)
+    if (seg_offsets is None and G != 1) or (seg_offsets is not None and seg_offsets.numel() != G + 1):
+        raise RuntimeError("seg_offsets do not match the groups")
     h = torch.empty(T, width, dtype=BF16, device=x.device)
-    with _Span("glu_up"):
-        _lib.check(lib.cd_glu_up(x.data_ptr(), packed_w.data_ptr(), h.data_ptr(), T, H, width, block_n,
-                                 float(alpha), float(limit), float(offset), _stream()), "cd_glu_up")
+    with _Span("glu_up" if seg_offsets is None else "glu_up_routed"):
+        _lib.check(lib.cd_glu_up(x.data_ptr(), _ptr(seg_offsets), G, packed_w.data_ptr(), h.data_ptr(), T, H, width,
+                                 block_n, float(alpha), float(limit), float(offset), _stream()), "cd_glu_up")
     return h
 
 
@@ -974,3 +1064,149 @@ def linear_attention_(proj: dict, out: torch.Tensor, weights: dict, state: torch
         _lib.check(lib.cd_gla_sequence(ref, fp32, _stream()), "cd_gla_sequence")
     with _Span("gla_finish"):
         _lib.check(lib.cd_gla_finish(ref, fp32, _stream()), "cd_gla_finish")
+
+
+def _need_pos_dev(pos_dev: Optional[torch.Tensor]) -> None:
+    if pos_dev is not None and (pos_dev.dtype != torch.int32 or not pos_dev.is_cuda or pos_dev.numel() != 1):
+        raise RuntimeError("pos_dev: expected one int32 on the device")
+
+
+def latent_attention_(proj: dict, out: torch.Tensor, weights: dict, cache: torch.Tensor, *, batch: int, seq_len: int,
+                      heads: int, dim: int, rot: int, rank: int, vdim: int, scale: float, eps: float,
+                      out_scale: float, pos0: int, pos_dev: Optional[torch.Tensor] = None) -> None:
+    """Latent attention of `seq_len` new tokens per sequence (cd_latent_attn).  proj: 'q', 'kv', 'gate'
+    column slices (q and kv are changed in place); weights: 'norm', 'cos', 'sin', 'uk' [H, dimp, rankp],
+    'uk_t' [H, rankp, dimp], 'uv' [H, vp, rankp]; cache [B, capacity, rankp + rotp] receives the new rows."""
+    lib = _lib.load()
+    dt = out.dtype
+    fp32 = 1 if dt == torch.float32 else 0
+    q, kv, gate = proj["q"], proj["kv"], proj["gate"]
+    uk, uk_t, uv = weights["uk"], weights["uk_t"], weights["uv"]
+    dimp, rankp, vp = uk.shape[1], uk.shape[2], uv.shape[1]
+    rotp = kv.shape[1] - rankp
+    T = batch * seq_len
+    if (tuple(q.shape) != (T, heads * (dimp + rotp)) or kv.shape[0] != T or rotp < rot or gate.shape[0] != T
+            or gate.shape[1] < heads or tuple(out.shape) != (T, heads * vp)):
+        raise RuntimeError("latent attention: projection columns do not match the head layout")
+    if q.stride(0) != kv.stride(0) or q.stride(0) != gate.stride(0):
+        raise RuntimeError("latent attention: q, kv and gate must share their row stride")
+    for name, shape in (("uk", (heads, dimp, rankp)), ("uk_t", (heads, rankp, dimp)), ("uv", (heads, vp, rankp)),
+                        ("norm", (rankp,))):
+        _need(weights[name], name, dt)
+        if tuple(weights[name].shape) != shape:
+            raise RuntimeError(f"latent attention: {name} has the wrong shape")
+    for name in ("cos", "sin"):
+        _need(weights[name], name, torch.float32)
+        if weights[name].shape[1] != rotp // 2:
+            raise RuntimeError(f"latent attention: {name} does not match the rotated part")
+    _need(cache, "latent cache", dt)
+    if cache.shape[0] != batch or cache.shape[2] != rankp + rotp:
+        raise RuntimeError("latent attention: cache does not match batch / widths")
+    _need_pos_dev(pos_dev)
+    if pos_dev is None and pos0 + seq_len > min(cache.shape[1], weights["cos"].shape[0]):
+        raise RuntimeError("latent attention: more tokens than the cache or the position tables hold")
+    a = _lib.LatentAttn(
+        q=_columns(q, "q", dt), kv=_columns(kv, "kv", dt), gate=_columns(gate, "gate", dt), ldp=q.stride(0),
+        norm_w=weights["norm"].data_ptr(), cos_t=weights["cos"].data_ptr(), sin_t=weights["sin"].data_ptr(),
+        uk=uk.data_ptr(), uk_t=uk_t.data_ptr(), uv=uv.data_ptr(), cache=cache.data_ptr(),
+        out=_columns(out, "out", dt), ldo=out.stride(0), pos_dev=_ptr(pos_dev), scale=float(scale), eps=float(eps),
+        out_scale=float(out_scale), B=batch, S=seq_len, H=heads, dim=dim, dimp=dimp, rot=rot, rotp=rotp, rank=rank,
+        rankp=rankp, vdim=vdim, vp=vp, capacity=cache.shape[1], positions=weights["cos"].shape[0], pos0=pos0)
+    ref = ctypes.byref(a)
+    with _Span("latent_prepare"):
+        _lib.check(lib.cd_latent_prepare(ref, fp32, _stream()), "cd_latent_prepare")
+    with _Span("latent_rows"):
+        _lib.check(lib.cd_latent_rows(ref, fp32, _stream()), "cd_latent_rows")
+
+
+def delta_attention_(proj: dict, out: torch.Tensor, weights: dict, ring: torch.Tensor, state: torch.Tensor, *,
+                     batch: int, seq_len: int, heads: int, kv_heads: int, dim: int, vdim: int, eps: float,
+                     out_scale: float, pos0: int, pos_dev: Optional[torch.Tensor] = None) -> None:
+    """Delta rule with per-channel decay over `seq_len` new tokens per sequence (cd_delta_attn).  proj: 'q',
+    'k', 'v', 'b' and 'inner' column slices; weights: 'inner' [H * dkp + H * dvp, inner width] (from the
+    inner projection to decay and gate inputs), 'taps' [taps, C], 'rate', 'dt_bias' (fp32), 'norm'; `ring`
+    [B, taps, C] and `state` [B, H, dkp, dvp] fp32 are carried on in place."""
+    lib = _lib.load()
+    dt = out.dtype
+    fp32 = 1 if dt == torch.float32 else 0
+    _need(state, "state", torch.float32)
+    _need(ring, "convolution ring", dt)
+    dkp, dvp, taps = state.shape[2], state.shape[3], ring.shape[1]
+    T, C = batch * seq_len, 2 * kv_heads * dkp + heads * dvp
+    for name, n in (("q", kv_heads * dkp), ("k", kv_heads * dkp), ("v", heads * dvp)):
+        if tuple(proj[name].shape) != (T, n) or proj[name].stride(0) != proj["b"].stride(0):
+            raise RuntimeError(f"delta rule: {name} columns do not match the head layout")
+    if proj["b"].shape[0] != T or proj["b"].shape[1] < heads or tuple(out.shape) != (T, heads * dvp):
+        raise RuntimeError("delta rule: columns do not match the head layout")
+    if tuple(state.shape[:2]) != (batch, heads) or ring.shape[0] != batch or ring.shape[2] != C:
+        raise RuntimeError("delta rule: state or ring does not match the head layout")
+    for name, n, d in (("taps", taps * C, dt), ("rate", heads, torch.float32),
+                       ("dt_bias", heads * dkp, torch.float32), ("norm", dvp, dt)):
+        _need(weights[name], name, d)
+        if weights[name].numel() != n:
+            raise RuntimeError(f"delta rule: {name} has the wrong size")
+    if weights["inner"].shape[0] != heads * (dkp + dvp):
+        raise RuntimeError("delta rule: inner weights do not match the head layout")
+    _need_pos_dev(pos_dev)
+    zg = linear_to_f32(proj["inner"], weights["inner"], tag="delta_inner")
+    act = torch.empty(T, C, dtype=dt, device=out.device)
+    inv = torch.empty(T, 2 * kv_heads, dtype=torch.float32, device=out.device)
+    o_raw = torch.empty(T, heads * dvp, dtype=torch.float32, device=out.device)
+    a = _lib.DeltaAttn(
+        q=_columns(proj["q"], "q", dt), k=_columns(proj["k"], "k", dt), v=_columns(proj["v"], "v", dt),
+        b=_columns(proj["b"], "b", dt), ldp=proj["b"].stride(0), zg=zg.data_ptr(), ldz=zg.shape[1],
+        taps_w=weights["taps"].data_ptr(), rate=weights["rate"].data_ptr(), dt_bias=weights["dt_bias"].data_ptr(),
+        norm_w=weights["norm"].data_ptr(), ring=ring.data_ptr(), state=state.data_ptr(),
+        out=_columns(out, "out", dt), ldo=out.stride(0), act=act.data_ptr(), inv=inv.data_ptr(),
+        o_raw=o_raw.data_ptr(), pos_dev=_ptr(pos_dev), eps=float(eps), out_scale=float(out_scale), B=batch,
+        S=seq_len, H=heads, G=kv_heads, dk=dim, dkp=dkp, dv=vdim, dvp=dvp, taps=taps, pos0=pos0)
+    ref = ctypes.byref(a)
+    with _Span("delta_prepare"):
+        _lib.check(lib.cd_delta_prepare(ref, fp32, _stream()), "cd_delta_prepare")
+    with _Span("delta_sequence"):
+        _lib.check(lib.cd_delta_sequence(ref, fp32, _stream()), "cd_delta_sequence")
+    with _Span("delta_finish"):
+        _lib.check(lib.cd_delta_finish(ref, fp32, _stream()), "cd_delta_finish")
+
+
+# --------------------------------------------------------------------------- learned routing
+def route_top(logits: torch.Tensor, experts: int, top: int, groups: int = 1, keep: int = 1):
+    """Experts [T, top] (int64) and weights [T, top] (fp32) from fp32 logits [T, >= experts] (cd_route_top)."""
+    lib = _lib.load()
+    _need(logits, "router logits", torch.float32)
+    T = logits.shape[0]
+    ids = torch.empty(T, top, dtype=torch.int64, device=logits.device)
+    weights = torch.empty(T, top, dtype=torch.float32, device=logits.device)
+    with _Span("route_top"):
+        _lib.check(lib.cd_route_top(logits.data_ptr(), logits.shape[1], T, experts, groups, keep, top, ids.data_ptr(),
+                                    weights.data_ptr(), _stream()), "cd_route_top")
+    return ids, weights
+
+
+def gather_div(x: torch.Tensor, perm: torch.Tensor, div: int) -> torch.Tensor:
+    """out[i] = x[perm[i] // div]"""
+    lib = _lib.load()
+    _storage(x, "x")
+    _need(perm, "perm", torch.int32)
+    out = torch.empty(perm.numel(), x.shape[1], dtype=x.dtype, device=x.device)
+    with _Span("gather_div"):
+        _lib.check(lib.cd_gather_div(x.data_ptr(), perm.data_ptr(), div, out.data_ptr(), perm.numel(), x.shape[0],
+                                     x.shape[1] * x.element_size(), _stream()), "cd_gather_div")
+    return out
+
+
+def combine_top_(stream: torch.Tensor, y: torch.Tensor, inv_perm: torch.Tensor, weights: torch.Tensor,
+                 scale: float) -> torch.Tensor:
+    """stream[t] += scale * sum_j weights[t, j] * y[inv_perm[t * top + j]]"""
+    lib = _lib.load()
+    fp32 = _storage(y, "y")
+    _need(stream, "stream", torch.float32)
+    _need(weights, "weights", torch.float32)
+    _need(inv_perm, "inv_perm", torch.int32)
+    T, top = weights.shape
+    if tuple(y.shape) != (T * top, stream.shape[1]) or stream.shape[0] != T or inv_perm.numel() != T * top:
+        raise RuntimeError("combine_top: shapes do not match")
+    with _Span("combine_top"):
+        _lib.check(lib.cd_combine_top(y.data_ptr(), inv_perm.data_ptr(), weights.data_ptr(), top, float(scale),
+                                      stream.data_ptr(), T, stream.shape[1], fp32, _stream()), "cd_combine_top")
+    return stream

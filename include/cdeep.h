@@ -382,20 +382,33 @@ int cd_linear(const void* x, const void* w, const void* residual, const void* re
 /* x[t, :W] = table[ids[t], :W] (rows ldw apart), columns [W, ldx) = 0; ids are clamped to [0, V). */
 int cd_embed_rows(const int64_t* ids, const void* table, float* x, int T, int V, int W, int ldw,
                   int ldx, int fp32, void* stream);
+/* The same plus a learned vector per position: x[t] += pos[p], p = pos0 + t % S (pos0 read from
+ * pos_dev when that is given), clamped to [0, P); pos [P, :W], rows ldw apart, in the table's type. */
+int cd_embed_positions(const int64_t* ids, const void* table, const void* pos, float* x, int T, int V,
+                       int P, int S, int pos0, const int32_t* pos_dev, int W, int ldw, int ldx,
+                       int fp32, void* stream);
 /* out = x / sqrt(mean_W(x^2) + eps) * (w + offset); x, out [T, ldx], w [ldx]. */
 int cd_rmsnorm_f32(const float* x, const void* w, float eps, float offset, void* out, int T, int W,
                    int ldx, int fp32, void* stream);
-/* bf16 operands, fp32 result: out = residual + col_scale * (x @ w^T); x [T, K], w [N, K],
- * col_scale bf16 [N] or NULL, residual fp32 [T, N] or NULL (may be `out`). */
-int cd_linear_f32out(const void* x, const void* w, const float* residual, const void* col_scale,
-                     float* out, int T, int K, int N, void* stream);
-/* The same with fp32 operands (K a multiple of 4). */
-int cd_linear_f32(const float* x, const float* w, const float* residual, const float* col_scale,
-                  float* out, int T, int K, int N, void* stream);
-/* Clamped gated unit on packed gate/up weights (cd_pack_gate_up, one group):
+/* Layer norm without a bias: d = x - mean_W(x), out = d / sqrt(mean_W(d^2) + eps) * w (w zero beyond W). */
+int cd_layernorm_f32(const float* x, const void* w, float eps, void* out, int T, int W, int ldx,
+                     int fp32, void* stream);
+/* bf16 operands, fp32 result: out = residual + scale * col_scale * (x @ w^T); x [T, K] with rows ldx
+ * apart, w [N, K], col_scale bf16 [N] or NULL, residual fp32 [T, N] or NULL (may be `out`). */
+int cd_linear_f32out(const void* x, int64_t ldx, const void* w, const float* residual,
+                     const void* col_scale, float scale, float* out, int T, int K, int N, void* stream);
+/* bf16 in, bf16 out, rows of x ldx apart: out = act(x @ w^T); act: 0 none, 1 the square of relu. */
+int cd_project(const void* x, int64_t ldx, const void* w, int act, void* out, int T, int K, int N,
+               void* stream);
+/* fp32 operands (K a multiple of 4): out = residual + scale * col_scale * act(x @ w^T).  With groups > 1
+ * (seg_offsets int32 [groups + 1]) row range g of x meets w[g], w [groups, N, K]. */
+int cd_linear_f32(const float* x, int64_t ldx, const float* w, const float* residual,
+                  const float* col_scale, float scale, int act, float* out, const int32_t* seg_offsets,
+                  int groups, int T, int K, int N, void* stream);
+/* Clamped gated unit on packed gate/up weights (cd_pack_gate_up; row ranges as in cd_moe_up):
  * h = g sigmoid(alpha g) (u + offset), g = min(x Wg^T, limit), u = clamp(x Wu^T, -limit, limit). */
-int cd_glu_up(const void* x, const void* packed_w, void* h, int T, int H, int I, int block_n,
-              float alpha, float limit, float offset, void* stream);
+int cd_glu_up(const void* x, const int32_t* seg_offsets, int groups, const void* packed_w, void* h, int T,
+              int H, int I, int block_n, float alpha, float limit, float offset, void* stream);
 /* The same function of fp32 pre-activations gu [T, 2 I] (gate columns, then up). */
 int cd_glu_f32(const float* gu, float* h, int T, int I, float alpha, float limit, float offset,
                void* stream);
@@ -481,6 +494,90 @@ int cd_gla_finish(const cd_linear_attn* h_args, int fp32, void* stream);
  * state).  The workspace size is 0 where the form does not apply (heads wider than 256). */
 size_t cd_gla_chunk_workspace_bytes(const cd_linear_attn* h_args);
 int cd_gla_chunk(const cd_linear_attn* h_args, void* workspace, size_t bytes, void* stream);
+
+/* ------------------------------------------------------------------ latent attention ---------
+ * Causal attention over a cached low-rank latent c_j (rank wide, RMS-normed) and one rotated key part
+ * r_j shared by all heads:
+ *   s_h(i, j) = scale ((uk_h c_j) . q_h(i) + r_j . q'_h(i)),   w = softmax over j <= i
+ *   out_h(i)  = out_scale sigmoid(gate_h(i)) sum_j w_h(i, j) uv_h c_j
+ * q' and r are rotated by position (interleaved pairs).  The score equals (uk_h^T q_h) . c + q'_h . r, so
+ * one cached row serves all heads without being expanded. */
+typedef struct cd_latent_attn {
+  void* q;              /* projection rows b * S + t, ldp elements apart: per head dimp, then rotp elements */
+  void* kv;             /* rankp latent elements, then rotp of the shared key part */
+  const void* gate;     /* H elements; q, kv, gate 16-byte aligned, ldp a multiple of 8 */
+  long long ldp;
+  const void* norm_w;   /* [rankp] weight of the latent's norm */
+  const float* cos_t;   /* [positions, rotp / 2], 1 / 0 beyond the rotated pairs */
+  const float* sin_t;
+  const void* uk;       /* [H, dimp, rankp] */
+  const void* uk_t;     /* [H, rankp, dimp] */
+  const void* uv;       /* [H, vp, rankp] */
+  void* cache;          /* [B, capacity, rankp + rotp]: normed latent, rotated key part */
+  void* out;            /* rows of H * vp elements, ldo apart */
+  long long ldo;
+  const int32_t* pos_dev;   /* position of the call's first token, read on the device ... */
+  float scale, eps, out_scale;
+  int B, S, H, dim, dimp, rot, rotp, rank, rankp, vdim, vp;
+  int capacity, positions;
+  int pos0;             /* ... or given here when pos_dev is NULL */
+} cd_latent_attn;
+
+/* Norms the latent (in place), rotates q' (in place) and the shared key part, appends to the cache. */
+int cd_latent_prepare(const cd_latent_attn* h_args, int fp32, void* stream);
+/* One block per query and head (any S, any sizes up to 1024 per head and latent). */
+int cd_latent_rows(const cd_latent_attn* h_args, int fp32, void* stream);
+
+/* ------------------------------------------------------------------ delta rule ---------------
+ * Short causal convolution and silu on q, k, v; q and k unit vectors per head; per head h with the q / k
+ * head h / (H / G), decay g per key channel, beta = sigmoid(b):
+ *   log g = -rate_h softplus(z + dt_bias);  S <- diag(g) S;  u = beta (v - S^T k);  S <- S + k u^T
+ *   o = S^T q / sqrt(dk);   out = out_scale (o / rms(o) * norm_w) sigmoid(gate) */
+typedef struct cd_delta_attn {
+  const void* q;        /* projection rows b * S + t, ldp elements apart; G heads of dkp (q, k), H heads */
+  const void* k;        /* of dvp (v), multiples of 16 of which dk / dv are in use and the rest zero; */
+  const void* v;        /* b: H elements */
+  const void* b;
+  long long ldp;
+  const float* zg;      /* rows of H * dkp decay inputs z, then H * dvp gate inputs; ldz elements apart */
+  long long ldz;
+  const void* taps_w;   /* [taps, C], C = 2 G dkp + H dvp (q, k, v channels); the last row is the current token's */
+  const float* rate;    /* [H] */
+  const float* dt_bias; /* [H * dkp] */
+  const void* norm_w;   /* [dvp] */
+  void* ring;           /* [B, taps, C] inputs of the convolution: position p in slot p % taps */
+  float* state;         /* [B, H, dkp, dvp] fp32, read and replaced */
+  void* out;            /* rows of H * dvp elements, ldo apart */
+  long long ldo;
+  void* act;            /* scratch [B * S, C]: q, k, v after convolution and silu */
+  float* inv;           /* scratch [B * S, 2 G]: 1 / norm of q (times 1 / sqrt(dk)) and of k */
+  float* o_raw;         /* scratch [B * S, H * dvp] (cd_delta_sequence, cd_delta_chunk, cd_delta_finish) */
+  const int32_t* pos_dev;   /* position of the call's first token, read on the device ... */
+  float eps, out_scale;
+  int B, S, H, G, dk, dkp, dv, dvp, taps;
+  int pos0;             /* ... or given here when pos_dev is NULL */
+} cd_delta_attn;
+
+int cd_delta_supported(const cd_delta_attn* h_args);
+/* Convolution, silu and the norms of q and k; brings the ring up to date. */
+int cd_delta_prepare(const cd_delta_attn* h_args, int fp32, void* stream);
+/* Walks the tokens one by one (o_raw, state). */
+int cd_delta_sequence(const cd_delta_attn* h_args, int fp32, void* stream);
+/* Head norm and gate on o_raw. */
+int cd_delta_finish(const cd_delta_attn* h_args, int fp32, void* stream);
+
+/* ------------------------------------------------------------------ learned routing ----------
+ * s = softmax(logits[t, :E]); the `keep` best of `count` equal groups of neighbouring experts (a group's
+ * score: its largest s); the `top` largest s within them, weights s / (sum of the chosen + 1e-20).
+ * ids and weights [T, top], best first; E <= 128. */
+int cd_route_top(const float* logits, int64_t ld, int T, int E, int count, int keep, int top, int64_t* ids,
+                 float* weights, void* stream);
+/* out[i] = x[perm[i] / div], rows of row_bytes (a multiple of 16). */
+int cd_gather_div(const void* x, const int32_t* perm, int div, void* out, int64_t n, int rows, int row_bytes,
+                  void* stream);
+/* stream[t] += scale * sum_j weights[t, j] * y[inv_perm[t * top + j]]; y [T * top, ldx]. */
+int cd_combine_top(const void* y, const int32_t* inv_perm, const float* weights, int top, float scale,
+                   float* stream_rows, int T, int ldx, int fp32, void* stream);
 
 #ifdef __cplusplus
 }
