@@ -156,6 +156,8 @@ SIGNATURES = {
     "cd_gla_chunk_workspace_bytes": (c_size_t, [ctypes.POINTER(LinearAttn)]),
     "cd_latent_prepare": _LATENT_FN,
     "cd_latent_rows": _LATENT_FN,
+    "cd_latent_prefill_supported": (c_int, [ctypes.POINTER(LatentAttn)]),
+    "cd_latent_prefill": (c_int, [ctypes.POINTER(LatentAttn), c_void_p, c_void_p]),
     "cd_delta_supported": (c_int, [ctypes.POINTER(DeltaAttn)]),
     "cd_delta_prepare": _DELTA_FN,
     "cd_delta_sequence": _DELTA_FN,

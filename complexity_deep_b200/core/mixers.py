@@ -212,11 +212,11 @@ class LatentAttention(Mixer):
 
         def make():
             H = self.heads
-            uk = pad_heads(self.uk_proj.weight.detach(), H, self.dim_width)
-            uv = pad_heads(self.uv_proj.weight.detach(), H, self.value_width)
-            expand = pad_rows(torch.cat([uk, uv], 0), uk.shape[0] + uv.shape[0], self.rank_width).contiguous()
-            uk, uv = expand[: uk.shape[0]], expand[uk.shape[0]:]
-            uk = uk.view(H, self.dim_width, self.rank_width)
+            uk, uv = (pad_rows(w.detach(), w.shape[0], self.rank_width)
+                      for w in (self.uk_proj.weight, self.uv_proj.weight))
+            uv = pad_heads(uv, H, self.value_width).contiguous()
+            expand = torch.cat([pad_heads(uk, H, round_up(self.dim, 64)), uv], 0)
+            uk = pad_heads(uk, H, self.dim_width).reshape(H, self.dim_width, self.rank_width).contiguous()
             cos, sin = interleaved_tables(self.positions, self.rot_dims, self.rot_width, self.rot_base, uk.device)
             return {"norm": pad_vector(self.kv_norm.detach(), self.rank_width), "uk": uk, "expand": expand,
                     "uk_t": uk.transpose(1, 2).contiguous(), "uv": uv.view(H, self.value_width, self.rank_width),

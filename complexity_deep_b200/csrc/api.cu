@@ -824,6 +824,17 @@ int cd_latent_rows(const cd_latent_attn* a, int fp32, void* stream) {
   return e == cudaSuccess ? CD_OK : cuda_fail(e, "latent rows launch");
 }
 
+int cd_latent_prefill_supported(const cd_latent_attn* a) {
+  return latent_args_ok(a) == CD_OK && latent_prefill_supported(*a) ? 1 : 0;
+}
+
+int cd_latent_prefill(const cd_latent_attn* a, const void* expanded, void* stream) {
+  if (latent_args_ok(a) != CD_OK || !expanded || !aligned16(expanded)) return CD_ERR_INVALID;
+  if (!latent_prefill_supported(*a)) return CD_ERR_UNSUPPORTED;
+  cudaError_t e = launch_latent_prefill(*a, expanded, device_status_word(), as_stream(stream));
+  return e == cudaSuccess ? CD_OK : cuda_fail(e, "latent prefill launch");
+}
+
 static int delta_args_ok(const cd_delta_attn* a) {
   if (!a || a->B < 0 || a->S < 0 || a->B > 65535 || a->H < 1 || a->H > 65535 || a->G < 1 || a->H % a->G || a->dk < 1 ||
       a->dv < 1 || a->dkp < a->dk || a->dvp < a->dv || (a->dkp & 15) || (a->dvp & 15) || a->taps < 1 || (a->ldp & 7) ||

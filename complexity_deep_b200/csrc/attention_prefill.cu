@@ -28,6 +28,11 @@
 // The running maximum m is only raised when it grew by more than 2^8 in the exp2 domain
 // (then O and the row sum are rescaled in TMEM); otherwise the stale maximum is kept, which
 // is exact as long as the final division uses the matching row sum.
+//
+// The same kernel serves the prompts of latent attention (kLatent, cd_latent_prefill): keys start before the
+// call's first query (cached tokens), q / k tiles are made of boxes of an unrotated part (per head, from
+// the expanded latent) and of a rotated part (one per token, from the cache), values have a width of
+// their own, and the result is multiplied by a gate per row and head.
 #include <cstdint>
 #include <cuda.h>
 #include <cuda_bf16.h>
@@ -56,16 +61,28 @@ struct AttnParams {
   int ldo;
   unsigned long long wait_limit_ns;
   int* status;
+  // kLatent only
+  int pos0, keys;       // position of the first query; keys per sequence (pos0 + S)
+  int capacity;         // cache rows per sequence (rows of the rotated key part)
+  int dimp, rotp, vp;   // widths of the unrotated and rotated parts of a query and of the values
+  int nope_boxes;       // 64-column boxes of the unrotated part (the rotated part's follow)
+  int rot_col;          // column of the rotated part in a cache row
+  const __nv_bfloat16* gate;   // [T, hq] before its sigmoid, rows ldg apart
+  long long ldg;
+  float out_scale;
 };
 
-template <int D>
+// KB, VB: 64-column boxes of a q / k row and of a v row
+template <int KB, int VB>
 struct AttnSmem {
   static constexpr int kBoxBytes = 128 * 64 * 2;           // one TMA box: 128 rows x 64 columns
-  static constexpr int kTileBytes = (D / 64) * kBoxBytes;  // a Q, K or V tile
+  static constexpr int kTileBytes = KB * kBoxBytes;        // a Q or K tile
+  static constexpr int kVBytes = VB * kBoxBytes;           // a V tile
+  static constexpr int kVStages = (4 * KB + 2 * VB) > 14 ? 1 : 2;
   static constexpr int kQOff = 0;                          // Q_A, Q_B
   static constexpr int kKOff = 2 * kTileBytes;             // K ring (2 stages)
-  static constexpr int kVOff = 4 * kTileBytes;             // V ring (2 stages)
-  static constexpr int kBarOff = 6 * kTileBytes;
+  static constexpr int kVOff = 4 * kTileBytes;             // V ring
+  static constexpr int kBarOff = kVOff + kVStages * kVBytes;
   static constexpr int kNumBars = 2 + 8 + 8;               // q_full/q_empty, k/v full/empty x2, s_full/p_full/o_done/o_free x2
   static constexpr int kMiscOff = kBarOff + kNumBars * 8;
   static constexpr int kTotal = kMiscOff + 16;
@@ -78,14 +95,18 @@ __device__ __forceinline__ float fast_exp2(float x) {
   return y;
 }
 
-template <int D>
+template <int KB, int VB, bool kLatent>
 __global__ void __launch_bounds__(kAttnThreads, 1)
-attention_prefill_kernel(const __grid_constant__ CUtensorMap tm_qkv, const AttnParams p) {
-  using L = AttnSmem<D>;
-  constexpr int kDBlocks = D / 64;                 // 64-column boxes per tile
+attention_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_kv,
+                         const __grid_constant__ CUtensorMap tm_rot, const AttnParams p) {
+  using L = AttnSmem<KB, VB>;
+  constexpr int DV = VB * 64;                      // accumulator columns of O
+  constexpr int kVStages = L::kVStages;
   constexpr uint32_t kTmemCols = 512;   // S_A, S_B (128 columns each), O_A, O_B (D each)
   auto s_col = [](int x) { return static_cast<uint32_t>(x * 128); };
-  auto o_col = [](int x) { return static_cast<uint32_t>(256 + x * D); };
+  auto o_col = [](int x) { return static_cast<uint32_t>(256 + x * DV); };
+  const int nope_boxes = kLatent ? p.nope_boxes : KB;
+  const int pos0 = kLatent ? p.pos0 : 0;
 
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) &
@@ -116,7 +137,7 @@ attention_prefill_kernel(const __grid_constant__ CUtensorMap tm_qkv, const AttnP
   const int total_items = p.pairs * per_pair;
   struct Item {
     int pair, head, batch, kv_head, n_a, n_b, n_max, q_col, k_col, v_col;
-    long long row0;
+    long long row0;     // first query row of the sequence
   };
   auto decode_item = [&](int item) {
     Item w;
@@ -125,21 +146,28 @@ attention_prefill_kernel(const __grid_constant__ CUtensorMap tm_qkv, const AttnP
     w.head = rem % p.hq;
     w.batch = rem / p.hq;
     w.kv_head = w.head / (p.hq / p.hkv);
-    // query tiles 2 * pair (A) and 2 * pair + 1 (B); tile t sees KV tiles 0 .. t
-    w.n_a = 2 * w.pair + 1;
-    w.n_b = (2 * w.pair + 1 < p.q_tiles) ? 2 * w.pair + 2 : 0;     // 0: B does not exist
+    // query tiles 2 * pair (A) and 2 * pair + 1 (B) and the KV tiles that they see
+    auto kv_tiles = [&](int tile) { return (pos0 + min((tile + 1) * kQTile, p.S) - 1) / kKvTile + 1; };
+    w.n_a = kv_tiles(2 * w.pair);
+    w.n_b = (2 * w.pair + 1 < p.q_tiles) ? kv_tiles(2 * w.pair + 1) : 0;     // 0: B does not exist
     w.n_max = w.n_b > w.n_a ? w.n_b : w.n_a;
     w.row0 = static_cast<long long>(w.batch) * p.S;
-    w.q_col = w.head * D;
-    w.k_col = (p.hq + w.kv_head) * D;
-    w.v_col = (p.hq + p.hkv + w.kv_head) * D;
+    if constexpr (kLatent) {
+      w.q_col = w.head * (p.dimp + p.rotp);
+      w.k_col = w.head * nope_boxes * 64;
+      w.v_col = p.hq * nope_boxes * 64 + w.head * p.vp;
+    } else {
+      w.q_col = w.head * DV;
+      w.k_col = (p.hq + w.kv_head) * DV;
+      w.v_col = (p.hq + p.hkv + w.kv_head) * DV;
+    }
     return w;
   };
 
   if (warp == 8 && lane == 0) {
     mbar_init(q_full, 1);
     mbar_init(q_empty, 1);
-    for (int s = 0; s < 2; ++s) {
+    for (int s = 0; s < 2; ++s) {      // (a single V stage leaves its second barrier pair unused)
       mbar_init(&k_full[s], 1);
       mbar_init(&k_empty[s], 1);
       mbar_init(&v_full[s], 1);
@@ -151,7 +179,11 @@ attention_prefill_kernel(const __grid_constant__ CUtensorMap tm_qkv, const AttnP
     }
     *abort_flag = 0;
     fence_barrier_init();
-    tma_prefetch_desc(&tm_qkv);
+    tma_prefetch_desc(&tm_q);
+    if constexpr (kLatent) {
+      tma_prefetch_desc(&tm_kv);
+      tma_prefetch_desc(&tm_rot);
+    }
   } else if (warp == 9) {
     tmem_alloc(tmem_base_slot, kTmemCols);
     tmem_relinquish();
@@ -176,22 +208,31 @@ attention_prefill_kernel(const __grid_constant__ CUtensorMap tm_qkv, const AttnP
         const int q_tiles_here = w.n_b > 0 ? 2 : 1;
         mbar_arrive_expect_tx(q_full, q_tiles_here * L::kTileBytes);
         for (int x = 0; x < q_tiles_here; ++x)
-          for (int d = 0; d < kDBlocks; ++d)
-            tma_load_2d(smem + L::kQOff + x * L::kTileBytes + d * L::kBoxBytes, &tm_qkv, q_full,
-                        w.q_col + d * 64, static_cast<int>(w.row0) + (2 * w.pair + x) * kQTile);
+          for (int d = 0; d < KB; ++d)
+            tma_load_2d(smem + L::kQOff + x * L::kTileBytes + d * L::kBoxBytes, &tm_q, q_full,
+                        w.q_col + (d < nope_boxes ? d * 64 : p.dimp + (d - nope_boxes) * 64),
+                        static_cast<int>(w.row0) + (2 * w.pair + x) * kQTile);
         for (int j = 0; j < w.n_max && ok; ++j, ++kv) {
           const int s = kv & 1;
           const uint32_t ph = (kv >> 1) & 1u;
-          const int kv_row = static_cast<int>(w.row0) + j * kKvTile;
+          const int sv = kv % kVStages;
+          const uint32_t phv = (kv / kVStages) & 1u;
+          const int kv_row = (kLatent ? w.batch * p.keys : static_cast<int>(w.row0)) + j * kKvTile;
           if (!mbar_wait(&k_empty[s], ph ^ 1u, abort_flag, wait_limit)) { ok = false; break; }
           mbar_arrive_expect_tx(&k_full[s], L::kTileBytes);
-          for (int d = 0; d < kDBlocks; ++d)
-            tma_load_2d(smem + L::kKOff + s * L::kTileBytes + d * L::kBoxBytes, &tm_qkv, &k_full[s],
+          for (int d = 0; d < nope_boxes; ++d)
+            tma_load_2d(smem + L::kKOff + s * L::kTileBytes + d * L::kBoxBytes, kLatent ? &tm_kv : &tm_q, &k_full[s],
                         w.k_col + d * 64, kv_row);
-          if (!mbar_wait(&v_empty[s], ph ^ 1u, abort_flag, wait_limit)) { ok = false; break; }
-          mbar_arrive_expect_tx(&v_full[s], L::kTileBytes);
-          for (int d = 0; d < kDBlocks; ++d)
-            tma_load_2d(smem + L::kVOff + s * L::kTileBytes + d * L::kBoxBytes, &tm_qkv, &v_full[s],
+          if constexpr (kLatent) {
+            const int rot_row = w.batch * p.capacity + j * kKvTile;
+            for (int d = nope_boxes; d < KB; ++d)
+              tma_load_2d(smem + L::kKOff + s * L::kTileBytes + d * L::kBoxBytes, &tm_rot, &k_full[s],
+                          p.rot_col + (d - nope_boxes) * 64, rot_row);
+          }
+          if (!mbar_wait(&v_empty[sv], phv ^ 1u, abort_flag, wait_limit)) { ok = false; break; }
+          mbar_arrive_expect_tx(&v_full[sv], L::kVBytes);
+          for (int d = 0; d < VB; ++d)
+            tma_load_2d(smem + L::kVOff + sv * L::kVBytes + d * L::kBoxBytes, kLatent ? &tm_kv : &tm_q, &v_full[sv],
                         w.v_col + d * 64, kv_row);
         }
       }
@@ -201,7 +242,7 @@ attention_prefill_kernel(const __grid_constant__ CUtensorMap tm_qkv, const AttnP
     // ---------------------------------------------------------------- MMA issuer
     if (lane == 0) {
       constexpr uint32_t idesc_s = make_idesc_bf16(kQTile, kKvTile);         // S = Q K^T
-      constexpr uint32_t idesc_o = make_idesc_bf16(kQTile, D, true);         // O = P V (V N-major)
+      constexpr uint32_t idesc_o = make_idesc_bf16(kQTile, DV, true);         // O = P V (V N-major)
       const uint32_t q_addr = smem_u32(smem + L::kQOff);
       const uint32_t k_addr = smem_u32(smem + L::kKOff);
       const uint32_t v_addr = smem_u32(smem + L::kVOff);
@@ -210,12 +251,13 @@ attention_prefill_kernel(const __grid_constant__ CUtensorMap tm_qkv, const AttnP
       uint32_t it = 0;               // items started
       uint32_t cnt[2] = {0, 0};      // tiles of A / B finished in earlier items (barrier phases)
       uint32_t items_x[2] = {0, 0};  // earlier items in which A / B existed (o_free phases)
-      // S_X = Q_X K^T for the K tile in ring stage `stage`: D / 16 MMAs over the 64-column boxes
+      // S_X = Q_X K^T for the K tile in ring stage `stage`: four MMAs per 64-column box
+      // (issued without conditions: columns that are not in use are zero in K)
       auto issue_s = [&](int x, int stage) {
         const uint32_t qa = q_addr + x * L::kTileBytes;
         const uint32_t ka = k_addr + stage * L::kTileBytes;
 #pragma unroll
-        for (int d = 0; d < kDBlocks; ++d) {
+        for (int d = 0; d < KB; ++d) {
           const uint64_t da = make_smem_desc_sw128(qa + d * L::kBoxBytes);
           const uint64_t db = make_smem_desc_sw128(ka + d * L::kBoxBytes);
 #pragma unroll
@@ -227,7 +269,7 @@ attention_prefill_kernel(const __grid_constant__ CUtensorMap tm_qkv, const AttnP
       // O_X (+)= P_X V: 8 MMAs of 16 keys; P sits in the first 64 columns of S_X (two bf16 per
       // column), the V tile is read N-major: 16 key rows = 2048 bytes further per step
       auto issue_pv = [&](int x, int stage, bool first) {
-        const uint64_t db0 = make_smem_desc_mn_sw128(v_addr + stage * L::kTileBytes, L::kBoxBytes);
+        const uint64_t db0 = make_smem_desc_mn_sw128(v_addr + stage * L::kVBytes, L::kBoxBytes);
         const uint32_t acc0 = first ? 0u : 1u;
 #pragma unroll
         for (int k = 0; k < kKvTile / 16; ++k)
@@ -248,8 +290,8 @@ attention_prefill_kernel(const __grid_constant__ CUtensorMap tm_qkv, const AttnP
         if (s_left == 0) umma_commit(q_empty);
         for (int j = 0; j < w.n_max && ok; ++j) {
           const uint32_t g = kv + j;                 // ring position of K_j / V_j
-          const int s = g & 1;
-          const uint32_t ph = (g >> 1) & 1u;
+          const int s = g % kVStages;                // V stage
+          const uint32_t ph = (g / kVStages) & 1u;
           for (int x = 0; x < 2 && ok; ++x) {
             if (j >= n_of[x]) continue;
             const bool last_user = (x == 1) || (j >= w.n_b);   // of V_j among the two tiles
@@ -299,16 +341,18 @@ attention_prefill_kernel(const __grid_constant__ CUtensorMap tm_qkv, const AttnP
       const Item w = decode_item(item);
       const int n_mine = x ? w.n_b : w.n_a;
       if (n_mine == 0) continue;             // the sequence has an odd number of tiles: no tile B here
-      const int q_pos = (2 * w.pair + x) * kQTile + quarter * 32 + lane;   // position of this thread's row
+      const int q_row = (2 * w.pair + x) * kQTile + quarter * 32 + lane;   // this thread's row of the call
+      const int q_pos = pos0 + q_row;                                      // and its position
+      const int tile_pos = pos0 + (2 * w.pair + x) * kQTile;               // position of the tile's first row
       float m_ref = -INFINITY;               // maximum the stored exponentials refer to (raw scores)
       float l_sum = 0.f;
       for (int j = 0; j < n_mine && ok; ++j) {
         const uint32_t g = cnt + j;          // index of this tile among all tiles of the slot
         if (!mbar_wait(&s_full[x], g & 1u, abort_flag, wait_limit)) { ok = false; break; }
         tc_fence_after();
-        const bool diagonal = (j == n_mine - 1);
         const int k_pos0 = j * kKvTile;
-        // keys of this tile the row may see: all 128, fewer on the diagonal tile (causal)
+        const bool diagonal = k_pos0 + kKvTile - 1 > tile_pos;
+        // keys of this tile the row may see: all 128, fewer on the diagonal (causal), perhaps none
         const int n_vis = diagonal ? min(kKvTile, max(q_pos - k_pos0 + 1, 0)) : kKvTile;
         // pass 1: row maximum.  The load of chunk c + 1 is in flight while chunk c is reduced.
         float m_tile = -INFINITY;
@@ -348,7 +392,7 @@ attention_prefill_kernel(const __grid_constant__ CUtensorMap tm_qkv, const AttnP
           const float alpha = grow ? fast_exp2((m_ref - m_new) * p.scale_log2) : 1.0f;
           l_sum *= alpha;
 #pragma unroll 1
-          for (int c = 0; c < D / 32; ++c) {
+          for (int c = 0; c < DV / 32; ++c) {
             uint32_t o[32];
             tmem_ld32(o_tmem + c * 32, o);
             tmem_ld_wait();
@@ -399,15 +443,21 @@ attention_prefill_kernel(const __grid_constant__ CUtensorMap tm_qkv, const AttnP
         // epilogue: O / l -> bf16 -> out[row, head * D ...]; then O may be overwritten
         if (mbar_wait(&o_done[x], (cnt + n_mine - 1) & 1u, abort_flag, wait_limit)) {
           tc_fence_after();
-          const float inv = 1.0f / l_sum;
-          const bool row_ok = q_pos < p.S;
-          __nv_bfloat16* dst = p.out + (w.row0 + q_pos) * p.ldo + w.q_col;
+          float inv = 1.0f / l_sum;
+          const bool row_ok = q_row < p.S;
+          __nv_bfloat16* dst = p.out + (w.row0 + q_row) * p.ldo + (kLatent ? w.head * p.vp : w.q_col);
+          if constexpr (kLatent) {
+            if (row_ok) {
+              const float g = __bfloat162float(p.gate[(w.row0 + q_row) * p.ldg + w.head]);
+              inv *= p.out_scale / (1.0f + expf(-g));
+            }
+          }
 #pragma unroll 1
-          for (int c = 0; c < D / 32; ++c) {
+          for (int c = 0; c < DV / 32; ++c) {
             uint32_t o[32];
             tmem_ld32(o_tmem + c * 32, o);
             tmem_ld_wait();
-            if (c == D / 32 - 1) {           // last read of O: the next item's first product may go
+            if (c == DV / 32 - 1) {           // last read of O: the next item's first product may go
               tc_fence_before();
               __syncwarp();
               if (lane == 0) mbar_arrive(&o_free[x]);
@@ -415,6 +465,7 @@ attention_prefill_kernel(const __grid_constant__ CUtensorMap tm_qkv, const AttnP
             if (row_ok) {
 #pragma unroll
               for (int q4 = 0; q4 < 4; ++q4) {
+                if (kLatent && c * 32 + q4 * 8 >= p.vp) continue;
                 uint4 wv;
                 uint32_t* ww = reinterpret_cast<uint32_t*>(&wv);
 #pragma unroll
@@ -446,6 +497,26 @@ attention_prefill_kernel(const __grid_constant__ CUtensorMap tm_qkv, const AttnP
   if (threadIdx.x == 0 && *abort_flag && p.status) atomicExch(p.status, 3);
 }
 
+template <int KB, int VB, bool kLatent>
+cudaError_t launch_one(const CUtensorMap& q, const CUtensorMap& kv, const CUtensorMap& rot, AttnParams& p,
+                       cudaStream_t stream) {
+  p.q_tiles = (p.S + kQTile - 1) / kQTile;
+  p.pairs = (p.q_tiles + 1) / 2;
+  // persistent CTAs: one per SM (up to 224 KB of shared memory and all of TMEM each), looping over items
+  const long long items = static_cast<long long>(p.pairs) * p.hq * p.batch;
+  const int sms = current_sm_count();
+  const dim3 grid(static_cast<unsigned>(items < sms ? items : sms), 1, 1);
+  constexpr int bytes = AttnSmem<KB, VB>::kDynamic;
+  static bool attr_done = false;
+  if (!attr_done) {
+    cudaError_t e = cudaFuncSetAttribute(attention_prefill_kernel<KB, VB, kLatent>,
+                                         cudaFuncAttributeMaxDynamicSharedMemorySize, bytes);
+    if (e != cudaSuccess) return e;
+    attr_done = true;
+  }
+  return launch_kernel(attention_prefill_kernel<KB, VB, kLatent>, grid, dim3(kAttnThreads), bytes, stream, q, kv, rot, p);
+}
+
 }  // namespace
 
 cudaError_t launch_attention_prefill(const void* qkv, void* out, int B, int S, int hq, int hkv, int D,
@@ -454,43 +525,56 @@ cudaError_t launch_attention_prefill(const void* qkv, void* out, int B, int S, i
   const int N = (hq + 2 * hkv) * D;
   CUtensorMap tm;
   if (!encode_map_2d(&tm, qkv, T, N, N, 128)) return cudaErrorInvalidValue;
-  AttnParams p;
+  AttnParams p = {};
   p.S = S;
   p.hq = hq;
   p.hkv = hkv;
-  p.q_tiles = (S + kQTile - 1) / kQTile;
-  p.pairs = (p.q_tiles + 1) / 2;
   p.batch = B;
   p.scale_log2 = scale * 1.4426950408889634f;
   p.out = static_cast<__nv_bfloat16*>(out);
   p.ldo = hq * D;
-  p.wait_limit_ns = 0;
   p.status = status;
-  // persistent CTAs: one per SM (192 KB of shared memory and all of TMEM each), looping over items
-  const long long items = static_cast<long long>(p.pairs) * hq * B;
-  const int sms = current_sm_count();
-  const dim3 grid(static_cast<unsigned>(items < sms ? items : sms), 1, 1);
-  static bool attr_done[2] = {false, false};
-  if (D == 128) {
-    if (!attr_done[1]) {
-      cudaError_t e = cudaFuncSetAttribute(attention_prefill_kernel<128>,
-                                           cudaFuncAttributeMaxDynamicSharedMemorySize,
-                                           AttnSmem<128>::kDynamic);
-      if (e != cudaSuccess) return e;
-      attr_done[1] = true;
-    }
-    return launch_kernel(attention_prefill_kernel<128>, grid, dim3(kAttnThreads),
-                         AttnSmem<128>::kDynamic, stream, tm, p);
-  }
-  if (!attr_done[0]) {
-    cudaError_t e = cudaFuncSetAttribute(attention_prefill_kernel<64>,
-                                         cudaFuncAttributeMaxDynamicSharedMemorySize,
-                                         AttnSmem<64>::kDynamic);
-    if (e != cudaSuccess) return e;
-    attr_done[0] = true;
-  }
-  return launch_kernel(attention_prefill_kernel<64>, grid, dim3(kAttnThreads), AttnSmem<64>::kDynamic,
-                       stream, tm, p);
+  return D == 128 ? launch_one<2, 2, false>(tm, tm, tm, p, stream) : launch_one<1, 1, false>(tm, tm, tm, p, stream);
+}
+
+static int boxes(int width) { return (width + 63) / 64; }
+
+bool latent_prefill_supported(const cd_latent_attn& a) {
+  const int kb = boxes(a.dimp) + boxes(a.rotp);
+  return kb <= 3 && a.vp <= 128 && !a.pos_dev && a.S > 0 && a.B > 0 &&
+         static_cast<long long>(a.B) * a.capacity <= 0x7fffffffLL &&
+         static_cast<long long>(a.B) * (a.pos0 + a.S) <= 0x7fffffffLL;
+}
+
+cudaError_t launch_latent_prefill(const cd_latent_attn& a, const void* expanded, int* status, cudaStream_t stream) {
+  AttnParams p = {};
+  p.S = a.S;
+  p.hq = p.hkv = a.H;
+  p.batch = a.B;
+  p.scale_log2 = a.scale * 1.4426950408889634f;
+  p.out = static_cast<__nv_bfloat16*>(a.out);
+  p.ldo = static_cast<int>(a.ldo);
+  p.status = status;
+  p.pos0 = a.pos0;
+  p.keys = a.pos0 + a.S;
+  p.capacity = a.capacity;
+  p.dimp = a.dimp;
+  p.rotp = a.rotp;
+  p.vp = a.vp;
+  p.nope_boxes = boxes(a.dimp);
+  p.rot_col = a.rankp;
+  p.gate = static_cast<const __nv_bfloat16*>(a.gate);
+  p.ldg = a.ldp;
+  p.out_scale = a.out_scale;
+  const int width = a.H * (p.nope_boxes * 64 + a.vp);
+  CUtensorMap q, kv, rot;
+  if (!encode_map_2d(&q, a.q, static_cast<long long>(a.B) * a.S, a.H * (a.dimp + a.rotp), a.ldp, 128) ||
+      !encode_map_2d(&kv, expanded, static_cast<long long>(a.B) * p.keys, width, width, 128) ||
+      !encode_map_2d(&rot, a.cache, static_cast<long long>(a.B) * a.capacity, a.rankp + a.rotp, a.rankp + a.rotp, 128))
+    return cudaErrorInvalidValue;
+  const int kb = p.nope_boxes + boxes(a.rotp), vb = boxes(a.vp);
+  if (kb == 2) return vb == 1 ? launch_one<2, 1, true>(q, kv, rot, p, stream) : launch_one<2, 2, true>(q, kv, rot, p, stream);
+  return vb == 1 ? launch_one<3, 1, true>(q, kv, rot, p, stream) : launch_one<3, 2, true>(q, kv, rot, p, stream);
 }
 
 }  // namespace cdeep

@@ -872,8 +872,9 @@ def linear_to_f32(x: torch.Tensor, w: torch.Tensor, residual: Optional[torch.Ten
 ACTIVATIONS = {None: 0, "relu2": 1}     # codes of the C ABI
 
 
-def project(x: torch.Tensor, w: torch.Tensor, tag: str = "linear", act: Optional[str] = None) -> torch.Tensor:
-    """``act(x @ w^T)`` in x's dtype; x may be columns of a wider buffer."""
+def project(x: torch.Tensor, w: torch.Tensor, tag: str = "linear", act: Optional[str] = None,
+            out: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """``act(x @ w^T)`` in x's dtype (into `out` if given); x may be columns of a wider buffer."""
     lib = _lib.load()
     fp32 = _rows(x, "x")
     _need(w, "weight", x.dtype)
@@ -881,7 +882,11 @@ def project(x: torch.Tensor, w: torch.Tensor, tag: str = "linear", act: Optional
     N = w.shape[0]
     if w.shape[1] != K:
         raise RuntimeError("weight does not match x")
-    out = torch.empty(T, N, dtype=x.dtype, device=x.device)
+    if out is None:
+        out = torch.empty(T, N, dtype=x.dtype, device=x.device)
+    _need(out, "out", x.dtype)
+    if tuple(out.shape) != (T, N):
+        raise RuntimeError("out does not match x and the weight")
     if not fp32:
         _split_k_auto(x)
     with _Span(tag):
@@ -1071,12 +1076,30 @@ def _need_pos_dev(pos_dev: Optional[torch.Tensor]) -> None:
         raise RuntimeError("pos_dev: expected one int32 on the device")
 
 
+_LATENT_EXPAND_MIN = 64     # shorter portions attend in the latent's space
+
+
+def _expand_latent(kv: torch.Tensor, cache: torch.Tensor, w: torch.Tensor, batch: int, seq_len: int,
+                   pos0: int) -> torch.Tensor:
+    """Unrotated keys and values [batch * (pos0 + seq_len), N] of all tokens so far: from the call's own
+    normed latents where nothing is cached before them, else from the cache."""
+    rank = w.shape[1]
+    if pos0 == 0:
+        return project(kv[:, :rank], w, tag="latent_expand")
+    n = pos0 + seq_len
+    out = torch.empty(batch * n, w.shape[0], dtype=w.dtype, device=w.device)
+    for b in range(batch):
+        project(cache[b, :n, :rank], w, tag="latent_expand", out=out[b * n:(b + 1) * n])
+    return out
+
+
 def latent_attention_(proj: dict, out: torch.Tensor, weights: dict, cache: torch.Tensor, *, batch: int, seq_len: int,
                       heads: int, dim: int, rot: int, rank: int, vdim: int, scale: float, eps: float,
                       out_scale: float, pos0: int, pos_dev: Optional[torch.Tensor] = None) -> None:
     """Latent attention of `seq_len` new tokens per sequence (cd_latent_attn).  proj: 'q', 'kv', 'gate'
     column slices (q and kv are changed in place); weights: 'norm', 'cos', 'sin', 'uk' [H, dimp, rankp],
-    'uk_t' [H, rankp, dimp], 'uv' [H, vp, rankp]; cache [B, capacity, rankp + rotp] receives the new rows."""
+    'uk_t' [H, rankp, dimp], 'uv' [H, vp, rankp], 'expand' [H * d64 + H * vp, rankp] (d64: dim rounded up to
+    64, zero rows beyond dim); cache [B, capacity, rankp + rotp] receives the new rows."""
     lib = _lib.load()
     dt = out.dtype
     fp32 = 1 if dt == torch.float32 else 0
@@ -1099,6 +1122,9 @@ def latent_attention_(proj: dict, out: torch.Tensor, weights: dict, cache: torch
         _need(weights[name], name, torch.float32)
         if weights[name].shape[1] != rotp // 2:
             raise RuntimeError(f"latent attention: {name} does not match the rotated part")
+    _need(weights["expand"], "expand", dt)
+    if tuple(weights["expand"].shape) != (heads * (-(-dim // 64) * 64 + vp), rankp):
+        raise RuntimeError("latent attention: expand has the wrong shape")
     _need(cache, "latent cache", dt)
     if cache.shape[0] != batch or cache.shape[2] != rankp + rotp:
         raise RuntimeError("latent attention: cache does not match batch / widths")
@@ -1115,6 +1141,11 @@ def latent_attention_(proj: dict, out: torch.Tensor, weights: dict, cache: torch
     ref = ctypes.byref(a)
     with _Span("latent_prepare"):
         _lib.check(lib.cd_latent_prepare(ref, fp32, _stream()), "cd_latent_prepare")
+    if not fp32 and seq_len >= _LATENT_EXPAND_MIN and lib.cd_latent_prefill_supported(ref):
+        expanded = _expand_latent(kv, cache, weights["expand"], batch, seq_len, pos0)
+        with _Span("latent_prefill"):
+            _lib.check(lib.cd_latent_prefill(ref, expanded.data_ptr(), _stream()), "cd_latent_prefill")
+        return
     with _Span("latent_rows"):
         _lib.check(lib.cd_latent_rows(ref, fp32, _stream()), "cd_latent_rows")
 

@@ -528,6 +528,13 @@ int cd_latent_prepare(const cd_latent_attn* h_args, int fp32, void* stream);
 /* One block per query and head (any S, any sizes up to 1024 per head and latent). */
 int cd_latent_rows(const cd_latent_attn* h_args, int fp32, void* stream);
 
+/* Prompts and portions in bf16 on the tensor cores (after cd_latent_prepare; position on the host): keys and
+ * values expanded from the latent for all pos0 + S tokens, expanded [B * (pos0 + S), H * d64 + H * vp] =
+ * latent @ [uk; uv]^T with d64 = dim rounded up to 64 (zeros beyond dim), the rotated key part from the cache.  At most three 64-column boxes of q / k and
+ * values up to 128 wide (cd_latent_prefill_supported). */
+int cd_latent_prefill_supported(const cd_latent_attn* h_args);
+int cd_latent_prefill(const cd_latent_attn* h_args, const void* expanded, void* stream);
+
 /* ------------------------------------------------------------------ delta rule ---------------
  * Short causal convolution and silu on q, k, v; q and k unit vectors per head; per head h with the q / k
  * head h / (H / G), decay g per key channel, beta = sigmoid(b):

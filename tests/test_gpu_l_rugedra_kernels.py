@@ -73,11 +73,13 @@ class Latent:
         dp, kp, vp, rp = _up(self.dim), _up(self.rank), _up(self.vdim), _up(self.rot)
         uk, uv = torch.zeros(self.H, dp, kp), torch.zeros(self.H, vp, kp)
         uk[:, :self.dim, :self.rank], uv[:, :self.vdim, :self.rank] = torch.tensor(self.uk), torch.tensor(self.uv)
-        expand = torch.cat([uk.view(-1, kp), uv.view(-1, kp)]).to(dtype=self.dtype, device="cuda")
+        d64 = -(-self.dim // 64) * 64
+        dev = dict(dtype=self.dtype, device="cuda")
+        expand = torch.cat([torch.nn.functional.pad(uk, (0, 0, 0, d64 - dp)).view(-1, kp), uv.view(-1, kp)]).to(**dev)
         cos, sin = interleaved_tables(self.T + 3, self.rot_dims, rp, self.base, "cuda")
-        return {"norm": torch.nn.functional.pad(torch.tensor(self.norm), (0, kp - self.rank)).to(dtype=self.dtype, device="cuda"),
-                "expand": expand, "uk": expand[: self.H * dp].view(self.H, dp, kp), "uv": expand[self.H * dp:].view(self.H, vp, kp),
-                "uk_t": expand[: self.H * dp].view(self.H, dp, kp).transpose(1, 2).contiguous(), "cos": cos, "sin": sin}
+        return {"norm": torch.nn.functional.pad(torch.tensor(self.norm), (0, kp - self.rank)).to(**dev),
+                "expand": expand, "uk": uk.to(**dev), "uv": uv.to(**dev), "uk_t": uk.transpose(1, 2).contiguous().to(**dev),
+                "cos": cos, "sin": sin}
 
     def new_cache(self, capacity=None):
         return torch.full((self.B, capacity or self.T + 5, _up(self.rank) + _up(self.rot)), 9.0, dtype=self.dtype,
