@@ -156,6 +156,8 @@ SIGNATURES = {
     "cd_gla_chunk_workspace_bytes": (c_size_t, [ctypes.POINTER(LinearAttn)]),
     "cd_latent_prepare": _LATENT_FN,
     "cd_latent_rows": _LATENT_FN,
+    "cd_latent_decode_workspace_bytes": (c_size_t, [ctypes.POINTER(LatentAttn)]),
+    "cd_latent_decode": (c_int, [ctypes.POINTER(LatentAttn), c_void_p, c_size_t, c_void_p]),
     "cd_latent_prefill_supported": (c_int, [ctypes.POINTER(LatentAttn)]),
     "cd_latent_prefill": (c_int, [ctypes.POINTER(LatentAttn), c_void_p, c_void_p]),
     "cd_delta_supported": (c_int, [ctypes.POINTER(DeltaAttn)]),

@@ -824,6 +824,18 @@ int cd_latent_rows(const cd_latent_attn* a, int fp32, void* stream) {
   return e == cudaSuccess ? CD_OK : cuda_fail(e, "latent rows launch");
 }
 
+size_t cd_latent_decode_workspace_bytes(const cd_latent_attn* a) {
+  return latent_args_ok(a) == CD_OK && latent_decode_supported(*a) ? latent_decode_workspace_bytes(*a) : 0;
+}
+
+int cd_latent_decode(const cd_latent_attn* a, void* ws, size_t ws_bytes, void* stream) {
+  if (latent_args_ok(a) != CD_OK) return CD_ERR_INVALID;
+  if (!latent_decode_supported(*a)) return CD_ERR_UNSUPPORTED;
+  if (!ws || !aligned16(ws) || ws_bytes < latent_decode_workspace_bytes(*a)) return CD_ERR_INVALID;
+  cudaError_t e = launch_latent_decode(*a, ws, as_stream(stream));
+  return e == cudaSuccess ? CD_OK : cuda_fail(e, "latent decode launch");
+}
+
 int cd_latent_prefill_supported(const cd_latent_attn* a) {
   return latent_args_ok(a) == CD_OK && latent_prefill_supported(*a) ? 1 : 0;
 }

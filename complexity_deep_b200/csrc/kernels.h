@@ -135,6 +135,9 @@ cudaError_t launch_gla_chunk(const cd_linear_attn& a, void* ws, cudaStream_t str
 bool latent_rows_supported(const cd_latent_attn& p);
 cudaError_t launch_latent_prepare(const cd_latent_attn& p, int fp32, cudaStream_t stream);
 cudaError_t launch_latent_rows(const cd_latent_attn& p, int fp32, cudaStream_t stream);
+bool latent_decode_supported(const cd_latent_attn& p);                       // latent_decode.cu
+size_t latent_decode_workspace_bytes(const cd_latent_attn& p);
+cudaError_t launch_latent_decode(const cd_latent_attn& p, void* ws, cudaStream_t stream);
 bool latent_prefill_supported(const cd_latent_attn& p);                      // attention_prefill.cu
 cudaError_t launch_latent_prefill(const cd_latent_attn& p, const void* expanded, int* status, cudaStream_t stream);
 bool delta_supported(const cd_delta_attn& p);

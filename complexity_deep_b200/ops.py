@@ -1146,6 +1146,12 @@ def latent_attention_(proj: dict, out: torch.Tensor, weights: dict, cache: torch
         with _Span("latent_prefill"):
             _lib.check(lib.cd_latent_prefill(ref, expanded.data_ptr(), _stream()), "cd_latent_prefill")
         return
+    ws_bytes = 0 if fp32 else lib.cd_latent_decode_workspace_bytes(ref)
+    if ws_bytes:
+        ws = torch.empty(ws_bytes, dtype=torch.uint8, device=out.device)
+        with _Span("latent_decode", 3):
+            _lib.check(lib.cd_latent_decode(ref, ws.data_ptr(), ws_bytes, _stream()), "cd_latent_decode")
+        return
     with _Span("latent_rows"):
         _lib.check(lib.cd_latent_rows(ref, fp32, _stream()), "cd_latent_rows")
 

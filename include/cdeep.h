@@ -528,6 +528,11 @@ int cd_latent_prepare(const cd_latent_attn* h_args, int fp32, void* stream);
 /* One block per query and head (any S, any sizes up to 1024 per head and latent). */
 int cd_latent_rows(const cd_latent_attn* h_args, int fp32, void* stream);
 
+/* A few new tokens per sequence in bf16 (after cd_latent_prepare): three kernels that take the queries to
+ * the latent's space, read the cache once per 16 or 32 (token, head) rows, and come back through uv.  The
+ * workspace size is 0 where the form does not apply (latents wider than 512 and the like). */
+size_t cd_latent_decode_workspace_bytes(const cd_latent_attn* h_args);
+int cd_latent_decode(const cd_latent_attn* h_args, void* workspace, size_t bytes, void* stream);
 /* Prompts and portions in bf16 on the tensor cores (after cd_latent_prepare; position on the host): keys and
  * values expanded from the latent for all pos0 + S tokens, expanded [B * (pos0 + S), H * d64 + H * vp] =
  * latent @ [uk; uv]^T with d64 = dim rounded up to 64 (zeros beyond dim), the rotated key part from the cache.  At most three 64-column boxes of q / k and
