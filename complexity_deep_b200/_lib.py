@@ -164,6 +164,10 @@ SIGNATURES = {
     "cd_delta_prepare": _DELTA_FN,
     "cd_delta_sequence": _DELTA_FN,
     "cd_delta_finish": _DELTA_FN,
+    "cd_delta_step_supported": (c_int, [ctypes.POINTER(DeltaAttn)]),
+    "cd_delta_step": _DELTA_FN,
+    "cd_delta_chunk_workspace_bytes": (c_size_t, [ctypes.POINTER(DeltaAttn)]),
+    "cd_delta_chunk": (c_int, [ctypes.POINTER(DeltaAttn), c_void_p, c_size_t, c_void_p]),
     "cd_route_top": (c_int, [c_void_p, c_longlong, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p]),
     "cd_gather_div": (c_int, [c_void_p, c_void_p, c_int, c_void_p, c_longlong, c_int, c_int, c_void_p]),
     "cd_combine_top": (c_int, [c_void_p, c_void_p, c_void_p, c_int, c_float, c_void_p, c_int, c_int, c_int, c_void_p]),

@@ -18,7 +18,7 @@ CHECKS_LIB_PATH = os.path.join(PKG_DIR, "libcdeep_checks.so")
 SOURCES = ["api.cu", "gemm.cu", "route.cu", "rowwise.cu", "attention_decode.cu", "attention_prefill.cu", "pack.cu", "ep_plan.cu",
            "stream_f32.cu", "window_attention.cu", "window_attention_decode.cu", "window_attention_prefill.cu",
            "linear_attention.cu", "linear_attention_chunk.cu", "latent_attention.cu", "latent_decode.cu",
-           "delta_rule.cu", "routed_experts.cu"]
+           "delta_rule.cu", "delta_rule_chunk.cu", "routed_experts.cu"]
 HEADERS = ["ptx.cuh", "checks.cuh", "gemm_sm100.cuh", "kernels.h", "elem.cuh", "mma.cuh", "window_attention.cuh", "linear_attention.cuh",
            "latent_attention.cuh", "delta_rule.cuh",
            os.path.join("..", "..", "include", "cdeep.h")]

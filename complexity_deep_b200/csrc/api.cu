@@ -878,6 +878,32 @@ int cd_delta_sequence(const cd_delta_attn* a, int fp32, void* stream) {
   return e == cudaSuccess ? CD_OK : cuda_fail(e, "delta sequence launch");
 }
 
+int cd_delta_step_supported(const cd_delta_attn* a) {
+  return delta_args_ok(a) == CD_OK && delta_step_supported(*a) ? 1 : 0;
+}
+
+int cd_delta_step(const cd_delta_attn* a, int fp32, void* stream) {
+  const int st = delta_args_ok(a);
+  if (st != CD_OK) return st;
+  if (!delta_step_supported(*a)) return CD_ERR_UNSUPPORTED;
+  cudaError_t e = launch_delta_step(*a, fp32, as_stream(stream));
+  return e == cudaSuccess ? CD_OK : cuda_fail(e, "delta step launch");
+}
+
+size_t cd_delta_chunk_workspace_bytes(const cd_delta_attn* a) {
+  return delta_args_ok(a) == CD_OK && delta_chunk_supported(*a) ? delta_chunk_workspace_bytes(*a) : 0;
+}
+
+int cd_delta_chunk(const cd_delta_attn* a, void* ws, size_t ws_bytes, void* stream) {
+  const int st = delta_args_ok(a);
+  if (st != CD_OK) return st;
+  if (!delta_chunk_supported(*a)) return CD_ERR_UNSUPPORTED;
+  if (!a->act || !a->inv || !a->o_raw || !ws || !aligned16(ws) || ws_bytes < delta_chunk_workspace_bytes(*a))
+    return CD_ERR_INVALID;
+  cudaError_t e = launch_delta_chunk(*a, ws, as_stream(stream));
+  return e == cudaSuccess ? CD_OK : cuda_fail(e, "delta chunk launch");
+}
+
 int cd_delta_finish(const cd_delta_attn* a, int fp32, void* stream) {
   const int st = delta_args_ok(a);
   if (st != CD_OK) return st;

@@ -157,6 +157,133 @@ delta_sequence_kernel(const DeltaParams p) {
   }
 }
 
+// ---------------------------------------------------------------- one token
+// Sum of the warps' values; every thread gets it (s: one float per warp; a barrier on both sides)
+__device__ __forceinline__ float block_add(float v, float* s) {
+  v = warp_add(v);
+  __syncthreads();
+  if ((threadIdx.x & 31) == 0) s[threadIdx.x >> 5] = v;
+  __syncthreads();
+  float t = 0.f;
+#pragma unroll
+  for (int w = 0; w < kThreads / 32; ++w) t += s[w];
+  return t;
+}
+
+// A block per head and sequence does the whole step: convolution, norms, decay, recurrence, head norm,
+// gate.  A thread keeps RP rows of four columns of the state in registers (loaded before anything
+// else), so the state is read and written once: with a = (g S)^T k and o = (g S)^T q from one pass,
+// u = beta (v - a), the new state is g S + k u^T and the result o + (k . q) u.
+template <typename T, int RP>
+__global__ void __launch_bounds__(kThreads)
+delta_step_kernel(const DeltaParams p) {
+  extern __shared__ float sm[];
+  __shared__ float s_red[kThreads / 32];
+  pdl_enter();
+  const int h = blockIdx.x, b = blockIdx.y, rep = p.H / p.G, g = h / rep, tid = threadIdx.x;
+  const int dkp = p.dkp, dvp = p.dvp, C = delta_channels(p);
+  float* sq = sm;                  // [dkp]
+  float* sk = sq + dkp;
+  float* sg = sk + dkp;            // decays
+  float* sv = sg + dkp;            // [dvp] v, then u
+  float* so = sv + dvp;            // [dvp] result
+  float* sp = so + dvp;            // [2][row groups][dvp] partial sums
+  const int cgs = dvp / 4, rgs = kThreads / cgs, rg = tid / cgs, col = (tid - rg * cgs) * 4;
+  const bool live = rg < rgs;
+  float* S = p.state + (static_cast<long long>(b) * p.H + h) * dkp * dvp + col;
+  float4 s[RP];
+#pragma unroll
+  for (int m = 0; m < RP; ++m) {
+    const int r = rg + m * rgs;
+    s[m] = (live && r < dkp) ? *reinterpret_cast<const float4*>(S + static_cast<long long>(r) * dvp)
+                             : make_float4(0.f, 0.f, 0.f, 0.f);
+  }
+  const int pos = first_position(p);
+  const T* ring = static_cast<const T*>(p.ring) + static_cast<long long>(b) * p.taps * C;
+  T* here = static_cast<T*>(p.ring) + (static_cast<long long>(b) * p.taps + pos % p.taps) * C;
+  const T* taps = static_cast<const T*>(p.taps_w);
+  // one channel after convolution and silu; `keep`: this block brings the ring up to date
+  auto conv = [&](const T* src, int c, int channel, bool keep) {
+    const T x = src[b * p.ldp + c];
+    float y = to_f32(taps[static_cast<long long>(p.taps - 1) * C + channel]) * to_f32(x);
+    for (int j = 1; j < p.taps && j <= pos; ++j)
+      y = fmaf(to_f32(taps[static_cast<long long>(p.taps - 1 - j) * C + channel]),
+               to_f32(ring[static_cast<long long>((pos - j) % p.taps) * C + channel]), y);
+    if (keep) here[channel] = x;
+    return to_f32(from_f32<T>(silu_precise(y)));
+  };
+  const bool first = h % rep == 0;
+  const float rate = p.rate[h];
+  const float* zg = p.zg + b * p.ldz;
+  float qq = 0.f, kk = 0.f, kq = 0.f;
+  for (int c = tid; c < dkp; c += kThreads) {
+    const float q = conv(static_cast<const T*>(p.q) + g * dkp, c, g * dkp + c, first);
+    const float k = conv(static_cast<const T*>(p.k) + g * dkp, c, (p.G + g) * dkp + c, first);
+    sq[c] = q;
+    sk[c] = k;
+    qq += q * q;
+    kk += k * k;
+    kq += k * q;
+    sg[c] = expf(-rate * softplus_precise(zg[h * dkp + c] + p.dt_bias[h * dkp + c]));
+  }
+  for (int c = tid; c < dvp; c += kThreads)
+    sv[c] = conv(static_cast<const T*>(p.v) + h * dvp, c, 2 * p.G * dkp + h * dvp + c, true);
+  qq = block_add(qq, s_red);
+  kk = block_add(kk, s_red);
+  kq = block_add(kq, s_red);
+  const float iq = 1.0f / sqrtf(static_cast<float>(p.dk)) / sqrtf(qq + 1e-6f), ik = 1.0f / sqrtf(kk + 1e-6f);
+  const float beta = sigmoid_precise(to_f32(static_cast<const T*>(p.b)[b * p.ldp + h]));
+  kq *= iq * ik;
+  float4 a = make_float4(0.f, 0.f, 0.f, 0.f), o = a;
+  if (live) {
+#pragma unroll
+    for (int m = 0; m < RP; ++m) {
+      const int r = rg + m * rgs;
+      if (r < dkp) {
+        const float f = sg[r], k = sk[r] * ik, q = sq[r] * iq;
+        s[m].x *= f; s[m].y *= f; s[m].z *= f; s[m].w *= f;
+        a.x = fmaf(s[m].x, k, a.x); a.y = fmaf(s[m].y, k, a.y); a.z = fmaf(s[m].z, k, a.z); a.w = fmaf(s[m].w, k, a.w);
+        o.x = fmaf(s[m].x, q, o.x); o.y = fmaf(s[m].y, q, o.y); o.z = fmaf(s[m].z, q, o.z); o.w = fmaf(s[m].w, q, o.w);
+      }
+    }
+    *reinterpret_cast<float4*>(sp + rg * dvp + col) = a;
+    *reinterpret_cast<float4*>(sp + (rgs + rg) * dvp + col) = o;
+  }
+  __syncthreads();
+  float ss = 0.f;
+  for (int c = tid; c < dvp; c += kThreads) {
+    float x = 0.f, y = 0.f;
+    for (int r = 0; r < rgs; ++r) {
+      x += sp[r * dvp + c];
+      y += sp[(rgs + r) * dvp + c];
+    }
+    const float u = beta * (sv[c] - x);
+    sv[c] = u;
+    y = fmaf(kq, u, y);
+    so[c] = y;
+    ss += y * y;
+  }
+  ss = block_add(ss, s_red);
+  if (live) {
+    const float4 u = *reinterpret_cast<const float4*>(sv + col);
+#pragma unroll
+    for (int m = 0; m < RP; ++m) {
+      const int r = rg + m * rgs;
+      if (r < dkp) {
+        const float k = sk[r] * ik;
+        s[m].x = fmaf(k, u.x, s[m].x); s[m].y = fmaf(k, u.y, s[m].y);
+        s[m].z = fmaf(k, u.z, s[m].z); s[m].w = fmaf(k, u.w, s[m].w);
+        *reinterpret_cast<float4*>(S + static_cast<long long>(r) * dvp) = s[m];
+      }
+    }
+  }
+  const float r = 1.0f / sqrtf(ss / static_cast<float>(p.dv) + p.eps);
+  T* out = static_cast<T*>(p.out) + b * p.ldo + static_cast<long long>(h) * dvp;
+  for (int c = tid; c < dvp; c += kThreads)
+    out[c] = from_f32<T>(so[c] * r * to_f32(static_cast<const T*>(p.norm_w)[c]) *
+                         sigmoid_precise(zg[p.H * dkp + h * dvp + c]) * p.out_scale);
+}
+
 // ---------------------------------------------------------------- head norm and gate
 // one warp per (row, head)
 template <typename T>
@@ -206,7 +333,33 @@ cudaError_t launch_sequence(const DeltaParams& p, cudaStream_t st) {
   return cudaErrorInvalidValue;
 }
 
+int step_rows(const DeltaParams& p) {       // rows of the state per thread
+  const int rgs = kThreads / (p.dvp / 4);
+  return rgs > 0 ? (p.dkp + rgs - 1) / rgs : 1 << 20;
+}
+
+template <typename T>
+cudaError_t launch_step(const DeltaParams& p, cudaStream_t st) {
+  const int rgs = kThreads / (p.dvp / 4), rp = step_rows(p);
+  const size_t bytes = (3 * p.dkp + 2 * p.dvp + 2 * rgs * p.dvp) * sizeof(float);
+  const dim3 grid(p.H, p.B), block(kThreads);
+  if (rp <= 4) return launch_kernel(delta_step_kernel<T, 4>, grid, block, bytes, st, p);
+  if (rp <= 8) return launch_kernel(delta_step_kernel<T, 8>, grid, block, bytes, st, p);
+  if (rp <= 16) return launch_kernel(delta_step_kernel<T, 16>, grid, block, bytes, st, p);
+  if (rp <= 32) return launch_kernel(delta_step_kernel<T, 32>, grid, block, bytes, st, p);
+  return cudaErrorInvalidValue;
+}
+
 }  // namespace
+
+bool delta_step_supported(const DeltaParams& p) {
+  return p.S == 1 && p.dvp <= 4 * kThreads && step_rows(p) <= 32;
+}
+
+cudaError_t launch_delta_step(const DeltaParams& p, int fp32, cudaStream_t st) {
+  if (p.B == 0) return cudaSuccess;
+  return fp32 ? launch_step<float>(p, st) : launch_step<bf16>(p, st);
+}
 
 bool delta_supported(const DeltaParams& p) { return p.dkp <= 512 && p.B <= 65535; }
 

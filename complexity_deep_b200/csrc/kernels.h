@@ -143,6 +143,11 @@ cudaError_t launch_latent_prefill(const cd_latent_attn& p, const void* expanded,
 bool delta_supported(const cd_delta_attn& p);
 cudaError_t launch_delta_prepare(const cd_delta_attn& p, int fp32, cudaStream_t stream);
 cudaError_t launch_delta_sequence(const cd_delta_attn& p, int fp32, cudaStream_t stream);
+bool delta_step_supported(const cd_delta_attn& p);
+cudaError_t launch_delta_step(const cd_delta_attn& p, int fp32, cudaStream_t stream);
+bool delta_chunk_supported(const cd_delta_attn& p);                          // delta_rule_chunk.cu
+size_t delta_chunk_workspace_bytes(const cd_delta_attn& p);
+cudaError_t launch_delta_chunk(const cd_delta_attn& p, void* ws, cudaStream_t stream);
 cudaError_t launch_delta_finish(const cd_delta_attn& p, int fp32, cudaStream_t stream);
 cudaError_t launch_route_top(const float* logits, long long ld, int T, int E, int count, int keep, int top,
                              long long* ids, float* weights, cudaStream_t stream);

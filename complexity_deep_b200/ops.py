@@ -1156,6 +1156,9 @@ def latent_attention_(proj: dict, out: torch.Tensor, weights: dict, cache: torch
         _lib.check(lib.cd_latent_rows(ref, fp32, _stream()), "cd_latent_rows")
 
 
+_DELTA_CHUNK_MIN = 16       # shorter portions walk token by token
+
+
 def delta_attention_(proj: dict, out: torch.Tensor, weights: dict, ring: torch.Tensor, state: torch.Tensor, *,
                      batch: int, seq_len: int, heads: int, kv_heads: int, dim: int, vdim: int, eps: float,
                      out_scale: float, pos0: int, pos_dev: Optional[torch.Tensor] = None) -> None:
@@ -1186,20 +1189,32 @@ def delta_attention_(proj: dict, out: torch.Tensor, weights: dict, ring: torch.T
         raise RuntimeError("delta rule: inner weights do not match the head layout")
     _need_pos_dev(pos_dev)
     zg = linear_to_f32(proj["inner"], weights["inner"], tag="delta_inner")
-    act = torch.empty(T, C, dtype=dt, device=out.device)
-    inv = torch.empty(T, 2 * kv_heads, dtype=torch.float32, device=out.device)
-    o_raw = torch.empty(T, heads * dvp, dtype=torch.float32, device=out.device)
     a = _lib.DeltaAttn(
         q=_columns(proj["q"], "q", dt), k=_columns(proj["k"], "k", dt), v=_columns(proj["v"], "v", dt),
         b=_columns(proj["b"], "b", dt), ldp=proj["b"].stride(0), zg=zg.data_ptr(), ldz=zg.shape[1],
         taps_w=weights["taps"].data_ptr(), rate=weights["rate"].data_ptr(), dt_bias=weights["dt_bias"].data_ptr(),
         norm_w=weights["norm"].data_ptr(), ring=ring.data_ptr(), state=state.data_ptr(),
-        out=_columns(out, "out", dt), ldo=out.stride(0), act=act.data_ptr(), inv=inv.data_ptr(),
-        o_raw=o_raw.data_ptr(), pos_dev=_ptr(pos_dev), eps=float(eps), out_scale=float(out_scale), B=batch,
+        out=_columns(out, "out", dt), ldo=out.stride(0), pos_dev=_ptr(pos_dev), eps=float(eps), out_scale=float(out_scale), B=batch,
         S=seq_len, H=heads, G=kv_heads, dk=dim, dkp=dkp, dv=vdim, dvp=dvp, taps=taps, pos0=pos0)
     ref = ctypes.byref(a)
+    if seq_len == 1 and lib.cd_delta_step_supported(ref):
+        with _Span("delta_step"):
+            _lib.check(lib.cd_delta_step(ref, fp32, _stream()), "cd_delta_step")
+        return
+    act = torch.empty(T, C, dtype=dt, device=out.device)
+    inv = torch.empty(T, 2 * kv_heads, dtype=torch.float32, device=out.device)
+    o_raw = torch.empty(T, heads * dvp, dtype=torch.float32, device=out.device)
+    a.act, a.inv, a.o_raw = act.data_ptr(), inv.data_ptr(), o_raw.data_ptr()
     with _Span("delta_prepare"):
         _lib.check(lib.cd_delta_prepare(ref, fp32, _stream()), "cd_delta_prepare")
+    ws_bytes = 0 if fp32 or seq_len < _DELTA_CHUNK_MIN else lib.cd_delta_chunk_workspace_bytes(ref)
+    if ws_bytes:
+        ws = torch.empty(ws_bytes, dtype=torch.uint8, device=out.device)
+        with _Span("delta_chunk", 2):
+            _lib.check(lib.cd_delta_chunk(ref, ws.data_ptr(), ws_bytes, _stream()), "cd_delta_chunk")
+        with _Span("delta_finish"):
+            _lib.check(lib.cd_delta_finish(ref, fp32, _stream()), "cd_delta_finish")
+        return
     with _Span("delta_sequence"):
         _lib.check(lib.cd_delta_sequence(ref, fp32, _stream()), "cd_delta_sequence")
     with _Span("delta_finish"):

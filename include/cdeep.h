@@ -571,10 +571,18 @@ typedef struct cd_delta_attn {
 } cd_delta_attn;
 
 int cd_delta_supported(const cd_delta_attn* h_args);
+/* One token per sequence (S = 1) in one kernel, convolution to gate (no scratch needed); for heads whose
+ * state fits the registers of a block (cd_delta_step_supported). */
+int cd_delta_step_supported(const cd_delta_attn* h_args);
+int cd_delta_step(const cd_delta_attn* h_args, int fp32, void* stream);
 /* Convolution, silu and the norms of q and k; brings the ring up to date. */
 int cd_delta_prepare(const cd_delta_attn* h_args, int fp32, void* stream);
 /* Walks the tokens one by one (o_raw, state). */
 int cd_delta_sequence(const cd_delta_attn* h_args, int fp32, void* stream);
+/* The same in bf16 in chunks of 64 tokens on the tensor cores.  The workspace size is 0 where the form does
+ * not apply (key heads wider than 128, value heads wider than 256). */
+size_t cd_delta_chunk_workspace_bytes(const cd_delta_attn* h_args);
+int cd_delta_chunk(const cd_delta_attn* h_args, void* workspace, size_t bytes, void* stream);
 /* Head norm and gate on o_raw. */
 int cd_delta_finish(const cd_delta_attn* h_args, int fp32, void* stream);
 
