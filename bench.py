@@ -1030,8 +1030,9 @@ def pimezen_work(z: dict, T: int, S: int) -> dict:
     }
 
 
-def pimezen_bench(z: dict, make, args, dev) -> dict:
-    """Prefill and decode throughput and the time of every kernel of one model."""
+def pimezen_bench(z: dict, make, args, dev, work_of=pimezen_work) -> dict:
+    """Prefill and decode throughput and the time of every kernel of one model; work_of(z, T, S) gives
+    (FLOP, bytes) of one launch by its name."""
     from complexity_deep_b200 import ops
     from complexity_deep_b200.models import DecodeGraph, PrefillGraph
     model, pk, out = make(z, dev), peaks(), {}
@@ -1057,7 +1058,7 @@ def pimezen_bench(z: dict, make, args, dev) -> dict:
             fn()
         prof = ops.PROFILE.collect()
         ops.PROFILE.reset(enabled=False)
-        work, res = pimezen_work(z, T, S), {}
+        work, res = work_of(z, T, S), {}
         for name, (calls, ms, _) in prof.items():
             us = ms / calls * 1e3
             res[name] = {"us": round(us, 1), "calls_per_step": calls // 3}
@@ -1082,7 +1083,8 @@ def pimezen_bench(z: dict, make, args, dev) -> dict:
             dec.cache.length = P
             if hasattr(dec.cache, "position"):
                 dec.cache.position.fill_(P)
-                tensors = [t for layer in dec.cache.layers for t in (layer["left"].k, layer["left"].v)]
+                tensors = [t for layer in dec.cache.layers for part in layer.values() for name in ("k", "v", "rows")
+                           for t in [getattr(part, name, None)] if t is not None]
             else:
                 dec.cache.set_length(P)
                 tensors = dec.cache.k + dec.cache.v
@@ -1121,6 +1123,128 @@ def run_pimezen(args):
                       "clocks": sampler.stop(), "sizes": sizes}), flush=True)
 
 
+# ---------------------------------------------------------------- Rugedra beside its closest models
+RUGEDRA_SIZES = {
+    # width, heads (128 + 64 rotated, values 128), latent, delta heads (128 x 128), experts of which `top` are
+    # used, ff (of the dense layer; an expert has ff / top)
+    "w1024": dict(width=1024, heads=8, kv=8, rank=512, d_heads=8, experts=32, top=4, ff=2816, layers=8),
+    "w2048": dict(width=2048, heads=16, kv=16, rank=512, d_heads=16, experts=64, top=8, ff=5632, layers=8),
+}
+RUGEDRA_LATENT_LAYERS = (0, 4)        # the others carry the delta rule; layer 0 is dense, the others have experts
+
+
+def rugedra_model(z: dict, device):
+    """Random weights of a Rugedra model of the size `z`."""
+    from complexity_deep_b200.models import RugedraConfig, RugedraModel
+    moe = {"kind": "moe", "expert": {"ff": z["ff"] // z["top"], "limit": 7.0},
+           "router": {"experts": z["experts"], "top": z["top"], "groups": {"count": 8, "keep": 4}}}
+    latent = {"heads": z["heads"], "dim": 128, "rot_dim": 64, "vdim": 128, "kv_rank": z["rank"], "scale": 192 ** -0.5,
+              "rot": {"base": 1e4, "dims": 64}}
+    delta = {"heads": z["d_heads"], "kv_heads": z["d_heads"], "dim": 128, "vdim": 128, "conv": 4}
+    layers = [{"type": "latent_attention" if i in RUGEDRA_LATENT_LAYERS else "channel_delta",
+               "mixer": latent if i in RUGEDRA_LATENT_LAYERS else delta,
+               "mlp": {"kind": "dense", "ff": z["ff"]} if i == 0 else moe} for i in range(z["layers"])]
+    cfg = RugedraConfig.from_dict({"architecture": "Rugedra", "vocab": PIMEZEN_VOCAB, "width": z["width"],
+                                   "max_positions": 8192, "norm": {"eps": 1e-6}, "residual_mult": 0.5,
+                                   "logit_scale": 1.0, "layers": layers})
+    for layer in cfg.layers:
+        if hasattr(layer.mixer, "gate_rank"):
+            layer.mixer.rank = layer.mixer.gate_rank = 128
+    torch.manual_seed(0)
+    with torch.device(device):
+        model = RugedraModel(cfg)
+    for name, p in model.named_parameters():
+        if name.endswith("_conv"):
+            torch.nn.init.normal_(p, std=0.5)
+        elif name.endswith("dt_bias"):
+            torch.nn.init.uniform_(p, -5.0, 0.0)
+    return model.to(torch.bfloat16).requires_grad_(False).eval()
+
+
+def rugedra_work(z: dict, T: int, S: int) -> dict:
+    """name -> (FLOP, bytes) of one launch at T tokens (S per sequence; S = 1: a decode step at 2 048 cached)."""
+    W, H, R, D, E, top, ff = (z[k] for k in ("width", "heads", "rank", "d_heads", "experts", "top", "ff"))
+    V, fe, P = PIMEZEN_VOCAB, z["ff"] // z["top"], PIMEZEN_PREFILL[1]
+    n_lat = len(RUGEDRA_LATENT_LAYERS)
+    gemm = lambda k, n, out, t=T: (2 * t * k * n, 2 * (t * k + k * n) + out * t * n)
+    mean = lambda a, b: tuple((n_lat * x + (z["layers"] - n_lat) * y) / z["layers"] for x, y in zip(a, b))
+    used = min(E, T * top)                  # experts whose weights are read
+    return {
+        "mixer_in": mean(gemm(W, H * 192 + R + 64, 2), gemm(W, D * 384 + D + 256, 2)),
+        "mixer_out": mean(gemm(H * 128, W, 8), gemm(D * 128, W, 8)),
+        "relu2_up": gemm(W, ff, 2), "relu2_down": gemm(ff, W, 8), "linear_lm_head": gemm(W, V, 4),
+        "router": gemm(W, E, 4), "layernorm_f32": (0, T * W * 6),
+        "gather_div": (0, T * (1 + top) * W * 2), "combine_top": (0, T * top * W * 2 + T * W * 8),
+        "glu_up_routed": (4 * T * top * W * fe, 2 * (T * top * (W + fe) + 2 * used * W * fe)),
+        "moe_down": (2 * T * top * W * fe, 2 * (T * top * (W + fe) + used * W * fe)),
+        "latent_prepare": (0, T * (H * 64 * 4 + (R + 64) * 4 + R * 2)),
+        "latent_expand": gemm(R, H * 256, 2),
+        "latent_prefill": (2 * T * (S + 1) / 2 * H * 320, T * H * (192 + 256 + 128) * 2),
+        "latent_decode": (2 * T * P * H * (2 * R + 64), T * P * (R + 64) * 2 + H * 256 * R * 2),
+        "delta_inner": gemm(256, D * 256, 4),
+        "delta_prepare": (0, T * D * 384 * 4),
+        # q, k, v, decay inputs in, result out (the state stays on chip in an ideal kernel)
+        "delta_chunk": (2 * T * D * 128 * 128 * 3, T * D * 128 * (3 * 2 + 4 + 4)),
+        "delta_finish": (0, T * D * 128 * (4 + 4 + 2)), "delta_step": (0, T * D * 128 * 128 * 8),
+    }
+
+
+def moe_complexity_model(z: dict, device):
+    """The reference's model at the same width and heads: attention over the whole sequence, experts routed
+    by token id beside a shared one, no mu guidance."""
+    import complexity_deep_b200 as cd
+    cfg = cd.ComplexityConfig(vocab_size=PIMEZEN_VOCAB, hidden_size=z["width"], intermediate_size=z["ff"],
+                              num_hidden_layers=z["layers"], num_attention_heads=z["heads"],
+                              num_key_value_heads=z["kv"] // 2, max_position_embeddings=8192,
+                              use_token_routed_mlp=True, num_experts=8, use_mu_guidance=False)
+    torch.manual_seed(0)
+    with torch.device(device):
+        model = cd.ComplexityModel(cfg)
+    return model.to(torch.bfloat16).requires_grad_(False).eval()
+
+
+def moe_complexity_work(z: dict, T: int, S: int) -> dict:
+    W, H, G, ff, V = z["width"], z["heads"], z["kv"] // 2, z["ff"], PIMEZEN_VOCAB
+    I, P = ff // 8, PIMEZEN_PREFILL[1]
+    gemm = lambda k, n, out: (2 * T * k * n, 2 * (T * k + k * n) + out * T * n)
+    return {
+        "mu_qkv": gemm(W, (H + 2 * G) * 128, 2), "linear_o_proj": gemm(H * 128, W, 6), "linear_lm_head": gemm(W, V, 2),
+        "rmsnorm": (0, T * W * 6), "rmsnorm_split": (0, T * W * 6),
+        "moe_up_pair": (8 * T * W * I, 2 * (T * W + 2 * 9 * W * I + 2 * T * I)),
+        "moe_up_routed": (4 * T * W * I, 2 * (T * W + 2 * 8 * W * I + T * I)),
+        "moe_up_shared": (4 * T * W * I, 2 * (T * W + 2 * W * I + T * I)),
+        "moe_down": (4 * T * W * I, 2 * (2 * T * I + 9 * W * I + 4 * T * W)),
+        "attention_prefill": (2 * T * (S + 1) / 2 * H * 256, T * (2 * H + 2 * G) * 256),
+        "decode_attention": (0, T * P * G * 512),
+    }
+
+
+def run_rugedra(args):
+    """Prefill and decode of Rugedra models (random weights) beside the two closest models at the same
+    width: the expert-routed Complexity model (attention, experts) and Pimezen (recurrent mixer, fp32
+    stream); decode starts at 2 048 tokens."""
+    dev = torch.device("cuda", 0)
+    torch.cuda.set_device(dev)
+    sampler = ClockSampler(0)
+    sampler.start()
+    sizes = {}
+    for name, z in RUGEDRA_SIZES.items():
+        if args.rugedra_size not in ("all", name):
+            continue
+        sizes[name] = {"config": z, "rugedra": pimezen_bench(z, rugedra_model, args, dev, rugedra_work)}
+        if not args.rugedra_alone:
+            sizes[name]["moe_complexity"] = pimezen_bench(z, moe_complexity_model, args, dev, moe_complexity_work)
+            sizes[name]["pimezen"] = pimezen_bench(PIMEZEN_SIZES[name], pimezen_model, args, dev)
+        torch.cuda.empty_cache()
+    last = sizes[list(sizes)[-1]]["rugedra"]["prefill"]
+    print(json.dumps({"metric": "prefill tokens/s (Rugedra, bf16)", "value": last["tokens_per_s"], "unit": "tokens/s",
+                      "n_gpus": 1, "steps": args.steps, "warmup": args.warmup, "ms_per_step": last["ms"],
+                      "higher_is_better": True, "dtype": "bf16", "data": "synthetic", "impl": "b200",
+                      "config": {"workload": "rugedra", "vocab": PIMEZEN_VOCAB,
+                                 "inputs": "weights and activations of a step exceed L2"},
+                      "clocks": sampler.stop(), "sizes": sizes}), flush=True)
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -1146,10 +1270,13 @@ def main():
     ap.add_argument("--cache-len", type=int, default=4096, help="decode_1b: prefilled KV tokens")
     ap.add_argument("--seq-len", type=int, default=SEQ_LEN, help="attn_prefill: sequence length")
     ap.add_argument("--workload", default="prefill_1b",
-                    choices=["prefill_1b", "decode_1b", "attn_prefill", "pimezen"] + list(LAYER_CONFIGS),
+                    choices=["prefill_1b", "decode_1b", "attn_prefill", "pimezen", "rugedra"] + list(LAYER_CONFIGS),
                     help="prefill_1b is the headline; the layer modes report MoE-layer TFLOP/s")
     ap.add_argument("--pimezen-size", default="all", choices=["all"] + list(PIMEZEN_SIZES),
                     help="pimezen: which size to run")
+    ap.add_argument("--rugedra-size", default="all", choices=["all"] + list(RUGEDRA_SIZES),
+                    help="rugedra: which size to run")
+    ap.add_argument("--rugedra-alone", action="store_true", help="rugedra: leave out the models beside it")
     args = ap.parse_args()
     if args.warmup < 3 and args.impl == "b200":
         args.warmup = 3
@@ -1163,6 +1290,8 @@ def main():
         run_attention(args)
     elif args.workload == "pimezen":
         run_pimezen(args)
+    elif args.workload == "rugedra":
+        run_rugedra(args)
     elif args.workload != "prefill_1b":
         run_layer(args)
     else:

@@ -68,6 +68,75 @@ delta_prepare_kernel(const DeltaParams p, int run) {
       }
 }
 
+// The usual sizes: up to four taps and heads up to 8 GL wide.  A group of GL lanes takes kRun tokens of one
+// head; a lane's eight channels of all of them are loaded up front and pass through a window in registers.
+constexpr int kRun = 8;
+constexpr int kWindow = 4;
+
+template <typename T, int GL>
+__global__ void __launch_bounds__(kThreads)
+delta_prepare_window_kernel(const DeltaParams p) {
+  pdl_enter();
+  const int slots = 2 * p.G + p.H, C = delta_channels(p), b = blockIdx.y;
+  const int runs = (p.S + kRun - 1) / kRun;
+  const int item = (blockIdx.x * kThreads + threadIdx.x) / GL, c = (threadIdx.x % GL) * 8;
+  const bool live = item < runs * slots;                    // idle groups stay for the shuffles
+  const int slot = live ? item % slots : 0, t0 = live ? item / slots * kRun : p.S;
+  const bool is_v = slot >= 2 * p.G;
+  const int width = is_v ? p.dvp : p.dkp;
+  const bool ok = live && c < width;
+  const int col = (is_v ? 2 * p.G * p.dkp + (slot - 2 * p.G) * p.dvp : slot * p.dkp) + c;
+  const T* src = static_cast<const T*>(is_v ? p.v : slot < p.G ? p.q : p.k) +
+                 (is_v ? (slot - 2 * p.G) * p.dvp : (slot < p.G ? slot : slot - p.G) * p.dkp) + c;
+  const long long row0 = static_cast<long long>(b) * p.S;
+  const T* taps = static_cast<const T*>(p.taps_w) + col;
+  T* ring = static_cast<T*>(p.ring) + static_cast<long long>(b) * p.taps * C + col;
+  const int pos0 = first_position(p);
+  Raw8<T> raw[kRun + kWindow - 1] = {};                     // tokens t0 - 3 ...
+#pragma unroll
+  for (int x = 0; x < kRun + kWindow - 1; ++x) {
+    const int t = t0 + x - (kWindow - 1);
+    if (!ok || t >= p.S || pos0 + t < 0) continue;
+    if (t >= 0) raw_load(src + (row0 + t) * p.ldp, raw[x]);
+    else if (-t < p.taps) raw_load(ring + static_cast<long long>((pos0 + t) % p.taps) * C, raw[x]);
+  }
+  float w[kWindow][8] = {};                                 // w[j]: j tokens back
+#pragma unroll
+  for (int j = 0; j < kWindow; ++j)
+    if (ok && j < p.taps) load8(taps + static_cast<long long>(p.taps - 1 - j) * C, w[j]);
+  float win[kWindow][8] = {};
+#pragma unroll
+  for (int x = 0; x < kWindow - 1; ++x) raw_unpack(raw[x], win[(x + 1) % kWindow]);
+  const float scale = slot < p.G ? 1.0f / sqrtf(static_cast<float>(p.dk)) : 1.0f;
+#pragma unroll
+  for (int x = 0; x < kRun; ++x) {
+    const int t = t0 + x;                                   // its input goes to window slot x % 4
+    raw_unpack(raw[x + kWindow - 1], win[x % kWindow]);
+    float y[8] = {}, ss = 0.f;
+#pragma unroll
+    for (int j = kWindow - 1; j >= 0; --j)
+#pragma unroll
+      for (int e = 0; e < 8; ++e) y[e] = fmaf(w[j][e], win[(x - j + kWindow) % kWindow][e], y[e]);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) {
+      y[e] = to_f32(from_f32<T>(sizeof(T) == 2 ? y[e] / (1.0f + exp2_approx(-1.4426950408889634f * y[e])) : silu_precise(y[e])));
+      ss += y[e] * y[e];
+    }
+#pragma unroll
+    for (int o = GL / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+    if (ok && t < p.S) {
+      store8(static_cast<T*>(p.act) + (row0 + t) * C + col, y);
+      if (!is_v && c == 0) p.inv[(row0 + t) * 2 * p.G + slot] = scale / sqrtf(ss + 1e-6f);
+    }
+  }
+  if (ok && t0 == 0)
+    for (int t = max(0, p.S - p.taps); t < p.S; ++t) {
+      float x[8];
+      load8(src + (row0 + t) * p.ldp, x);
+      store8(ring + static_cast<long long>((pos0 + t) % p.taps) * C, x);
+    }
+}
+
 // ---------------------------------------------------------------- token by token
 constexpr int kSteps = 16;     // tokens staged in shared memory at a time
 constexpr int kCols = 32;      // state columns per block, four per warp
@@ -158,16 +227,54 @@ delta_sequence_kernel(const DeltaParams p) {
 }
 
 // ---------------------------------------------------------------- one token
-// Sum of the warps' values; every thread gets it (s: one float per warp; a barrier on both sides)
-__device__ __forceinline__ float block_add(float v, float* s) {
-  v = warp_add(v);
-  __syncthreads();
-  if ((threadIdx.x & 31) == 0) s[threadIdx.x >> 5] = v;
-  __syncthreads();
-  float t = 0.f;
+// Sums of N values over the block; every thread gets them (a barrier on both sides)
+template <int N>
+__device__ __forceinline__ void block_add(float (&v)[N], float* s) {
 #pragma unroll
-  for (int w = 0; w < kThreads / 32; ++w) t += s[w];
-  return t;
+  for (int x = 0; x < N; ++x) v[x] = warp_add(v[x]);
+  __syncthreads();
+  if ((threadIdx.x & 31) == 0) {
+#pragma unroll
+    for (int x = 0; x < N; ++x) s[x * (kThreads / 32) + (threadIdx.x >> 5)] = v[x];
+  }
+  __syncthreads();
+#pragma unroll
+  for (int x = 0; x < N; ++x) {
+    v[x] = 0.f;
+#pragma unroll
+    for (int w = 0; w < kThreads / 32; ++w) v[x] += s[x * (kThreads / 32) + w];
+  }
+}
+
+// A channel's convolution inputs of one token, loaded before any is used
+template <typename T>
+struct ConvTap {
+  T x[kWindow], w[kWindow];
+};
+template <typename T>
+__device__ __forceinline__ void conv_load(const DeltaParams& p, const T* now, const T* ring, int channel, int C, int pos,
+                                          ConvTap<T>& r) {
+  const T* taps = static_cast<const T*>(p.taps_w) + channel;
+  r.x[0] = *now;
+  r.w[0] = taps[static_cast<long long>(p.taps - 1) * C];
+#pragma unroll
+  for (int j = 1; j < kWindow; ++j) {
+    const bool ok = j < p.taps && j <= pos;
+    r.x[j] = ok ? ring[static_cast<long long>((pos - j) % p.taps) * C + channel] : from_f32<T>(0.f);
+    r.w[j] = ok ? taps[static_cast<long long>(p.taps - 1 - j) * C] : from_f32<T>(0.f);
+  }
+}
+template <typename T>
+__device__ __forceinline__ float conv_value(const DeltaParams& p, const T* ring, int channel, int C, int pos,
+                                            const ConvTap<T>& r) {
+  float y = 0.f;
+  for (int j = p.taps - 1; j >= kWindow; --j)               // more taps than the window holds
+    if (j <= pos)
+      y = fmaf(to_f32(static_cast<const T*>(p.taps_w)[static_cast<long long>(p.taps - 1 - j) * C + channel]),
+               to_f32(ring[static_cast<long long>((pos - j) % p.taps) * C + channel]), y);
+#pragma unroll
+  for (int j = kWindow - 1; j >= 0; --j) y = fmaf(to_f32(r.w[j]), to_f32(r.x[j]), y);
+  return to_f32(from_f32<T>(silu_precise(y)));
 }
 
 // A block per head and sequence does the whole step: convolution, norms, decay, recurrence, head norm,
@@ -175,10 +282,10 @@ __device__ __forceinline__ float block_add(float v, float* s) {
 // else), so the state is read and written once: with a = (g S)^T k and o = (g S)^T q from one pass,
 // u = beta (v - a), the new state is g S + k u^T and the result o + (k . q) u.
 template <typename T, int RP>
-__global__ void __launch_bounds__(kThreads)
+__global__ void __launch_bounds__(kThreads, RP <= 16 ? 2 : 1)
 delta_step_kernel(const DeltaParams p) {
   extern __shared__ float sm[];
-  __shared__ float s_red[kThreads / 32];
+  __shared__ float s_red[3 * kThreads / 32];
   pdl_enter();
   const int h = blockIdx.x, b = blockIdx.y, rep = p.H / p.G, g = h / rep, tid = threadIdx.x;
   const int dkp = p.dkp, dvp = p.dvp, C = delta_channels(p);
@@ -201,39 +308,45 @@ delta_step_kernel(const DeltaParams p) {
   const int pos = first_position(p);
   const T* ring = static_cast<const T*>(p.ring) + static_cast<long long>(b) * p.taps * C;
   T* here = static_cast<T*>(p.ring) + (static_cast<long long>(b) * p.taps + pos % p.taps) * C;
-  const T* taps = static_cast<const T*>(p.taps_w);
-  // one channel after convolution and silu; `keep`: this block brings the ring up to date
-  auto conv = [&](const T* src, int c, int channel, bool keep) {
-    const T x = src[b * p.ldp + c];
-    float y = to_f32(taps[static_cast<long long>(p.taps - 1) * C + channel]) * to_f32(x);
-    for (int j = 1; j < p.taps && j <= pos; ++j)
-      y = fmaf(to_f32(taps[static_cast<long long>(p.taps - 1 - j) * C + channel]),
-               to_f32(ring[static_cast<long long>((pos - j) % p.taps) * C + channel]), y);
-    if (keep) here[channel] = x;
-    return to_f32(from_f32<T>(silu_precise(y)));
-  };
   const bool first = h % rep == 0;
   const float rate = p.rate[h];
   const float* zg = p.zg + b * p.ldz;
-  float qq = 0.f, kk = 0.f, kq = 0.f;
-  for (int c = tid; c < dkp; c += kThreads) {
-    const float q = conv(static_cast<const T*>(p.q) + g * dkp, c, g * dkp + c, first);
-    const float k = conv(static_cast<const T*>(p.k) + g * dkp, c, (p.G + g) * dkp + c, first);
-    sq[c] = q;
-    sk[c] = k;
-    qq += q * q;
-    kk += k * k;
-    kq += k * q;
-    sg[c] = expf(-rate * softplus_precise(zg[h * dkp + c] + p.dt_bias[h * dkp + c]));
+  float sums[3] = {0.f, 0.f, 0.f};        // |q|^2, |k|^2, k . q
+  for (int c = tid; c < max(dkp, dvp); c += kThreads) {
+    const T* q_in = static_cast<const T*>(p.q) + b * p.ldp + g * dkp + c;
+    const T* k_in = static_cast<const T*>(p.k) + b * p.ldp + g * dkp + c;
+    const T* v_in = static_cast<const T*>(p.v) + b * p.ldp + h * dvp + c;
+    const int qc = g * dkp + c, kc = (p.G + g) * dkp + c, vc = 2 * p.G * dkp + h * dvp + c;
+    ConvTap<T> tq, tk, tv;
+    float z = 0.f;
+    if (c < dkp) {
+      conv_load(p, q_in, ring, qc, C, pos, tq);
+      conv_load(p, k_in, ring, kc, C, pos, tk);
+      z = zg[h * dkp + c] + p.dt_bias[h * dkp + c];
+    }
+    if (c < dvp) conv_load(p, v_in, ring, vc, C, pos, tv);
+    if (c < dkp) {
+      const float q = conv_value(p, ring, qc, C, pos, tq), k = conv_value(p, ring, kc, C, pos, tk);
+      sq[c] = q;
+      sk[c] = k;
+      sums[0] += q * q;
+      sums[1] += k * k;
+      sums[2] += k * q;
+      sg[c] = expf(-rate * softplus_precise(z));
+      if (first) {                        // this block brings the ring up to date
+        here[qc] = tq.x[0];
+        here[kc] = tk.x[0];
+      }
+    }
+    if (c < dvp) {
+      sv[c] = conv_value(p, ring, vc, C, pos, tv);
+      here[vc] = tv.x[0];
+    }
   }
-  for (int c = tid; c < dvp; c += kThreads)
-    sv[c] = conv(static_cast<const T*>(p.v) + h * dvp, c, 2 * p.G * dkp + h * dvp + c, true);
-  qq = block_add(qq, s_red);
-  kk = block_add(kk, s_red);
-  kq = block_add(kq, s_red);
-  const float iq = 1.0f / sqrtf(static_cast<float>(p.dk)) / sqrtf(qq + 1e-6f), ik = 1.0f / sqrtf(kk + 1e-6f);
+  block_add(sums, s_red);
+  const float iq = 1.0f / sqrtf(static_cast<float>(p.dk)) / sqrtf(sums[0] + 1e-6f), ik = 1.0f / sqrtf(sums[1] + 1e-6f);
+  const float kq = sums[2] * iq * ik;
   const float beta = sigmoid_precise(to_f32(static_cast<const T*>(p.b)[b * p.ldp + h]));
-  kq *= iq * ik;
   float4 a = make_float4(0.f, 0.f, 0.f, 0.f), o = a;
   if (live) {
 #pragma unroll
@@ -250,7 +363,7 @@ delta_step_kernel(const DeltaParams p) {
     *reinterpret_cast<float4*>(sp + (rgs + rg) * dvp + col) = o;
   }
   __syncthreads();
-  float ss = 0.f;
+  float ss[1] = {0.f};
   for (int c = tid; c < dvp; c += kThreads) {
     float x = 0.f, y = 0.f;
     for (int r = 0; r < rgs; ++r) {
@@ -261,9 +374,9 @@ delta_step_kernel(const DeltaParams p) {
     sv[c] = u;
     y = fmaf(kq, u, y);
     so[c] = y;
-    ss += y * y;
+    ss[0] += y * y;
   }
-  ss = block_add(ss, s_red);
+  block_add(ss, s_red);
   if (live) {
     const float4 u = *reinterpret_cast<const float4*>(sv + col);
 #pragma unroll
@@ -277,7 +390,7 @@ delta_step_kernel(const DeltaParams p) {
       }
     }
   }
-  const float r = 1.0f / sqrtf(ss / static_cast<float>(p.dv) + p.eps);
+  const float r = 1.0f / sqrtf(ss[0] / static_cast<float>(p.dv) + p.eps);
   T* out = static_cast<T*>(p.out) + b * p.ldo + static_cast<long long>(h) * dvp;
   for (int c = tid; c < dvp; c += kThreads)
     out[c] = from_f32<T>(so[c] * r * to_f32(static_cast<const T*>(p.norm_w)[c]) *
@@ -305,8 +418,65 @@ delta_finish_kernel(const DeltaParams p) {
     out[c] = from_f32<T>(o[c] * r * to_f32(static_cast<const T*>(p.norm_w)[c]) * sigmoid_precise(gate[c]) * p.out_scale);
 }
 
+// heads up to 8 GL wide: a group of GL lanes per (row, head), eight columns per lane
+template <typename T, int GL>
+__global__ void __launch_bounds__(kThreads)
+delta_finish_group_kernel(const DeltaParams p) {
+  pdl_enter();
+  const long long items = static_cast<long long>(p.B) * p.S * p.H;
+  const long long item = (static_cast<long long>(blockIdx.x) * kThreads + threadIdx.x) / GL;
+  const int c = (threadIdx.x % GL) * 8;
+  const bool ok = item < items && c < p.dvp;
+  const long long row = ok ? item / p.H : 0;
+  const int h = ok ? static_cast<int>(item - row * p.H) : 0;
+  float o[8] = {}, gate[8] = {}, w[8] = {}, ss = 0.f;
+  if (ok) {
+    load8(p.o_raw + item * p.dvp + c, o);
+    load8(p.zg + row * p.ldz + p.H * p.dkp + static_cast<long long>(h) * p.dvp + c, gate);
+    load8(static_cast<const T*>(p.norm_w) + c, w);
+  }
+#pragma unroll
+  for (int e = 0; e < 8; ++e) ss += o[e] * o[e];
+#pragma unroll
+  for (int d = GL / 2; d > 0; d >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, d);
+  const float r = p.out_scale / sqrtf(ss / static_cast<float>(p.dv) + p.eps);
+#pragma unroll
+  for (int e = 0; e < 8; ++e)
+    o[e] *= r * w[e] * (sizeof(T) == 2 ? 1.0f / (1.0f + exp2_approx(-1.4426950408889634f * gate[e])) : sigmoid_precise(gate[e]));
+  if (ok) store8(static_cast<T*>(p.out) + row * p.ldo + static_cast<long long>(h) * p.dvp + c, o);
+}
+
+template <typename T, int GL>
+cudaError_t launch_window(const DeltaParams& p, cudaStream_t st) {
+  const long long lanes = static_cast<long long>((p.S + kRun - 1) / kRun) * (2 * p.G + p.H) * GL;
+  return launch_kernel(delta_prepare_window_kernel<T, GL>, dim3(static_cast<unsigned>((lanes + kThreads - 1) / kThreads), p.B),
+                       dim3(kThreads), 0, st, p);
+}
+
+template <typename T, int GL>
+cudaError_t launch_finish_group(const DeltaParams& p, cudaStream_t st) {
+  const long long lanes = static_cast<long long>(p.B) * p.S * p.H * GL;
+  return launch_kernel(delta_finish_group_kernel<T, GL>, dim3(static_cast<unsigned>((lanes + kThreads - 1) / kThreads)),
+                       dim3(kThreads), 0, st, p);
+}
+
+template <typename T>
+cudaError_t launch_finish(const DeltaParams& p, cudaStream_t st) {
+  if (p.dvp <= 64) return launch_finish_group<T, 8>(p, st);
+  if (p.dvp <= 128) return launch_finish_group<T, 16>(p, st);
+  if (p.dvp <= 256) return launch_finish_group<T, 32>(p, st);
+  const long long items = static_cast<long long>(p.B) * p.S * p.H;
+  return launch_kernel(delta_finish_kernel<T>, dim3(static_cast<unsigned>((items + 7) / 8)), dim3(kThreads), 0, st, p);
+}
+
 template <typename T>
 cudaError_t launch_prepare(const DeltaParams& p, cudaStream_t st) {
+  const int widest = p.dkp > p.dvp ? p.dkp : p.dvp;
+  if (p.taps <= kWindow) {
+    if (widest <= 64) return launch_window<T, 8>(p, st);
+    if (widest <= 128) return launch_window<T, 16>(p, st);
+    if (widest <= 256) return launch_window<T, 32>(p, st);
+  }
   const int run = p.taps > 9 ? p.taps - 1 : 8;
   const long long items = static_cast<long long>((p.S + run - 1) / run) * (2 * p.G + p.H);
   return launch_kernel(delta_prepare_kernel<T>, dim3(static_cast<unsigned>((items + 7) / 8), p.B), dim3(kThreads), 0, st,
@@ -376,9 +546,7 @@ cudaError_t launch_delta_sequence(const DeltaParams& p, int fp32, cudaStream_t s
 cudaError_t launch_delta_finish(const DeltaParams& p, int fp32, cudaStream_t st) {
   const long long items = static_cast<long long>(p.B) * p.S * p.H;
   if (items == 0) return cudaSuccess;
-  const dim3 grid(static_cast<unsigned>((items + 7) / 8));
-  return fp32 ? launch_kernel(delta_finish_kernel<float>, grid, dim3(kThreads), 0, st, p)
-              : launch_kernel(delta_finish_kernel<bf16>, grid, dim3(kThreads), 0, st, p);
+  return fp32 ? launch_finish<float>(p, st) : launch_finish<bf16>(p, st);
 }
 
 }  // namespace cdeep

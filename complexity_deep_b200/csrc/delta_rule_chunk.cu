@@ -58,15 +58,14 @@ __device__ __forceinline__ float2 pair_of(const bf16* p) {
 
 // ---------------------------------------------------------------- everything that does not need S
 struct LocalSmem {     // byte offsets
-  int b, q, k, v, m, t, th, tmp, row, total;
+  int b, q, k, m, t, tmp, row, total;
 };
 __host__ __device__ inline LocalSmem local_smem(int dkp, int dvp) {
   LocalSmem s;
   s.b = 0;                                        // [kC][dkp + 4] fp32
-  s.q = s.b + kC * (dkp + 4) * 4;                 // [kC][dkp + 8] bf16
-  s.k = s.q + kC * (dkp + 8) * 2;
-  s.v = s.k + kC * (dkp + 8) * 2;                 // [kC][dvp + 8]
-  s.m = s.v + kC * (dvp + 8) * 2;                 // [kC][kLdM] fp32, later T's parts [2][kC][kLdA] bf16
+  s.q = s.b + kC * (dkp + 4) * 4;                 // [kC][dkp + 8] bf16, later v [kC][dvp + 8]
+  s.k = s.q + kC * ((dkp > dvp ? dkp : dvp) + 8) * 2;
+  s.m = s.k + kC * (dkp + 8) * 2;                 // [kC][kLdM] fp32, later T's parts [2][kC][kLdA] bf16
   s.t = s.m + 2 * kC * kLdA * 2;                  // [kC][kLdM] fp32
   s.tmp = s.t + kC * kLdM * 4;                    // [3][16][17] fp32 / segment sums [kThreads]
   s.row = s.tmp + 3 * 16 * 17 * 4;                // 1 / |q|, 1 / |k|, beta: [3][kC]
@@ -116,7 +115,7 @@ __device__ __forceinline__ void block_products(const float* sB, int ldb, const b
   }
 }
 
-__global__ void __launch_bounds__(kThreads)
+__global__ void __launch_bounds__(kThreads, 2)
 delta_chunk_local_kernel(const ChunkParams p) {
   extern __shared__ __align__(16) unsigned char smem[];
   pdl_enter();
@@ -129,7 +128,7 @@ delta_chunk_local_kernel(const ChunkParams p) {
   float* sB = reinterpret_cast<float*>(smem + off.b);
   bf16* sq = reinterpret_cast<bf16*>(smem + off.q);
   bf16* sk = reinterpret_cast<bf16*>(smem + off.k);
-  bf16* sv = reinterpret_cast<bf16*>(smem + off.v);
+  bf16* sv = sq;                       // once q has been used
   float* sM = reinterpret_cast<float*>(smem + off.m);
   bf16* sTh = reinterpret_cast<bf16*>(smem + off.m);
   bf16* sTl = sTh + kC * kLdA;
@@ -153,7 +152,6 @@ delta_chunk_local_kernel(const ChunkParams p) {
   };
   copy_rows(sq, ldk, g * dkp, dkp);
   copy_rows(sk, ldk, (a.G + g) * dkp, dkp);
-  copy_rows(sv, ldv, 2 * a.G * dkp + h * dvp, dvp);
   copy_commit();
   if (tid < kC) {
     const bool ok = tid < n;
@@ -171,14 +169,21 @@ delta_chunk_local_kernel(const ChunkParams p) {
     if (seg < segs) {
       const float bias = a.dt_bias[h * dkp + c];
       const float* z = a.zg + row0 * a.ldz + h * dkp + c;
-      for (int t0 = seg * len; t0 < (seg + 1) * len; t0 += 8) {
-        float zv[8];
+      constexpr int kAhead = 8;
+      float zv[kAhead], nx[kAhead];
+      auto load = [&](int t0, float (&v)[kAhead]) {
 #pragma unroll
-        for (int x = 0; x < 8; ++x) zv[x] = t0 + x < n ? z[(t0 + x) * a.ldz] : 0.f;
+        for (int x = 0; x < kAhead; ++x) v[x] = t0 + x < n ? z[(t0 + x) * a.ldz] : 0.f;
+      };
+      const int t_end = (seg + 1) * len;
+      load(seg * len, zv);
+      for (int t0 = seg * len; t0 < t_end; t0 += kAhead) {
+        if (t0 + kAhead < t_end) load(t0 + kAhead, nx);
 #pragma unroll
-        for (int x = 0; x < 8; ++x) {
-          if (t0 + x < n) sum -= rate * softplus_precise(zv[x] + bias);
+        for (int x = 0; x < kAhead; ++x) {
+          if (t0 + x < n) sum -= rate * softplus_fast(zv[x] + bias);
           sB[(t0 + x) * ldb + c] = sum;
+          zv[x] = nx[x];
         }
       }
       s_tmp[seg * dkp + c] = sum;
@@ -256,6 +261,8 @@ delta_chunk_local_kernel(const ChunkParams p) {
     }
   }
   __syncthreads();
+  copy_rows(sv, ldv, 2 * a.G * dkp + h * dvp, dvp);
+  copy_commit();
   // ---- T = (I + sM)^-1: diagonal blocks by forward substitution, a column per lane ...
   if (warp < 4) {
     const int d0 = warp * 16;
@@ -278,6 +285,7 @@ delta_chunk_local_kernel(const ChunkParams p) {
     for (int j = 0; j + dist < 4; ++j) {
       const int i = j + dist;
       float v = 0.f;
+#pragma unroll 16
       for (int s = j * 16; s < i * 16; ++s) v = fmaf(sM[(i * 16 + br) * kLdM + s], sT[s * kLdM + j * 16 + bc], v);
       s_tmp[(j * 16 + br) * 17 + bc] = v;
     }
@@ -298,6 +306,7 @@ delta_chunk_local_kernel(const ChunkParams p) {
     const float v0 = ok ? sT[t * kLdM + s] * s_beta[s] : 0.f, v1 = ok ? sT[t * kLdM + s + 1] * s_beta[s + 1] : 0.f;
     store_split2(sTh + t * kLdA + s, sTl + t * kLdA + s, s <= t ? v0 : 0.f, s + 1 <= t ? v1 : 0.f);
   }
+  copy_wait<0>();
   __syncthreads();
   // ---- W = T K~ and U0 = T V: a warp takes 16 columns for all 64 rows
   const int k_cols = dkp / 16, v_cols = dvp / 16, r_lo = lane >> 2, c_lo = (lane & 3) * 2;

@@ -326,19 +326,26 @@ latent_finish_kernel(const DecodeParams p) {
     if (lane < p.splits) s_w[i][lane] = sum > 0.f ? f / sum : 0.f;
   }
   __syncthreads();
+#pragma unroll 2
   for (int i = threadIdx.x; i < 16 * per; i += kThreads) {
     const int r = i / per, c = (i - r * per) * 8, row = m0 + r;
     float o[8] = {};
     if (row < rows) {
       const int b = row / a.S, t = row - b * a.S;
       const float* src = p.o + (static_cast<long long>(b) * p.splits * R + t * a.H + h) * a.rankp + c;
-      for (int s = 0; s < p.splits; ++s) {
-        const float w = s_w[r][s];
-        if (w == 0.f) continue;
-        float f[8];
-        load8(src + static_cast<long long>(s) * R * a.rankp, f);
+      for (int s0 = 0; s0 < p.splits; s0 += 4) {
+        float w[4], f[4][8];
 #pragma unroll
-        for (int e = 0; e < 8; ++e) o[e] = fmaf(w, f[e], o[e]);
+        for (int x = 0; x < 4; ++x) {
+          w[x] = s0 + x < p.splits ? s_w[r][s0 + x] : 0.f;   // zero: the split has no rows to read
+          if (w[x] != 0.f) load8(src + static_cast<long long>(s0 + x) * R * a.rankp, f[x]);
+        }
+#pragma unroll
+        for (int x = 0; x < 4; ++x)
+          if (w[x] != 0.f) {
+#pragma unroll
+            for (int e = 0; e < 8; ++e) o[e] = fmaf(w[x], f[x][e], o[e]);
+          }
       }
     }
     store8(sa + r * ld + c, o);
