@@ -486,8 +486,7 @@ cudaError_t launch_prepare(const DeltaParams& p, cudaStream_t st) {
 template <typename T, int M>
 cudaError_t launch_sequence_m(const DeltaParams& p, cudaStream_t st) {
   const size_t bytes = (3 * kSteps * p.dkp + kSteps * kCols + 2 * kSteps) * sizeof(float);
-  cudaError_t e = cudaFuncSetAttribute(delta_sequence_kernel<T, M>, cudaFuncAttributeMaxDynamicSharedMemorySize,
-                                       static_cast<int>(bytes));
+  cudaError_t e = allow_smem<delta_sequence_kernel<T, M>>(static_cast<int>(bytes));
   if (e != cudaSuccess) return e;
   return launch_kernel(delta_sequence_kernel<T, M>, dim3((p.dvp + kCols - 1) / kCols, p.H, p.B), dim3(kThreads), bytes,
                        st, p);

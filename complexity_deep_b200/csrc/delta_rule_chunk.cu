@@ -592,10 +592,9 @@ int chunk_count(int S) { return (S + kC - 1) / kC; }
 template <int NB, int KT>
 cudaError_t launch_scan(const ChunkParams& p, cudaStream_t st) {
   const int bytes = scan_smem(p.a.dkp, NB).total;
-  auto kern = delta_chunk_scan_kernel<NB, KT>;
-  cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, bytes);
+  cudaError_t e = allow_smem<delta_chunk_scan_kernel<NB, KT>>(bytes);
   if (e != cudaSuccess) return e;
-  return launch_kernel(kern, dim3((p.a.dvp + NB - 1) / NB, p.a.H, p.a.B), dim3(kThreads), bytes, st, p);
+  return launch_kernel(delta_chunk_scan_kernel<NB, KT>, dim3((p.a.dvp + NB - 1) / NB, p.a.H, p.a.B), dim3(kThreads), bytes, st, p);
 }
 
 struct Sizes {         // bytes per (sequence, head, chunk)
@@ -637,7 +636,7 @@ cudaError_t launch_delta_chunk(const DeltaParams& a, void* ws, cudaStream_t st) 
   p.att = reinterpret_cast<bf16*>(take(s.att));
   p.total = reinterpret_cast<float*>(take(s.total));
   const int bytes = local_smem(a.dkp, a.dvp).total;
-  cudaError_t e = cudaFuncSetAttribute(delta_chunk_local_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, bytes);
+  cudaError_t e = allow_smem<delta_chunk_local_kernel>(bytes);
   if (e != cudaSuccess) return e;
   e = launch_kernel(delta_chunk_local_kernel, dim3(p.chunks, a.H, a.B), dim3(kThreads), bytes, st, p);
   if (e != cudaSuccess) return e;

@@ -1,5 +1,6 @@
 // Internal launch functions shared by the translation units of libcdeep.so.
 #pragma once
+#include <atomic>
 #include <cstddef>
 #include <cstdlib>
 #include <cuda_runtime.h>
@@ -32,6 +33,16 @@ inline cudaError_t launch_kernel(void (*kern)(P...), dim3 grid, dim3 block, size
   cfg.attrs = attr;
   cfg.numAttrs = 1;
   return cudaLaunchKernelEx(&cfg, kern, static_cast<A&&>(args)...);
+}
+
+// Raises a kernel's limit of dynamic shared memory; asks the driver only when it grows.
+template <auto kKernel>
+inline cudaError_t allow_smem(int bytes) {
+  static std::atomic<int> allowed{0};
+  if (bytes <= allowed.load(std::memory_order_relaxed)) return cudaSuccess;
+  const cudaError_t e = cudaFuncSetAttribute(kKernel, cudaFuncAttributeMaxDynamicSharedMemorySize, bytes);
+  if (e == cudaSuccess) allowed.store(bytes, std::memory_order_relaxed);
+  return e;
 }
 
 size_t route_workspace_bytes(int T, int E);
