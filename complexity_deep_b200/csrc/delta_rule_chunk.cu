@@ -378,16 +378,18 @@ __host__ __device__ inline ScanSmem scan_smem(int dkp, int nb) {
   return s;
 }
 
-// NB value columns per block; the warps tile the state as KT row tiles of 16 (dkp <= 16 KT) by 8 / KT column
-// slices, and the chunk's rows as four row tiles by two column slices
-template <int NB, int KT>
-__global__ void __launch_bounds__(kThreads)
+// NB value columns per block; the NW warps tile the state as KT row tiles of 16 (dkp <= 16 KT) by NW / KT
+// column slices, and the chunk's rows as four row tiles by NW / 4 column slices
+template <int NB, int KT, int NW>
+__global__ void __launch_bounds__(NW * 32, 1)
 delta_chunk_scan_kernel(const ChunkParams p) {
   extern __shared__ __align__(16) unsigned char smem[];
   pdl_enter();
   const DeltaParams& a = p.a;
-  constexpr int kSlices = 8 / KT, kSN = NB / 8 / kSlices;     // n-tiles of the state per warp
-  constexpr int kON = NB / 16;                                // n-tiles of U and O per warp
+  constexpr int kThreads = NW * 32;
+  constexpr int kSlices = NW / KT, kSN = NB / 8 / kSlices;    // n-tiles of the state per warp
+  constexpr int kON = NB / 8 / (NW / 4);                      // n-tiles of U and O per warp
+  static_assert(kSN % 2 == 0 && kON % 2 == 0, "column slices are pairs of n-tiles");
   constexpr int ldn = NB + 8;
   const int col0 = blockIdx.x * NB, h = blockIdx.y, b = blockIdx.z;
   const int dkp = a.dkp, dvp = a.dvp, ldk = dkp + 8;
@@ -451,7 +453,7 @@ delta_chunk_scan_kernel(const ChunkParams p) {
   };
   put_state();
 
-  const int mt = warp & 3, oc = (warp >> 2) * (NB / 2);       // this warp's rows and columns of U and O
+  const int mt = warp & 3, oc = (warp >> 2) * (kON * 8);       // this warp's rows and columns of U and O
   // acc += x S for this warp's tile; x: [2][kC][ldk] in shared memory
   auto times_state = [&](const bf16* x, float (&acc)[kON][4]) {
 #pragma unroll 2
@@ -589,12 +591,25 @@ delta_chunk_scan_kernel(const ChunkParams p) {
 
 int chunk_count(int S) { return (S + kC - 1) / kC; }
 
-template <int NB, int KT>
+template <int NB, int KT, int NW>
 cudaError_t launch_scan(const ChunkParams& p, cudaStream_t st) {
   const int bytes = scan_smem(p.a.dkp, NB).total;
-  cudaError_t e = allow_smem<delta_chunk_scan_kernel<NB, KT>>(bytes);
+  cudaError_t e = allow_smem<delta_chunk_scan_kernel<NB, KT, NW>>(bytes);
   if (e != cudaSuccess) return e;
-  return launch_kernel(delta_chunk_scan_kernel<NB, KT>, dim3((p.a.dvp + NB - 1) / NB, p.a.H, p.a.B), dim3(kThreads), bytes, st, p);
+  return launch_kernel(delta_chunk_scan_kernel<NB, KT, NW>, dim3((p.a.dvp + NB - 1) / NB, p.a.H, p.a.B), dim3(NW * 32),
+                       bytes, st, p);
+}
+
+// Columns per block: rounds of blocks (one block per SM) times the measured relative time of a block
+int pick_columns(const DeltaParams& a) {
+  const int sms = current_sm_count();
+  auto cost = [&](int nb, int t) {
+    const long long blocks = static_cast<long long>(a.B) * a.H * ((a.dvp + nb - 1) / nb);
+    return (blocks + sms - 1) / sms * t;
+  };
+  const long long c32 = cost(32, 75), c64 = cost(64, 100), c128 = cost(128, 130);
+  if (c128 < c64 && c128 < c32) return 128;
+  return c64 <= c32 ? 64 : 32;
 }
 
 struct Sizes {         // bytes per (sequence, head, chunk)
@@ -640,11 +655,11 @@ cudaError_t launch_delta_chunk(const DeltaParams& a, void* ws, cudaStream_t st) 
   if (e != cudaSuccess) return e;
   e = launch_kernel(delta_chunk_local_kernel, dim3(p.chunks, a.H, a.B), dim3(kThreads), bytes, st, p);
   if (e != cudaSuccess) return e;
-  // slices of 64 columns when they fill the SMs, else of 32
-  const bool wide = static_cast<long long>(a.B) * a.H * ((a.dvp + 63) / 64) * 4 >= 3LL * current_sm_count();
-  if (a.dkp <= 32) return launch_scan<64, 2>(p, st);
-  if (a.dkp <= 64) return wide ? launch_scan<64, 4>(p, st) : launch_scan<32, 4>(p, st);
-  return wide ? launch_scan<64, 8>(p, st) : launch_scan<32, 8>(p, st);
+  const int nb = pick_columns(a);
+  if (a.dkp <= 32) return launch_scan<64, 2, 8>(p, st);
+  if (a.dkp <= 64)
+    return nb == 32 ? launch_scan<32, 4, 8>(p, st) : nb == 64 ? launch_scan<64, 4, 8>(p, st) : launch_scan<128, 4, 16>(p, st);
+  return nb == 32 ? launch_scan<32, 8, 8>(p, st) : nb == 64 ? launch_scan<64, 8, 8>(p, st) : launch_scan<128, 8, 16>(p, st);
 }
 
 }  // namespace cdeep
