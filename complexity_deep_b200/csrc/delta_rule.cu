@@ -119,7 +119,7 @@ delta_prepare_window_kernel(const DeltaParams p) {
       for (int e = 0; e < 8; ++e) y[e] = fmaf(w[j][e], win[(x - j + kWindow) % kWindow][e], y[e]);
 #pragma unroll
     for (int e = 0; e < 8; ++e) {
-      y[e] = to_f32(from_f32<T>(sizeof(T) == 2 ? y[e] / (1.0f + exp2_approx(-1.4426950408889634f * y[e])) : silu_precise(y[e])));
+      y[e] = to_f32(from_f32<T>(sizeof(T) == 2 ? silu_fast(y[e]) : silu_precise(y[e])));
       ss += y[e] * y[e];
     }
 #pragma unroll

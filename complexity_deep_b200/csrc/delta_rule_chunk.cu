@@ -142,13 +142,12 @@ delta_chunk_local_kernel(const ChunkParams p) {
 
   // ---- rows of q, k, v (zero beyond the sequence), norms, beta
   const bf16* act = static_cast<const bf16*>(a.act) + row0 * C;
-  auto copy_rows = [&](bf16* dst, int ld, int col, int width) {
-    const int per = width / 8;
-    for (int i = tid; i < kC * per; i += kThreads) {
-      const int t = i / per, c = (i - t * per) * 8;
-      if (t < n) copy16_async(dst + t * ld + c, act + static_cast<long long>(t) * C + col + c);
-      else *reinterpret_cast<uint4*>(dst + t * ld + c) = make_uint4(0, 0, 0, 0);
-    }
+  auto copy_rows = [&](bf16* dst, int ld, int col, int width) {       // half a warp per row
+    for (int t = tid >> 4; t < kC; t += kThreads / 16)
+      for (int c = (tid & 15) * 8; c < width; c += 128) {
+        if (t < n) copy16_async(dst + t * ld + c, act + static_cast<long long>(t) * C + col + c);
+        else *reinterpret_cast<uint4*>(dst + t * ld + c) = make_uint4(0, 0, 0, 0);
+      }
   };
   copy_rows(sq, ldk, g * dkp, dkp);
   copy_rows(sk, ldk, (a.G + g) * dkp, dkp);
@@ -248,16 +247,17 @@ delta_chunk_local_kernel(const ChunkParams p) {
   {
     bf16* qh = p.q + slot * 2 * kC * dkp;
     bf16* kh = p.k + slot * 2 * kC * dkp;
-    const int half = dkp / 2;
-    for (int i = tid; i < kC * half; i += kThreads) {
-      const int t = i / half, c = (i - t * half) * 2;
-      const float2 bt = *reinterpret_cast<const float2*>(sB + t * ldb + c);
+    for (int c = lane * 2; c < dkp; c += 64) {
       const float2 bl = *reinterpret_cast<const float2*>(sB + (kC - 1) * ldb + c);
-      const float2 qv = pair_of(sq + t * ldk + c), kv = pair_of(sk + t * ldk + c);
-      const float iq = s_iq[t], ik = s_ik[t];
-      store_split2(qh + t * dkp + c, qh + (kC + t) * dkp + c, qv.x * iq * exp2_approx(bt.x), qv.y * iq * exp2_approx(bt.y));
-      store_split2(kh + t * dkp + c, kh + (kC + t) * dkp + c, kv.x * ik * exp2_approx(bl.x - bt.x),
-                   kv.y * ik * exp2_approx(bl.y - bt.y));
+#pragma unroll 4
+      for (int t = warp; t < kC; t += kThreads / 32) {
+        const float2 bt = *reinterpret_cast<const float2*>(sB + t * ldb + c);
+        const float2 qv = pair_of(sq + t * ldk + c), kv = pair_of(sk + t * ldk + c);
+        const float iq = s_iq[t], ik = s_ik[t];
+        const int at = t * dkp + c;
+        store_split2(qh + at, qh + kC * dkp + at, qv.x * iq * exp2_approx(bt.x), qv.y * iq * exp2_approx(bt.y));
+        store_split2(kh + at, kh + kC * dkp + at, kv.x * ik * exp2_approx(bl.x - bt.x), kv.y * ik * exp2_approx(bl.y - bt.y));
+      }
     }
   }
   __syncthreads();
@@ -309,6 +309,8 @@ delta_chunk_local_kernel(const ChunkParams p) {
   copy_wait<0>();
   __syncthreads();
   // ---- W = T K~ and U0 = T V: a warp takes 16 columns for all 64 rows
+  float* u0 = p.u0 + slot * kC * dvp;
+  bf16* wh = p.w + slot * 2 * kC * dkp;
   const int k_cols = dkp / 16, v_cols = dvp / 16, r_lo = lane >> 2, c_lo = (lane & 3) * 2;
   for (int item = warp; item < k_cols + v_cols; item += kThreads / 32) {
     const bool is_v = item >= k_cols;
@@ -354,10 +356,9 @@ delta_chunk_local_kernel(const ChunkParams p) {
         for (int r = 0; r < 2; ++r) {
           const int t = mt * 16 + r_lo + r * 8, c = col + y * 8 + c_lo;
           if (is_v)
-            *reinterpret_cast<float2*>(p.u0 + (slot * kC + t) * dvp + c) = make_float2(acc[mt][y][2 * r], acc[mt][y][2 * r + 1]);
+            *reinterpret_cast<float2*>(u0 + t * dvp + c) = make_float2(acc[mt][y][2 * r], acc[mt][y][2 * r + 1]);
           else
-            store_split2(p.w + (slot * 2 * kC + t) * dkp + c, p.w + (slot * 2 * kC + kC + t) * dkp + c, acc[mt][y][2 * r],
-                         acc[mt][y][2 * r + 1]);
+            store_split2(wh + t * dkp + c, wh + (kC + t) * dkp + c, acc[mt][y][2 * r], acc[mt][y][2 * r + 1]);
         }
   }
 }
@@ -404,12 +405,9 @@ delta_chunk_scan_kernel(const ChunkParams p) {
   const long long slot0 = (static_cast<long long>(b) * a.H + h) * p.chunks;
   const long long row0 = static_cast<long long>(b) * a.S;
 
-  const int per = dkp / 8;
-  auto fetch = [&](bf16* dst, const bf16* src) {              // [2][kC][dkp] -> [2][kC][ldk]
-    for (int i = tid; i < 2 * kC * per; i += kThreads) {
-      const int t = i / per, c = (i - t * per) * 8;
-      copy16_async(dst + t * ldk + c, src + static_cast<long long>(t) * dkp + c);
-    }
+  auto fetch = [&](bf16* dst, const bf16* src) {              // [2][kC][dkp] -> [2][kC][ldk], half a warp per row
+    for (int t = tid >> 4; t < 2 * kC; t += kThreads / 16)
+      for (int c = (tid & 15) * 8; c < dkp; c += 128) copy16_async(dst + t * ldk + c, src + t * dkp + c);
   };
   auto fetch_w = [&](int n) { fetch(sw, p.w + (slot0 + n) * 2 * kC * dkp); };
   auto fetch_rest = [&](int n) {

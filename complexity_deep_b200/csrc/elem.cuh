@@ -98,6 +98,10 @@ template <typename T> __device__ __forceinline__ float score_log1p(float x) {
 }
 
 __device__ __forceinline__ float sigmoid_precise(float z) { return 1.0f / (1.0f + expf(-z)); }
+// silu for results that are rounded to bf16 (__fdividef returns 0 once the divisor passes 2^126, as silu does)
+__device__ __forceinline__ float silu_fast(float g) {
+  return __fdividef(g, 1.0f + exp2_approx(-1.4426950408889634f * g));
+}
 __device__ __forceinline__ float silu_precise(float g) { return g / (1.0f + expf(-g)); }
 
 }  // namespace cdeep
