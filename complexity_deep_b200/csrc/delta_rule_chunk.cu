@@ -143,11 +143,15 @@ delta_chunk_local_kernel(const ChunkParams p) {
   // ---- rows of q, k, v (zero beyond the sequence), norms, beta
   const bf16* act = static_cast<const bf16*>(a.act) + row0 * C;
   auto copy_rows = [&](bf16* dst, int ld, int col, int width) {       // half a warp per row
-    for (int t = tid >> 4; t < kC; t += kThreads / 16)
-      for (int c = (tid & 15) * 8; c < width; c += 128) {
-        if (t < n) copy16_async(dst + t * ld + c, act + static_cast<long long>(t) * C + col + c);
+    for (int c = (tid & 15) * 8; c < width; c += 128) {
+      const bf16* src = act + static_cast<long long>(tid >> 4) * C + col + c;
+#pragma unroll
+      for (int x = 0; x < kC / (kThreads / 16); ++x, src += static_cast<long long>(kThreads / 16) * C) {
+        const int t = (tid >> 4) + x * (kThreads / 16);
+        if (t < n) copy16_async(dst + t * ld + c, src);
         else *reinterpret_cast<uint4*>(dst + t * ld + c) = make_uint4(0, 0, 0, 0);
       }
+    }
   };
   copy_rows(sq, ldk, g * dkp, dkp);
   copy_rows(sk, ldk, (a.G + g) * dkp, dkp);
@@ -406,16 +410,22 @@ delta_chunk_scan_kernel(const ChunkParams p) {
   const long long row0 = static_cast<long long>(b) * a.S;
 
   auto fetch = [&](bf16* dst, const bf16* src) {              // [2][kC][dkp] -> [2][kC][ldk], half a warp per row
-    for (int t = tid >> 4; t < 2 * kC; t += kThreads / 16)
-      for (int c = (tid & 15) * 8; c < dkp; c += 128) copy16_async(dst + t * ldk + c, src + t * dkp + c);
+    const int c = (tid & 15) * 8;                             // dkp <= 128
+    if (c >= dkp) return;
+#pragma unroll
+    for (int x = 0; x < 2 * kC / (kThreads / 16); ++x) {
+      const int t = (tid >> 4) + x * (kThreads / 16);
+      copy16_async(dst + t * ldk + c, src + t * dkp + c);
+    }
   };
   auto fetch_w = [&](int n) { fetch(sw, p.w + (slot0 + n) * 2 * kC * dkp); };
   auto fetch_rest = [&](int n) {
     fetch(sq, p.q + (slot0 + n) * 2 * kC * dkp);
     fetch(sk, p.k + (slot0 + n) * 2 * kC * dkp);
     const bf16* src = p.att + (slot0 + n) * 2 * kC * kC;
-    for (int i = tid; i < 2 * kC * kC / 8; i += kThreads) {
-      const int t = i / (kC / 8), c = (i - t * (kC / 8)) * 8;
+#pragma unroll
+    for (int x = 0; x < 2 * kC * kC / 8 / kThreads; ++x) {
+      const int i = tid + x * kThreads, t = i / (kC / 8), c = (i - t * (kC / 8)) * 8;
       copy16_async(sa + t * kLdA + c, src + t * kC + c);
     }
   };

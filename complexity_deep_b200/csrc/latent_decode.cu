@@ -338,14 +338,16 @@ latent_finish_kernel(const DecodeParams p) {
   pdl_enter();
   const LatentParams& a = p.a;
   const int n0 = blockIdx.x * kValueCols, h = blockIdx.y, m0 = blockIdx.z * 16, rows = a.B * a.S;
-  const int R = a.S * a.H, ld = a.rankp + 8, per = a.rankp / 8;
+  const int R = a.S * a.H, ld = a.rankp + 8;
   bf16* sa = reinterpret_cast<bf16*>(smem);        // [16][ld]
   bf16* sb = sa + 16 * ld;                         // [kValueCols][ld]
   const bf16* uv = static_cast<const bf16*>(a.uv) + (static_cast<long long>(h) * a.vp + n0) * a.rankp;
-  for (int i = threadIdx.x; i < kValueCols * per; i += kThreads) {
-    const int r = i / per, c = (i - r * per) * 8;
-    if (n0 + r < a.vp) copy16_async(sb + r * ld + c, uv + static_cast<long long>(r) * a.rankp + c);
-    else *reinterpret_cast<uint4*>(sb + r * ld + c) = make_uint4(0, 0, 0, 0);
+  {
+    const int r = threadIdx.x / (kThreads / kValueCols);
+    for (int c = threadIdx.x % (kThreads / kValueCols) * 8; c < a.rankp; c += kThreads / kValueCols * 8) {
+      if (n0 + r < a.vp) copy16_async(sb + r * ld + c, uv + r * a.rankp + c);
+      else *reinterpret_cast<uint4*>(sb + r * ld + c) = make_uint4(0, 0, 0, 0);
+    }
   }
   copy_commit();
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
@@ -373,38 +375,29 @@ latent_finish_kernel(const DecodeParams p) {
     if (lane < p.splits) s_w[i][lane] = sum > 0.f ? f / sum : 0.f;
   }
   __syncthreads();
-  // four pieces of eight elements per thread, all in flight together
-  constexpr int kItems = 4;
-  for (int i0 = threadIdx.x; i0 < 16 * per; i0 += kItems * kThreads) {
+  // sixteen threads per row, up to four pieces of eight elements each, all in flight together
+  {
+    constexpr int kItems = 4;
+    const int i = threadIdx.x >> 4, row = m0 + i, c0 = (threadIdx.x & 15) * 8;
+    const bool live = row < rows;
+    const int b = live ? row / a.S : 0, t = live ? row - b * a.S : 0;
+    const float* src = p.o + (static_cast<long long>(b) * p.splits * R + t * a.H + h) * a.rankp + c0;
     float o[kItems][8] = {};
-    const float* src[kItems];
-    int row[kItems];
-#pragma unroll
-    for (int x = 0; x < kItems; ++x) {
-      const int i = i0 + x * kThreads, r = i / per;
-      row[x] = i < 16 * per && m0 + r < rows ? r : -1;
-      const int b = row[x] < 0 ? 0 : (m0 + r) / a.S, t = row[x] < 0 ? 0 : m0 + r - b * a.S;
-      src[x] = p.o + (static_cast<long long>(b) * p.splits * R + t * a.H + h) * a.rankp + (i - r * per) * 8;
-    }
+#pragma unroll 2
     for (int s = 0; s < p.splits; ++s) {
-      float f[kItems][8], w[kItems];
-#pragma unroll
-      for (int x = 0; x < kItems; ++x) {
-        w[x] = row[x] < 0 ? 0.f : s_w[row[x]][s];            // zero: the split has no rows to read
-        if (w[x] != 0.f) load8(src[x] + static_cast<long long>(s) * R * a.rankp, f[x]);
-      }
+      const float w = live ? s_w[i][s] : 0.f;                // zero: the split has no rows to read
+      float f[kItems][8] = {};
 #pragma unroll
       for (int x = 0; x < kItems; ++x)
-        if (w[x] != 0.f) {
+        if (w != 0.f && c0 + x * 128 < a.rankp) load8(src + static_cast<long long>(s) * R * a.rankp + x * 128, f[x]);
 #pragma unroll
-          for (int e = 0; e < 8; ++e) o[x][e] = fmaf(w[x], f[x][e], o[x][e]);
-        }
+      for (int x = 0; x < kItems; ++x)
+#pragma unroll
+        for (int e = 0; e < 8; ++e) o[x][e] = fmaf(w, f[x][e], o[x][e]);
     }
 #pragma unroll
-    for (int x = 0; x < kItems; ++x) {
-      const int i = i0 + x * kThreads, r = i / per;
-      if (i < 16 * per) store8(sa + r * ld + (i - r * per) * 8, o[x]);
-    }
+    for (int x = 0; x < kItems; ++x)
+      if (c0 + x * 128 < a.rankp) store8(sa + i * ld + c0 + x * 128, o[x]);
   }
   copy_wait<0>();
   __syncthreads();
