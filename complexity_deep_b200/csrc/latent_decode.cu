@@ -375,25 +375,27 @@ latent_finish_kernel(const DecodeParams p) {
     if (lane < p.splits) s_w[i][lane] = sum > 0.f ? f / sum : 0.f;
   }
   __syncthreads();
-  // sixteen threads per row, up to four pieces of eight elements each, all in flight together
+  // sixteen threads per row, up to four pieces of eight elements each.  Every load is made, all in flight
+  // together: what a split without rows left in the workspace is replaced by zero afterwards.
   {
     constexpr int kItems = 4;
-    const int i = threadIdx.x >> 4, row = m0 + i, c0 = (threadIdx.x & 15) * 8;
-    const bool live = row < rows;
-    const int b = live ? row / a.S : 0, t = live ? row - b * a.S : 0;
-    const float* src = p.o + (static_cast<long long>(b) * p.splits * R + t * a.H + h) * a.rankp + c0;
+    const int i = threadIdx.x >> 4, row = min(m0 + i, rows - 1), c0 = (threadIdx.x & 15) * 8;
+    const int b = row / a.S, t = row - b * a.S;
+    const float* src = p.o + (static_cast<long long>(b) * p.splits * R + t * a.H + h) * a.rankp;
+    int at[kItems];
+#pragma unroll
+    for (int x = 0; x < kItems; ++x) at[x] = c0 + x * 128 < a.rankp ? c0 + x * 128 : 0;
     float o[kItems][8] = {};
 #pragma unroll 2
-    for (int s = 0; s < p.splits; ++s) {
-      const float w = live ? s_w[i][s] : 0.f;                // zero: the split has no rows to read
-      float f[kItems][8] = {};
+    for (int s = 0; s < p.splits; ++s, src += static_cast<long long>(R) * a.rankp) {
+      const float w = s_w[i][s];
+      float f[kItems][8];
+#pragma unroll
+      for (int x = 0; x < kItems; ++x) load8(src + at[x], f[x]);
 #pragma unroll
       for (int x = 0; x < kItems; ++x)
-        if (w != 0.f && c0 + x * 128 < a.rankp) load8(src + static_cast<long long>(s) * R * a.rankp + x * 128, f[x]);
 #pragma unroll
-      for (int x = 0; x < kItems; ++x)
-#pragma unroll
-        for (int e = 0; e < 8; ++e) o[x][e] = fmaf(w, f[x][e], o[x][e]);
+        for (int e = 0; e < 8; ++e) o[x][e] = fmaf(w, w != 0.f ? f[x][e] : 0.f, o[x][e]);
     }
 #pragma unroll
     for (int x = 0; x < kItems; ++x)
@@ -446,7 +448,7 @@ int pick_mt(const LatentParams& a) {
 }
 
 // Key ranges per row tile: fewest rounds of blocks, counting about four tiles per block for its start
-// and end.
+// and end, and half a tile per range for the sum over them.
 int pick_splits(const LatentParams& a) {
   const int mt = pick_mt(a);
   const int sms = current_sm_count() * (attend_smem(a.rankp + a.rotp, mt).total <= kHalfSmem && mt == 1 ? 2 : 1);
@@ -455,7 +457,7 @@ int pick_splits(const LatentParams& a) {
   int best = 1;
   long long cost = -1;
   for (int s = 1; s <= kMaxSplits && s <= tiles; ++s) {
-    const long long c = (blocks * s + sms - 1) / sms * ((tiles + s - 1) / s + 4);
+    const long long c = (blocks * s + sms - 1) / sms * ((tiles + s - 1) / s + 4) * 2 + s;
     if (cost < 0 || c < cost) {
       cost = c;
       best = s;
