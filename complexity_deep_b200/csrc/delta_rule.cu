@@ -246,36 +246,13 @@ __device__ __forceinline__ void block_add(float (&v)[N], float* s) {
   }
 }
 
-// A channel's convolution inputs of one token, loaded before any is used
+// One of the values that a step needs before its recurrence: a channel of q, k or v after convolution and
+// silu, or a decay.  Loaded before it is used, so that a thread has several on the way.
 template <typename T>
-struct ConvTap {
+struct StepItem {
   T x[kWindow], w[kWindow];
+  float z;
 };
-template <typename T>
-__device__ __forceinline__ void conv_load(const DeltaParams& p, const T* now, const T* ring, int channel, int C, int pos,
-                                          ConvTap<T>& r) {
-  const T* taps = static_cast<const T*>(p.taps_w) + channel;
-  r.x[0] = *now;
-  r.w[0] = taps[static_cast<long long>(p.taps - 1) * C];
-#pragma unroll
-  for (int j = 1; j < kWindow; ++j) {
-    const bool ok = j < p.taps && j <= pos;
-    r.x[j] = ok ? ring[static_cast<long long>((pos - j) % p.taps) * C + channel] : from_f32<T>(0.f);
-    r.w[j] = ok ? taps[static_cast<long long>(p.taps - 1 - j) * C] : from_f32<T>(0.f);
-  }
-}
-template <typename T>
-__device__ __forceinline__ float conv_value(const DeltaParams& p, const T* ring, int channel, int C, int pos,
-                                            const ConvTap<T>& r) {
-  float y = 0.f;
-  for (int j = p.taps - 1; j >= kWindow; --j)               // more taps than the window holds
-    if (j <= pos)
-      y = fmaf(to_f32(static_cast<const T*>(p.taps_w)[static_cast<long long>(p.taps - 1 - j) * C + channel]),
-               to_f32(ring[static_cast<long long>((pos - j) % p.taps) * C + channel]), y);
-#pragma unroll
-  for (int j = kWindow - 1; j >= 0; --j) y = fmaf(to_f32(r.w[j]), to_f32(r.x[j]), y);
-  return to_f32(from_f32<T>(silu_precise(y)));
-}
 
 // A block per head and sequence does the whole step: convolution, norms, decay, recurrence, head norm,
 // gate.  A thread keeps RP rows of four columns of the state in registers (loaded before anything
@@ -306,42 +283,69 @@ delta_step_kernel(const DeltaParams p) {
                              : make_float4(0.f, 0.f, 0.f, 0.f);
   }
   const int pos = first_position(p);
-  const T* ring = static_cast<const T*>(p.ring) + static_cast<long long>(b) * p.taps * C;
-  T* here = static_cast<T*>(p.ring) + (static_cast<long long>(b) * p.taps + pos % p.taps) * C;
-  const bool first = h % rep == 0;
+  T* ring = static_cast<T*>(p.ring) + static_cast<long long>(b) * p.taps * C;
+  const T* taps = static_cast<const T*>(p.taps_w);
+  int back[kWindow];                      // offset in the ring of the input j tokens back, -1: none
+#pragma unroll
+  for (int j = 0; j < kWindow; ++j) back[j] = j < p.taps && j <= pos ? (pos - j) % p.taps * C : -1;
+  const bool first = h % rep == 0;        // the block that brings the ring up to date for its q / k head
   const float rate = p.rate[h];
   const float* zg = p.zg + b * p.ldz;
+  // items: q, k, v channels, decays
+  const int n_k = dkp, n_v = 2 * dkp, n_g = n_v + dvp, total = n_g + dkp;
+  auto channel_of = [&](int i) { return i < n_v ? (i < n_k ? g * dkp + i : (p.G + g) * dkp + i - n_k) : 2 * p.G * dkp + h * dvp + i - n_v; };
+  auto load = [&](int i, StepItem<T>& r) {
+    if (i >= total) return;
+    if (i >= n_g) {
+      const int c = h * dkp + i - n_g;
+      r.z = zg[c] + p.dt_bias[c];
+      return;
+    }
+    const T* in = i < n_k ? static_cast<const T*>(p.q) + g * dkp + i
+                          : i < n_v ? static_cast<const T*>(p.k) + g * dkp + i - n_k
+                                    : static_cast<const T*>(p.v) + h * dvp + i - n_v;
+    const int ch = channel_of(i);
+    r.x[0] = in[b * p.ldp];
+    r.w[0] = taps[(p.taps - 1) * C + ch];
+#pragma unroll
+    for (int j = 1; j < kWindow; ++j) {
+      r.x[j] = back[j] >= 0 ? ring[back[j] + ch] : from_f32<T>(0.f);
+      r.w[j] = back[j] >= 0 ? taps[(p.taps - 1 - j) * C + ch] : from_f32<T>(0.f);
+    }
+  };
+  auto finish = [&](int i, const StepItem<T>& r) {
+    if (i >= total) return;
+    if (i >= n_g) {
+      sg[i - n_g] = sizeof(T) == 2 ? exp2_approx(-rate * 1.4426950408889634f * softplus_fast(r.z))
+                                   : expf(-rate * softplus_precise(r.z));
+      return;
+    }
+    const int ch = channel_of(i);
+    float y = 0.f;
+    for (int j = p.taps - 1; j >= kWindow; --j)             // more taps than the window holds
+      if (j <= pos)
+        y = fmaf(to_f32(taps[(p.taps - 1 - j) * C + ch]), to_f32(ring[(pos - j) % p.taps * C + ch]), y);
+#pragma unroll
+    for (int j = kWindow - 1; j >= 0; --j) y = fmaf(to_f32(r.w[j]), to_f32(r.x[j]), y);
+    y = to_f32(from_f32<T>(sizeof(T) == 2 ? silu_fast(y) : silu_precise(y)));
+    if (i < n_v) sq[i] = y;               // k follows q
+    else sv[i - n_v] = y;
+    if (i >= n_v || first) ring[back[0] + ch] = r.x[0];
+  };
+  for (int i = tid; i < total; i += 2 * kThreads) {
+    StepItem<T> r0, r1;
+    load(i, r0);
+    load(i + kThreads, r1);
+    finish(i, r0);
+    finish(i + kThreads, r1);
+  }
+  __syncthreads();
   float sums[3] = {0.f, 0.f, 0.f};        // |q|^2, |k|^2, k . q
-  for (int c = tid; c < max(dkp, dvp); c += kThreads) {
-    const T* q_in = static_cast<const T*>(p.q) + b * p.ldp + g * dkp + c;
-    const T* k_in = static_cast<const T*>(p.k) + b * p.ldp + g * dkp + c;
-    const T* v_in = static_cast<const T*>(p.v) + b * p.ldp + h * dvp + c;
-    const int qc = g * dkp + c, kc = (p.G + g) * dkp + c, vc = 2 * p.G * dkp + h * dvp + c;
-    ConvTap<T> tq, tk, tv;
-    float z = 0.f;
-    if (c < dkp) {
-      conv_load(p, q_in, ring, qc, C, pos, tq);
-      conv_load(p, k_in, ring, kc, C, pos, tk);
-      z = zg[h * dkp + c] + p.dt_bias[h * dkp + c];
-    }
-    if (c < dvp) conv_load(p, v_in, ring, vc, C, pos, tv);
-    if (c < dkp) {
-      const float q = conv_value(p, ring, qc, C, pos, tq), k = conv_value(p, ring, kc, C, pos, tk);
-      sq[c] = q;
-      sk[c] = k;
-      sums[0] += q * q;
-      sums[1] += k * k;
-      sums[2] += k * q;
-      sg[c] = expf(-rate * softplus_precise(z));
-      if (first) {                        // this block brings the ring up to date
-        here[qc] = tq.x[0];
-        here[kc] = tk.x[0];
-      }
-    }
-    if (c < dvp) {
-      sv[c] = conv_value(p, ring, vc, C, pos, tv);
-      here[vc] = tv.x[0];
-    }
+  for (int c = tid; c < dkp; c += kThreads) {
+    const float q = sq[c], k = sk[c];
+    sums[0] += q * q;
+    sums[1] += k * k;
+    sums[2] += k * q;
   }
   block_add(sums, s_red);
   const float iq = 1.0f / sqrtf(static_cast<float>(p.dk)) / sqrtf(sums[0] + 1e-6f), ik = 1.0f / sqrtf(sums[1] + 1e-6f);
