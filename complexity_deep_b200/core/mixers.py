@@ -167,8 +167,8 @@ class GatedLinearAttention(Mixer):
 
 
 class LatentAttention(Mixer):
-    """Softmax attention over a cached low-rank latent and one rotated key part shared by all heads, with
-    a sigmoid gate per head (see cd_latent_attn in include/cdeep.h).  `positions`: most tokens of a
+    """Softmax attention over a cached low-rank latent beside a rotated key that the heads have in common,
+    with a sigmoid gate per head (see cd_latent_attn in include/cdeep.h).  `positions`: most tokens of a
     sequence; `rot_dims` of the `rot` rotated elements turn, with the given base."""
 
     def __init__(self, width: int, heads: int, dim: int, rot: int, vdim: int, rank: int, scale: float,
@@ -237,7 +237,7 @@ class LatentAttention(Mixer):
 
 
 class DeltaRule(Mixer):
-    """Gated delta rule with one decay per head and key channel, short convolutions ahead of q, k and v,
+    """Gated delta rule whose state decays at a rate per key channel, with short convolutions ahead of q, k and v,
     grouped q / k heads, a head norm and a sigmoid gate on the result (see cd_delta_attn in
     include/cdeep.h).  Decay and gate come from two-step projections of inner width `rank` and
     `gate_rank`, whose first steps are part of the common input projection."""

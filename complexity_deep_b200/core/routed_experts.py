@@ -14,8 +14,8 @@ from .padding import ROW_ALIGN, pad_rows, round_up
 class RoutedExperts(nn.Module):
     """sum over the chosen experts of weight * expert(x); expert(x) = down(g sigmoid(alpha g) (u + offset))
     with g = min(gate(x), limit), u = clamp(up(x), -limit, limit).  Of `groups` equal groups of experts
-    only the `keep` with the largest score can be chosen from; the weights are the chosen experts'
-    softmax scores divided by their sum."""
+    only the `keep` with the largest score can be chosen from; what is chosen is weighted in proportion to
+    its softmax score, weights adding up to one."""
 
     def __init__(self, hidden_size: int, intermediate_size: int, experts: int, top: int, limit: float,
                  groups: int = 1, keep: int = 1, alpha: float = 1.702, offset: float = 1.0):

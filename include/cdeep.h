@@ -496,8 +496,8 @@ size_t cd_gla_chunk_workspace_bytes(const cd_linear_attn* h_args);
 int cd_gla_chunk(const cd_linear_attn* h_args, void* workspace, size_t bytes, void* stream);
 
 /* ------------------------------------------------------------------ latent attention ---------
- * Causal attention over a cached low-rank latent c_j (rank wide, RMS-normed) and one rotated key part
- * r_j shared by all heads:
+ * Causal attention over a cached low-rank latent c_j (rank wide, RMS-normed) and a rotated key r_j that
+ * the heads have in common:
  *   s_h(i, j) = scale ((uk_h c_j) . q_h(i) + r_j . q'_h(i)),   w = softmax over j <= i
  *   out_h(i)  = out_scale sigmoid(gate_h(i)) sum_j w_h(i, j) uv_h c_j
  * q' and r are rotated by position (interleaved pairs).  The score equals (uk_h^T q_h) . c + q'_h . r, so
