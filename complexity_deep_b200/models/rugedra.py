@@ -216,6 +216,11 @@ class RugedraModel(StreamDecoder):
             if isinstance(m, (nn.Linear, nn.Embedding)):
                 nn.init.normal_(m.weight, std=0.02)
 
+    def new_state(self, batch: int, capacity: Optional[int] = None) -> DecoderState:
+        if capacity is not None and capacity > self.config.max_positions:
+            raise ValueError(f"a capacity of {capacity} tokens, but the model has {self.config.max_positions} positions")
+        return super().new_state(batch, capacity)
+
     # ------------------------------------------------------------------ forward
     def embed(self, input_ids: torch.Tensor, state: DecoderState) -> torch.Tensor:
         table = self.padded_rows("table", self.embed_tokens.weight)

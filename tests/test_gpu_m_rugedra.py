@@ -172,6 +172,8 @@ def test_more_tokens_than_positions_are_refused(tmp_path_factory):
     out = model(torch.tensor(tokens(cfg, limit)[None], device="cuda"), use_cache=True)
     with pytest.raises(RuntimeError):
         model(torch.zeros(1, 1, dtype=torch.int64, device="cuda"), past_key_values=out.past_key_values)
+    with pytest.raises(ValueError):
+        model.make_decode_cache(1, limit + 1)
 
 
 @pytest.mark.parametrize("dtype", ["bfloat16", "float32"])
